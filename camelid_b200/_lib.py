@@ -29,6 +29,17 @@ class Tensor(C.Structure):
     _fields_ = [("data", C.c_void_p), ("nbytes", C.c_uint64), ("qtype", C.c_int32), ("reserved", C.c_int32)]
 
 
+class LayerDesc(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("type", "heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "ff")] + [
+        ("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.POINTER(C.c_float))]
+
+
+class LayeredConfig(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("n_layers", "loop_start", "loop_stop", "loop_times", "streams", "width", "vocab", "max_pos",
+                                         "max_seqs", "dtype", "device", "flags")] + [
+        ("eps", C.c_float), ("layers", C.POINTER(LayerDesc))]
+
+
 def lib_path() -> Path:
     return PKG / "libcamelid_b200.so"
 
@@ -117,6 +128,14 @@ def lib():
         "cmld_engine_prefill_tokens": (i32, [vp, i32, vp, i64, i64, P(C.c_uint32)]),
         "cmld_engine_decode_greedy": (i32, [vp, i32, vp, vp, vp, i32, vp]),
         "cmld_engine_step_batch": (i32, [vp, i32, vp, vp, vp, vp, vp, vp]),
+        "cmld_engine_extend": (i32, [vp, i32, vp, i64, i64, vp, i32, vp, vp, P(C.c_uint32)]),
+        "cmld_engine_sample_row": (i32, [vp, i32, f32, f32, u64, P(C.c_uint32)]),
+        "cmld_engine_create_layered": (i32, [P(LayeredConfig), P(vp)]),
+        "cmld_engine_named_count": (i32, [vp]),
+        "cmld_engine_named_info": (i32, [vp, i32, P(C.c_char_p), P(i64), P(i64)]),
+        "cmld_engine_set_named": (i32, [vp, C.c_char_p, i32, vp, u64]),
+        "cmld_engine_synth_named": (i32, [vp, C.c_char_p, u64, u64, f32, f32]),
+        "cmld_engine_slot_filled": (i32, [vp, i32, P(i64)]),
         "cmld_engine_last_timing": (i32, [vp, P(f32), P(i64)]),
         "cmld_peer_wait_selftest": (i32, [i32]),
         "cmld_exact_sum_selftest": (i32, [vp, i32, vp]),

@@ -4,8 +4,10 @@
 """
 from __future__ import annotations
 
+import fcntl
 import hashlib
 import os
+import re
 import shutil
 import subprocess
 import sys
@@ -31,12 +33,31 @@ def nvcc() -> str:
     return cand
 
 
+def _with_headers(src: Path, seen: dict | None = None) -> dict:
+    """The source and every project header it includes, directly or not: path -> bytes."""
+    seen = {} if seen is None else seen
+    src = src.resolve()
+    if src not in seen and src.exists():
+        seen[src] = src.read_bytes()
+        for name in re.findall(rb'^\s*#\s*include\s+"([^"]+)"', seen[src], re.M):
+            _with_headers(src.parent / name.decode(), seen)
+    return seen
+
+
 def _stamp(src: Path, flags: list[str]) -> str:
     h = hashlib.sha256()
     h.update(" ".join(flags).encode())
-    for f in [src, CSRC / "common.cuh", PKG.parent / "include" / "camelid_b200.h", *sorted(CSRC.glob("*.cuh"))]:
-        h.update(f.read_bytes())
+    for _, text in sorted(_with_headers(src).items()):
+        h.update(text)
     return h.hexdigest()
+
+
+def build_locked() -> Path:
+    """``build()`` for programs that may start at the same time: one compiles, the others wait for it."""
+    OBJ.mkdir(exist_ok=True)
+    with open(OBJ / "lock", "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        return build()
 
 
 def build(force: bool = False, verbose: bool = False) -> Path:

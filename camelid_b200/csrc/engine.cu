@@ -3,12 +3,8 @@
 // `CudaResidentDecode` (src/cuda_resident.rs:15093 in the Camelid tree): same call surface,
 // same argument meaning, errors as status codes instead of Result<_, String>.
 #include <cmath>
-#include <string>
-#include <map>
-#include <tuple>
-#include <vector>
 
-#include "common.cuh"
+#include "engine.cuh"
 
 namespace cmld {
 
@@ -94,125 +90,6 @@ int32_t weight_upload(Weight &w, int32_t qt, int64_t rows, int64_t cols, const v
 
 // ------------------------------------------------------------------ engine
 
-struct LayerW {
-  Weight proj[7];  // q k v o gate up down
-  float *attn_norm = nullptr, *ffn_norm = nullptr;
-  bool dense_set = false;
-  // Mixtral
-  float *router = nullptr;
-  Weight exps[3];  // gate, up, down slabs: rows = n_experts * rows_per_expert
-  bool moe_set = false;
-};
-
-}  // namespace cmld
-
-using namespace cmld;
-
-struct cmld_engine {
-  cmld_config cfg{};   // dimensions of THIS rank: n_heads, n_kv_heads and ffn_dim are the tensor-parallel shares
-  cmld_config full{};  // the model's dimensions as given to cmld_engine_create
-  int32_t tp = 1, ep = 1, shard_rank = 0;
-  int32_t vocab_local = 0;  // rows of the output matrix held here
-  void *comm = nullptr;     // NCCL communicator of a sharded engine
-  unsigned long long *am_keys = nullptr;  // packed (value, index) per row for the sharded argmax
-  float *logits_gather = nullptr, *logits_full = nullptr;
-  // Peer-memory link of a tensor-parallel group: one region per rank, mapped into every rank.
-  //   parts: [2 slots][rank][kPeerRows][hidden] f32, then arrival words [2 slots][rank] u32
-  struct PeerLink {
-    bool ready = false;
-    uint8_t *region[kMaxPeers] = {};  // [shard_rank] is this rank's own allocation
-    uint32_t *local = nullptr;        // epochs[2], tickets[2]
-    unsigned long long timeout_ns = 0;
-  } peer;
-  float *mma_scratch = nullptr;  // per-chunk partial sums of the batched tensor-core matvec
-  uint8_t *kq8 = nullptr, *vq8 = nullptr;  // CMLD_FLAG_KV_Q8_0: the KV cache as Q8_0 blocks, [layer][slot][kv_head][max_pos][hd/32] x 34 B
-  int64_t kv_q8_bytes = 0;                 // bytes of one layer of one side
-  uint32_t *tree_mask = nullptr;  // [kTreeMaxNodes] ancestor masks of a draft tree (one word: at most 32 nodes)
-  std::vector<float> rope_freq;  // per-pair angular frequency of the engine-owned RoPE table (rope_pair_frequency)
-  uint8_t *tc5_pack = nullptr;   // packed activation records of the tcgen05 batched matvec
-  int64_t tc5_pack_bytes = 0;
-  int64_t mma_scratch_floats = 0;
-  unsigned long long *trace = nullptr;  // matvec timeline (environment CMLD_TRACE=<file>), dumped at destroy
-  unsigned long long *attn_phases = nullptr;  // with CMLD_TRACE: the last attention launch's phase clocks (8 words)
-  std::string trace_path;
-  std::map<int32_t, bool> peer_fit;   // rows -> every matvec of a step fits the staged kernel in one pass
-  int device = 0;
-  cudaStream_t stream = nullptr;
-  int32_t max_rows = 0;  // scratch rows (sequences per step)
-  int32_t n_splits = 1, sm_count = 148;
-  int32_t q_width = 0, kv_width = 0;
-  std::vector<LayerW> layers;
-  Weight output, token_embd;
-  float *final_norm = nullptr;
-  bool has_output = false, has_embd = false;
-  __half *kcache = nullptr, *vcache = nullptr;
-  int64_t kv_layer_elems = 0;  // halfs per layer per side
-  float *cos_all = nullptr, *sin_all = nullptr, *cos_step = nullptr, *sin_step = nullptr;
-  float *h = nullptr, *normed = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *attn = nullptr, *gate = nullptr,
-        *up = nullptr, *logits = nullptr, *taps = nullptr;
-  uint8_t *act_k = nullptr, *act_0 = nullptr;  // Q8_K and Q8_0 operand buffers (widest row)
-  float *attn_part = nullptr;
-  uint32_t *attn_tickets = nullptr;
-  float *am_val = nullptr;
-  int32_t *am_idx = nullptr;
-  uint32_t *am_ticket = nullptr;  // [2*max_rows]: tickets, then history lengths
-  int32_t *out_idx = nullptr, *d_tokens = nullptr, *d_positions = nullptr, *d_slots = nullptr, *d_history = nullptr;
-  int64_t history_cap = 0;
-  int32_t *moe_sel_idx = nullptr, *moe_counts = nullptr, *moe_lists = nullptr;
-  float *moe_sel_w = nullptr, *moe_g = nullptr, *moe_u = nullptr, *moe_act = nullptr, *moe_down = nullptr;
-  // tensor-core expert path: three Q8_K rows per assignment, `moe_cap` rows per local expert
-  int32_t *moe_pos = nullptr;
-  int32_t moe_cap = 0, moe_pass_rows = 0;
-  uint8_t *moe_act3_h = nullptr, *moe_act3_f = nullptr;
-  float *moe_g3 = nullptr, *moe_u3 = nullptr, *moe_d3 = nullptr, *moe_scratch = nullptr;
-  int64_t moe_scratch_floats = 0;
-  int32_t *d_status = nullptr;  // set by a kernel whose bounded wait gave up
-  int64_t filled = 0;
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-  float last_ms = 0.0f;
-  int64_t last_launches = 0, launches = 0;
-  std::vector<void *> allocs;
-  // CUDA graphs of whole steps, keyed by (rows, option bits, score-scale bits).  A key's first
-  // step runs as plain launches (it also sets kernel attributes); its second is captured.
-  struct StepGraph {
-    cudaGraphExec_t exec = nullptr;
-    int64_t launches = 0;
-    int uses = 0;
-  };
-  std::map<std::tuple<int32_t, uint32_t, uint32_t>, StepGraph> graphs;
-  bool graphs_off = false;
-};
-
-namespace cmld {
-
-struct DeviceGuard {
-  int prev = -1;
-  bool ok = true;
-  explicit DeviceGuard(int dev) {
-    if (cudaGetDevice(&prev) != cudaSuccess) ok = false;
-    if (ok && prev != dev && cudaSetDevice(dev) != cudaSuccess) ok = false;
-  }
-  ~DeviceGuard() {
-    if (prev >= 0) cudaSetDevice(prev);
-  }
-};
-
-#define CMLD_ENGINE_ENTER(e)                                              \
-  if (!(e)) return fail(CMLD_ERR_INVALID, "engine handle is null");       \
-  DeviceGuard guard__((e)->device);                                       \
-  if (!guard__.ok) return fail(CMLD_ERR_CUDA, "cannot select CUDA device %d", (e)->device)
-
-template <typename T>
-static int32_t dev_alloc(cmld_engine *e, T **p, int64_t count, bool zero = true) {
-  void *raw = nullptr;
-  const size_t bytes = (size_t)std::max<int64_t>(count, 1) * sizeof(T);
-  CMLD_CUDA(cudaMalloc(&raw, bytes));
-  e->allocs.push_back(raw);
-  if (zero) CMLD_CUDA(cudaMemsetAsync(raw, 0, bytes, e->stream));
-  *p = static_cast<T *>(raw);
-  return CMLD_OK;
-}
-
 // cos/sin of position * frequency for every position and pair, by the host libm, onto the device.
 static int32_t upload_rope_tables(cmld_engine *e) {
   const cmld_config &c = e->cfg;
@@ -251,13 +128,43 @@ static int32_t validate_config(const cmld_config &c) {
   return CMLD_OK;
 }
 
-static int32_t engine_init(cmld_engine *e) {
-  const cmld_config &c = e->cfg;
+// What every engine has, whatever its design: the device, a stream, two timing events.
+int32_t engine_open(cmld_engine *e, int32_t device) {
+  e->device = device;
   CMLD_CUDA(cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking));
   CMLD_CUDA(cudaEventCreate(&e->ev0));
   CMLD_CUDA(cudaEventCreate(&e->ev1));
+  e->sm_count = 148;
+  cudaDeviceGetAttribute(&e->sm_count, cudaDevAttrMultiProcessorCount, device);
+  return CMLD_OK;
+}
+
+// The rows of a step: token, position and slot of each, the logits of `logit_rows` of them, greedy argmax with its
+// history, the status word of bounded waits.
+int32_t init_rows(cmld_engine *e, int64_t rows, int64_t logit_rows, int64_t vocab_local) {
+  e->max_rows = (int32_t)rows;
+  e->logit_rows = (int32_t)logit_rows;
+  CMLD_TRY(dev_alloc(e, &e->logits, logit_rows * vocab_local));
+  CMLD_TRY(dev_alloc(e, &e->am_keys, logit_rows));
+  CMLD_TRY(dev_alloc(e, &e->am_val, logit_rows * argmax_blocks()));
+  CMLD_TRY(dev_alloc(e, &e->am_idx, logit_rows * argmax_blocks()));
+  CMLD_TRY(dev_alloc(e, &e->am_ticket, 2 * logit_rows));
+  CMLD_TRY(dev_alloc(e, &e->out_idx, logit_rows));
+  CMLD_TRY(dev_alloc(e, &e->d_tokens, rows));
+  CMLD_TRY(dev_alloc(e, &e->d_positions, rows));
+  CMLD_TRY(dev_alloc(e, &e->d_slots, rows));
+  e->history_cap = 4096;
+  CMLD_TRY(dev_alloc(e, &e->d_history, e->history_cap * logit_rows));
+  CMLD_TRY(dev_alloc(e, &e->d_status, 1));
+  return CMLD_OK;
+}
+
+static int32_t engine_init(cmld_engine *e) {
+  const cmld_config &c = e->cfg;
+  CMLD_TRY(engine_open(e, e->device));
   const int seqs = std::max(1, c.max_seqs);
-  e->max_rows = std::max(seqs, 32);  // a prompt is ingested 32 rows at a time (one tensor-core pass over the weights)
+  const int64_t R = std::max(seqs, 32);  // a prompt is ingested 32 rows at a time (one tensor-core pass over the weights)
+  CMLD_TRY(init_rows(e, R, R, e->vocab_local));
   e->q_width = c.n_heads * c.head_dim;
   e->kv_width = c.n_kv_heads * c.head_dim;
   e->layers.resize(c.n_layers);
@@ -289,7 +196,6 @@ static int32_t engine_init(cmld_engine *e) {
     CMLD_TRY(dev_alloc(e, &e->sin_all, (int64_t)c.max_pos * half, false));
     CMLD_TRY(upload_rope_tables(e));
   }
-  const int64_t R = e->max_rows;
   CMLD_TRY(dev_alloc(e, &e->cos_step, R * half));
   CMLD_TRY(dev_alloc(e, &e->sin_step, R * half));
   CMLD_TRY(dev_alloc(e, &e->h, R * c.hidden));
@@ -300,8 +206,6 @@ static int32_t engine_init(cmld_engine *e) {
   CMLD_TRY(dev_alloc(e, &e->attn, R * e->q_width));
   CMLD_TRY(dev_alloc(e, &e->gate, R * c.ffn_dim));
   CMLD_TRY(dev_alloc(e, &e->up, R * c.ffn_dim));
-  CMLD_TRY(dev_alloc(e, &e->logits, R * (int64_t)e->vocab_local));
-  CMLD_TRY(dev_alloc(e, &e->am_keys, R));
   if (e->tp > 1) {
     CMLD_TRY(dev_alloc(e, &e->logits_gather, R * (int64_t)c.vocab));
     CMLD_TRY(dev_alloc(e, &e->logits_full, R * (int64_t)c.vocab));
@@ -311,20 +215,11 @@ static int32_t engine_init(cmld_engine *e) {
   CMLD_TRY(dev_alloc(e, &e->act_k, R * act_row_stride(widest)));
   CMLD_TRY(dev_alloc(e, &e->act_0, R * act_row_stride(widest)));
   // flash-decoding splits: enough CTAs to cover the SMs twice at batch 1
-  int sms = 148;
-  cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, e->device);
-  e->sm_count = sms;
+  const int sms = e->sm_count;
   e->n_splits = std::max(1, std::min<int>(64, (2 * sms + c.n_kv_heads - 1) / c.n_kv_heads));
   e->n_splits = (int)std::min<int64_t>(e->n_splits, std::max<int64_t>(1, c.max_pos / 32));
   CMLD_TRY(dev_alloc(e, &e->attn_part, R * c.n_heads * e->n_splits * (c.head_dim + 2)));
   CMLD_TRY(dev_alloc(e, &e->attn_tickets, R * c.n_kv_heads));
-  CMLD_TRY(dev_alloc(e, &e->am_val, R * argmax_blocks()));
-  CMLD_TRY(dev_alloc(e, &e->am_idx, R * argmax_blocks()));
-  CMLD_TRY(dev_alloc(e, &e->am_ticket, 2 * R));
-  CMLD_TRY(dev_alloc(e, &e->out_idx, R));
-  CMLD_TRY(dev_alloc(e, &e->d_tokens, R));
-  CMLD_TRY(dev_alloc(e, &e->d_positions, R));
-  CMLD_TRY(dev_alloc(e, &e->d_slots, R));
   if (c.n_experts > 0) {
     const int64_t na = R * c.n_experts_used;
     CMLD_TRY(dev_alloc(e, &e->moe_sel_idx, na));
@@ -374,9 +269,6 @@ static int32_t engine_init(cmld_engine *e) {
     CMLD_TRY(dev_alloc(e, &e->trace, 1 + 8 * (int64_t)kTraceRecords + (int64_t)kTraceCtas * (1 + 4 * (int64_t)kTraceCtaRecords)));
     CMLD_TRY(dev_alloc(e, &e->attn_phases, 8));
   }
-  e->history_cap = 4096;
-  CMLD_TRY(dev_alloc(e, &e->d_history, e->history_cap * R));
-  CMLD_TRY(dev_alloc(e, &e->d_status, 1));
   CMLD_CUDA(cudaStreamSynchronize(e->stream));
   return CMLD_OK;
 }
@@ -452,6 +344,7 @@ static void engine_free(cmld_engine *e) {
   e->comm = nullptr;
   peer_link_close(e);
 
+  layered_free(e);
   for (auto &L : e->layers) {
     for (auto &w : L.proj) weight_free(w);
     for (auto &w : L.exps) weight_free(w);
@@ -652,24 +545,6 @@ static int32_t gemv_fused(cmld_engine *e, const Proj *p, int n, int32_t batch, i
   return run_gemv_group(e, p, n, batch);
 }
 
-struct StepOpts {
-  int32_t batch = 1;
-  bool from_tokens = false;    // gather embeddings of d_tokens, else h holds them
-  bool rope_by_position = true;  // index the engine's all-position table, else cos_step/sin_step rows
-  float scale = 0.0f;
-  bool logits = true;
-  bool argmax = true;
-  bool feed_back = false;  // argmax writes next token / position / history
-  bool taps = false;
-  int32_t layer_begin = 0, layer_end = -1;  // layers to run; -1 = through the last
-  bool attn_cluster = false;  // short contexts, few rows: attention ranges as a thread-block cluster (host-side choice)
-  int32_t attn_cap = 0;       // bound on the context length of every row of this step (a bucket: 1024, 2048, 4096, 8192), 0 = unknown
-  const uint32_t *tree_mask = nullptr;  // tree verification: per-row ancestor masks (device), nodes at cache rows tree_base..
-  int32_t tree_base = 0, tree_words = 0;
-  bool shared_slots = false;  // several rows of this step belong to one sequence (prefill, verify): row b
-                              // reads K/V that rows < b write, so the KV append must be a kernel of its own
-};
-
 // moe.cu
 int32_t moe_route(const float *normed, const float *router, int hidden, int n_exp, int k, int batch, int32_t *sel_idx,
                   float *sel_w, int32_t *counts, int32_t *lists, cudaStream_t s, int32_t *pos);
@@ -836,6 +711,7 @@ static bool peer_step_ok(cmld_engine *e, int32_t B, bool taps) {
 }
 
 static int32_t engine_step(cmld_engine *e, const StepOpts &o) {
+  if (e->lay) return layered_step(e, o);
   const cmld_config &c = e->cfg;
   const int32_t B = o.batch;
   const bool sharded = e->tp > 1 || e->ep > 1;
@@ -1074,13 +950,14 @@ static int32_t engine_step(cmld_engine *e, const StepOpts &o) {
 
 // A step through a CUDA graph when possible: one graph launch replaces ~200 kernel launches, and
 // the programmatic-dependent-launch edges between the matvec kernels are kept inside the graph.
-static int32_t run_step(cmld_engine *e, const StepOpts &o) {
-  if ((e->cfg.flags & CMLD_FLAG_NO_GRAPH) || e->graphs_off || o.tree_mask) return engine_step(e, o);
+int32_t run_step(cmld_engine *e, const StepOpts &o) {
+  // (a layered design's portion of one sequence has launch shapes that depend on its place: no graph)
+  if ((e->cfg.flags & CMLD_FLAG_NO_GRAPH) || e->graphs_off || o.tree_mask || (e->lay && o.shared_slots)) return engine_step(e, o);
   uint32_t bits = (o.from_tokens ? 1u : 0u) | (o.rope_by_position ? 2u : 0u) | (o.logits ? 4u : 0u) | (o.argmax ? 8u : 0u) |
                   (o.feed_back ? 16u : 0u) | (o.taps ? 32u : 0u) | (o.shared_slots ? 64u : 0u) | (o.attn_cluster ? 128u : 0u) | ((uint32_t)(o.layer_begin & 0xfff) << 8) | ((uint32_t)((o.layer_end + 1) & 0xfff) << 20);
   uint32_t scale_bits;
   memcpy(&scale_bits, &o.scale, 4);
-  auto &g = e->graphs[std::make_tuple(o.batch | (o.attn_cap << 8), bits, scale_bits)];
+  auto &g = e->graphs[std::make_tuple((int64_t)o.batch | ((int64_t)o.attn_cap << 32), bits, scale_bits)];
   if (g.exec) {
     CMLD_CUDA(cudaGraphLaunch(g.exec, e->stream));
     e->launches += g.launches;
@@ -1115,6 +992,7 @@ static int32_t run_step(cmld_engine *e, const StepOpts &o) {
 }
 
 static int32_t require_weights(const cmld_engine *e, bool need_output) {
+  if (e->lay) return layered_ready(e, true) ? CMLD_OK : CMLD_ERR_STATE;
   for (size_t i = 0; i < e->layers.size(); ++i) {
     const LayerW &L = e->layers[i];
     if (!L.dense_set) return fail(CMLD_ERR_STATE, "layer %zu has no weights", i);
@@ -1132,14 +1010,14 @@ static bool use_attn_cluster(int32_t rows, int64_t max_position) { return rows <
 
 // Bound on the context length handed to the reference-order attention kernel: the smallest of a few buckets
 // that holds every row's context (a step graph is kept per bucket), 0 beyond the largest.
-static int32_t attn_cap_for(int64_t max_position) {
+int32_t attn_cap_for(int64_t max_position) {
   for (int32_t cap : {1024, 2048, 4096, 8192})
     if (max_position < cap) return cap;
   return 0;
 }
 
 // Rows of one step: tokens (or none), positions and KV slots to the device.
-static int32_t stage_rows(cmld_engine *e, int32_t n, const int32_t *tokens, const int32_t *positions, const int32_t *slots) {
+int32_t stage_rows(cmld_engine *e, int32_t n, const int32_t *tokens, const int32_t *positions, const int32_t *slots) {
   if (tokens) CMLD_CUDA(cudaMemcpyAsync(e->d_tokens, tokens, (size_t)n * 4, cudaMemcpyHostToDevice, e->stream));
   CMLD_CUDA(cudaMemcpyAsync(e->d_positions, positions, (size_t)n * 4, cudaMemcpyHostToDevice, e->stream));
   CMLD_CUDA(cudaMemcpyAsync(e->d_slots, slots, (size_t)n * 4, cudaMemcpyHostToDevice, e->stream));
@@ -1166,7 +1044,7 @@ static int32_t settle(cmld_engine *e) {
   }, e);
 }
 
-static int32_t finish(cmld_engine *e, const char *what) {
+int32_t finish(cmld_engine *e, const char *what) {
   CMLD_TRY(settle(e));
   int32_t st = 0;
   cudaError_t ce = cudaMemcpyAsync(&st, e->d_status, 4, cudaMemcpyDeviceToHost, e->stream);
@@ -1179,11 +1057,27 @@ static int32_t finish(cmld_engine *e, const char *what) {
   return CMLD_OK;
 }
 
+// Calls that speak of llama-shaped layers (embedding rows, K/V rows, projections by name).
+static int32_t llama_only(const cmld_engine *e) {
+  if (e->lay) return fail(CMLD_ERR_UNSUPPORTED, "this engine runs a layered design: only the token-driven calls apply");
+  return CMLD_OK;
+}
+
+// The attention kernels' bound on the context, as a bucket (a step graph is kept per bucket).  The layered designs'
+// kernels take any length: powers of two.
+static int32_t context_bucket(const cmld_engine *e, int64_t max_position) {
+  if (!e->lay) return attn_cap_for(max_position);
+  int64_t cap = 512;
+  while (cap <= max_position) cap *= 2;
+  return (int32_t)cap;
+}
+
 // One sequence-0 row fed by an embedding vector: the forward_token family.
 static int32_t forward_embedding_rows(cmld_engine *e, const float *embeddings, const float *cosv, const float *sinv,
                                       int64_t position0, int32_t n_rows, float scale, bool logits, bool argmax, bool taps,
                                       int32_t layer_begin = 0, int32_t layer_end = -1) {
   const cmld_config &c = e->cfg;
+  CMLD_TRY(llama_only(e));
   if (!embeddings || !cosv || !sinv) return fail(CMLD_ERR_INVALID, "embedding / cos / sin pointer is null");
   if (position0 < 0 || position0 + n_rows > c.max_pos)
     return fail(CMLD_ERR_STATE, "positions %lld..%lld exceed max_pos %d", (long long)position0,
@@ -1433,6 +1327,7 @@ int32_t cmld_engine_comm_init(cmld_engine *e, const uint8_t id[128], int32_t ran
 int32_t cmld_engine_set_layer(cmld_engine *e, int32_t layer, const cmld_tensor projs[7], const float *attn_norm,
                               const float *ffn_norm) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   const cmld_config &c = e->cfg;
   if (layer < 0 || layer >= c.n_layers) return fail(CMLD_ERR_INVALID, "set_layer: layer %d out of range", layer);
@@ -1459,6 +1354,7 @@ int32_t cmld_engine_set_layer(cmld_engine *e, int32_t layer, const cmld_tensor p
 int32_t cmld_engine_set_layer_moe(cmld_engine *e, int32_t layer, const float *router, const cmld_tensor *gate_exps,
                                   const cmld_tensor *up_exps, const cmld_tensor *down_exps) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   const cmld_config &c = e->cfg;
   if (c.n_experts <= 0) return fail(CMLD_ERR_STATE, "set_layer_moe: engine was created without experts");
@@ -1482,6 +1378,7 @@ int32_t cmld_engine_set_layer_moe(cmld_engine *e, int32_t layer, const float *ro
 
 int32_t cmld_engine_set_output(cmld_engine *e, const float *final_norm, const cmld_tensor *output) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   if (!output) return fail(CMLD_ERR_INVALID, "set_output: tensor is null");
   CMLD_TRY(weight_upload(e->output, output->qtype, e->vocab_local, e->cfg.hidden, output->data, output->nbytes, e->stream));
@@ -1493,6 +1390,7 @@ int32_t cmld_engine_set_output(cmld_engine *e, const float *final_norm, const cm
 
 int32_t cmld_engine_set_token_embd(cmld_engine *e, const cmld_tensor *t) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   if (!t) return fail(CMLD_ERR_INVALID, "set_token_embd: tensor is null");
   CMLD_TRY(weight_upload(e->token_embd, t->qtype, e->cfg.vocab, e->cfg.hidden, t->data, t->nbytes, e->stream));
@@ -1528,6 +1426,7 @@ static int32_t adopt(Weight &dst, cmld_weight *src, int64_t rows, int64_t cols, 
 int32_t cmld_engine_adopt_layer(cmld_engine *e, int32_t layer, cmld_weight *const projs[7], const float *attn_norm,
                                 const float *ffn_norm) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   const cmld_config &c = e->cfg;
   if (layer < 0 || layer >= c.n_layers) return fail(CMLD_ERR_INVALID, "adopt_layer: layer %d out of range", layer);
@@ -1549,6 +1448,7 @@ int32_t cmld_engine_adopt_layer(cmld_engine *e, int32_t layer, cmld_weight *cons
 int32_t cmld_engine_adopt_layer_moe(cmld_engine *e, int32_t layer, cmld_weight *router_f32, cmld_weight *gate_exps,
                                     cmld_weight *up_exps, cmld_weight *down_exps) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   const cmld_config &c = e->cfg;
   if (c.n_experts <= 0) return fail(CMLD_ERR_STATE, "adopt_layer_moe: engine was created without experts");
@@ -1575,6 +1475,7 @@ int32_t cmld_engine_adopt_layer_moe(cmld_engine *e, int32_t layer, cmld_weight *
 
 int32_t cmld_engine_adopt_output(cmld_engine *e, const float *final_norm, cmld_weight *output) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   if (!output) return fail(CMLD_ERR_INVALID, "adopt_output: weight is null");
   CMLD_TRY(adopt(e->output, output, e->vocab_local, e->cfg.hidden, "adopt_output"));
@@ -1585,6 +1486,7 @@ int32_t cmld_engine_adopt_output(cmld_engine *e, const float *final_norm, cmld_w
 
 int32_t cmld_engine_adopt_token_embd(cmld_engine *e, cmld_weight *token_embd) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   drop_graphs(e);
   if (!token_embd) return fail(CMLD_ERR_INVALID, "adopt_token_embd: weight is null");
   CMLD_TRY(adopt(e->token_embd, token_embd, e->cfg.vocab, e->cfg.hidden, "adopt_token_embd", true));
@@ -1594,6 +1496,7 @@ int32_t cmld_engine_adopt_token_embd(cmld_engine *e, cmld_weight *token_embd) {
 
 int32_t cmld_engine_weights_ready(const cmld_engine *e) {
   if (!e) return 0;
+  if (e->lay) return layered_ready(e, false);
   for (const auto &L : e->layers)
     if (!L.dense_set || (e->cfg.n_experts > 0 && !L.moe_set)) return 0;
   return e->has_output ? 1 : 0;
@@ -1746,6 +1649,7 @@ int32_t cmld_engine_verify_tree(cmld_engine *e, const float *embeddings, const f
                                 const int32_t *node_kvslot, const uint32_t *ancestor_bits, int32_t words, int64_t base_position,
                                 int32_t n, float scale, uint32_t *tokens_out) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   const cmld_config &c = e->cfg;
   if (n < 1 || n > CMLD_TREE_MAX_NODES) return fail(CMLD_ERR_INVALID, "verify_tree: n=%d out of 1..=%d", n, CMLD_TREE_MAX_NODES);
   if (!embeddings || !cos_all || !sin_all || !node_kvslot || !ancestor_bits || !tokens_out) return fail(CMLD_ERR_INVALID, "verify_tree: null argument");
@@ -1804,6 +1708,7 @@ __global__ void kv_compact_kernel(__half *kc, __half *vc, int64_t layer_elems, i
 // to the contiguous rows base + r (front to back; path[r] >= r, so a source is never overwritten before it is read).
 int32_t cmld_engine_compact_tree_kv_path(cmld_engine *e, const int32_t *path, int32_t len, int64_t base_position) {
   CMLD_ENGINE_ENTER(e);
+  CMLD_TRY(llama_only(e));
   const cmld_config &c = e->cfg;
   if (!path || len < 0 || len > CMLD_TREE_MAX_NODES) return fail(CMLD_ERR_INVALID, "compact_tree_kv_path: bad path");
   if (e->kq8) return fail(CMLD_ERR_UNSUPPORTED, "compact_tree_kv_path: not supported over a Q8_0 KV cache");
@@ -1834,6 +1739,7 @@ __global__ void kv_convert_kernel(__half *cache, float *host_layout, int n_kv, i
 
 static int32_t kv_transfer(cmld_engine *e, int32_t layer, float *ck, float *cv, int64_t n_pos, bool to_cache) {
   const cmld_config &c = e->cfg;
+  CMLD_TRY(llama_only(e));
   if (layer < 0 || layer >= c.n_layers) return fail(CMLD_ERR_INVALID, "layer %d out of range", layer);
   if (n_pos < 0 || n_pos > c.max_pos) return fail(CMLD_ERR_INVALID, "n_positions %lld out of range", (long long)n_pos);
   if (n_pos == 0) return CMLD_OK;
@@ -1910,6 +1816,8 @@ int32_t cmld_engine_step_batch(cmld_engine *e, int32_t n_seqs, const int32_t *se
   std::vector<int32_t> pos32;
   CMLD_TRY(check_rows(e, n_seqs, seqs, tokens_in, positions, 1, pos32));
   CMLD_TRY(require_weights(e, true));
+  if (e->lay && hidden_out) CMLD_TRY(llama_only(e));
+  if (e->lay) CMLD_TRY(layered_claim(e, n_seqs, seqs, positions));
   CMLD_TRY(stage_rows(e, n_seqs, tokens_in, pos32.data(), seqs));
   e->launches = 0;
   CMLD_CUDA(cudaEventRecord(e->ev0, e->stream));
@@ -1922,7 +1830,7 @@ int32_t cmld_engine_step_batch(cmld_engine *e, int32_t n_seqs, const int32_t *se
     int64_t mx = 0;
     for (int i = 0; i < n_seqs; ++i) mx = std::max<int64_t>(mx, positions[i]);
     o.attn_cluster = use_attn_cluster(n_seqs, mx);
-    o.attn_cap = attn_cap_for(mx);
+    o.attn_cap = context_bucket(e, mx);
   }
   CMLD_TRY(run_step(e, o));
   CMLD_CUDA(cudaEventRecord(e->ev1, e->stream));
@@ -1933,6 +1841,8 @@ int32_t cmld_engine_step_batch(cmld_engine *e, int32_t n_seqs, const int32_t *se
   if (logits_out) CMLD_CUDA(cudaMemcpyAsync(logits_out, e->tp > 1 ? e->logits_full : e->logits, (size_t)n_seqs * e->cfg.vocab * 4, cudaMemcpyDeviceToHost, e->stream));
   if (hidden_out) CMLD_CUDA(cudaMemcpyAsync(hidden_out, e->h, (size_t)n_seqs * e->cfg.hidden * 4, cudaMemcpyDeviceToHost, e->stream));
   CMLD_TRY(finish(e, "step_batch"));
+  if (e->lay) layered_advance(e, n_seqs, seqs, positions, 1);
+  e->last_logit_row = n_seqs - 1;
   cudaEventElapsedTime(&e->last_ms, e->ev0, e->ev1);
   e->last_launches = e->launches;
   if (tokens_out)
@@ -1940,15 +1850,11 @@ int32_t cmld_engine_step_batch(cmld_engine *e, int32_t n_seqs, const int32_t *se
   return CMLD_OK;
 }
 
-int32_t cmld_engine_prefill_tokens(cmld_engine *e, int32_t seq, const int32_t *tokens, int64_t n, int64_t start_pos,
-                                   uint32_t *next_token_out) {
-  CMLD_ENGINE_ENTER(e);
-  if (n < 1 || !tokens) return fail(CMLD_ERR_INVALID, "prefill_tokens: no tokens");
-  CMLD_TRY(require_weights(e, true));
+// Tokens of one sequence through the llama-shaped engine, a chunk of rows at a time.
+static int32_t llama_extend(cmld_engine *e, int32_t seq, const int32_t *tokens, int64_t n, int64_t start_pos, const int32_t *want, int32_t n_want,
+                            float *logits_out) {
   const int chunk = (n > 8 && !(e->cfg.flags & CMLD_FLAG_EXACT_ORDER)) ? 32 : 8;
-  e->launches = 0;
-  CMLD_CUDA(cudaEventRecord(e->ev0, e->stream));
-  int last_rows = 0;
+  int32_t w = 0;
   for (int64_t i = 0; i < n; i += chunk) {
     const int rows = (int)std::min<int64_t>(chunk, n - i);
     std::vector<int32_t> seqs(rows, seq), pos32;
@@ -1956,26 +1862,76 @@ int32_t cmld_engine_prefill_tokens(cmld_engine *e, int32_t seq, const int32_t *t
     for (int r = 0; r < rows; ++r) pos[r] = start_pos + i + r;
     CMLD_TRY(check_rows(e, rows, seqs.data(), tokens + i, pos.data(), 1, pos32));
     CMLD_TRY(stage_rows(e, rows, tokens + i, pos32.data(), seqs.data()));
+    const bool wanted = w < n_want && want[w] < i + rows;
     StepOpts o;
     o.batch = rows;
     o.shared_slots = rows > 1;
     o.from_tokens = true;
     o.scale = 1.0f / sqrtf((float)e->cfg.head_dim);
-    o.logits = o.argmax = (i + chunk >= n);
+    o.logits = o.argmax = (i + chunk >= n) || wanted;
     o.attn_cluster = use_attn_cluster(rows, start_pos + i + rows - 1);
     o.attn_cap = attn_cap_for(start_pos + i + rows - 1);
     CMLD_TRY(run_step(e, o));
-    last_rows = rows;
+    if (wanted) {
+      if (e->tp > 1) CMLD_TRY(gather_logits(e, rows));
+      CMLD_TRY(settle(e));
+      const float *src = e->tp > 1 ? e->logits_full : e->logits;
+      for (; w < n_want && want[w] < i + rows; ++w)
+        CMLD_CUDA(cudaMemcpyAsync(logits_out + (int64_t)w * e->cfg.vocab, src + (want[w] - i) * e->cfg.vocab, (size_t)e->cfg.vocab * 4,
+                                  cudaMemcpyDeviceToHost, e->stream));
+    }
+    e->last_logit_row = rows - 1;
   }
+  return CMLD_OK;
+}
+
+int32_t cmld_engine_extend(cmld_engine *e, int32_t seq, const int32_t *tokens, int64_t n, int64_t start_pos, const int32_t *want, int32_t n_want,
+                           float *logits_out, float *taps_out, uint32_t *next_token_out) {
+  CMLD_ENGINE_ENTER(e);
+  if (n < 1 || !tokens) return fail(CMLD_ERR_INVALID, "extend: no tokens");
+  if (n_want < 0 || (n_want > 0 && (!want || !logits_out))) return fail(CMLD_ERR_INVALID, "extend: places or logits pointer is null");
+  for (int32_t i = 0; i < n_want; ++i)
+    if (want[i] < 0 || want[i] >= n || (i > 0 && want[i] <= want[i - 1])) return fail(CMLD_ERR_INVALID, "extend: places must rise and lie within the tokens");
+  if (taps_out && !e->lay) return fail(CMLD_ERR_UNSUPPORTED, "extend: the residual stream after every layer is offered for layered designs only");
+  CMLD_TRY(require_weights(e, true));
+  e->launches = 0;
+  CMLD_CUDA(cudaEventRecord(e->ev0, e->stream));
+  CMLD_TRY(e->lay ? layered_extend(e, seq, tokens, n, start_pos, want, n_want, logits_out, taps_out)
+                  : llama_extend(e, seq, tokens, n, start_pos, want, n_want, logits_out));
   CMLD_CUDA(cudaEventRecord(e->ev1, e->stream));
   int32_t tok = 0;
   CMLD_TRY(settle(e));
-  CMLD_CUDA(cudaMemcpyAsync(&tok, e->out_idx + (last_rows - 1), 4, cudaMemcpyDeviceToHost, e->stream));
-  CMLD_TRY(finish(e, "prefill_tokens"));
+  CMLD_CUDA(cudaMemcpyAsync(&tok, e->out_idx + e->last_logit_row, 4, cudaMemcpyDeviceToHost, e->stream));
+  CMLD_TRY(finish(e, "extend"));
+  if (e->lay) {
+    const int64_t at = start_pos;
+    layered_advance(e, 1, &seq, &at, n);
+  }
   cudaEventElapsedTime(&e->last_ms, e->ev0, e->ev1);
   e->last_launches = e->launches;
   if (next_token_out) *next_token_out = (uint32_t)tok;
   return CMLD_OK;
+}
+
+int32_t cmld_engine_prefill_tokens(cmld_engine *e, int32_t seq, const int32_t *tokens, int64_t n, int64_t start_pos,
+                                   uint32_t *next_token_out) {
+  return cmld_engine_extend(e, seq, tokens, n, start_pos, nullptr, 0, nullptr, nullptr, next_token_out);
+}
+
+int32_t cmld_engine_sample_row(cmld_engine *e, int32_t row, float temperature, float min_p, uint64_t seed, uint32_t *token_out) {
+  CMLD_ENGINE_ENTER(e);
+  if (!token_out) return fail(CMLD_ERR_INVALID, "token_out is null");
+  if (!(temperature > 0.0f) || !std::isfinite(temperature)) return fail(CMLD_ERR_INVALID, "temperature must be a finite positive number");
+  if (min_p > 0.0f && !(min_p <= 1.0f)) return fail(CMLD_ERR_INVALID, "min_p must lie in (0, 1]");
+  if (e->tp > 1) return fail(CMLD_ERR_UNSUPPORTED, "sampling on a tensor-parallel engine is not supported");
+  if (row < 0) row = e->last_logit_row;
+  if (row >= e->logit_rows) return fail(CMLD_ERR_INVALID, "row %d out of range", row);
+  const float *logits = e->logits + (int64_t)row * e->cfg.vocab;
+  uint32_t *d_tok = reinterpret_cast<uint32_t *>(e->out_idx + row);
+  if (min_p > 0.0f) CMLD_TRY(launch_sample_gumbel_filtered(logits, e->cfg.vocab, temperature, min_p, seed, d_tok, e->stream));
+  else CMLD_TRY(launch_sample_gumbel(logits, e->cfg.vocab, 1.0f / temperature, seed, d_tok, e->stream));
+  CMLD_CUDA(cudaMemcpyAsync(token_out, d_tok, 4, cudaMemcpyDeviceToHost, e->stream));
+  return finish(e, "sample_row");
 }
 
 int32_t cmld_engine_decode_greedy(cmld_engine *e, int32_t n_seqs, const int32_t *seqs, const int32_t *tokens_in,
@@ -1986,8 +1942,9 @@ int32_t cmld_engine_decode_greedy(cmld_engine *e, int32_t n_seqs, const int32_t 
   std::vector<int32_t> pos32;
   CMLD_TRY(check_rows(e, n_seqs, seqs, tokens_in, positions, n_steps, pos32));
   CMLD_TRY(require_weights(e, true));
+  if (e->lay) CMLD_TRY(layered_claim(e, n_seqs, seqs, positions));
   CMLD_TRY(stage_rows(e, n_seqs, tokens_in, pos32.data(), seqs));
-  CMLD_CUDA(cudaMemsetAsync(e->am_ticket, 0, (size_t)2 * e->max_rows * 4, e->stream));
+  CMLD_CUDA(cudaMemsetAsync(e->am_ticket, 0, (size_t)2 * e->logit_rows * 4, e->stream));
   e->launches = 0;
   CMLD_CUDA(cudaEventRecord(e->ev0, e->stream));
   StepOpts o;
@@ -2000,7 +1957,7 @@ int32_t cmld_engine_decode_greedy(cmld_engine *e, int32_t n_seqs, const int32_t 
   for (int i = 0; i < n_seqs; ++i) max_start = std::max<int64_t>(max_start, positions[i]);
   for (int s = 0; s < n_steps; ++s) {
     o.attn_cluster = use_attn_cluster(n_seqs, max_start + s);
-    o.attn_cap = attn_cap_for(max_start + s);
+    o.attn_cap = context_bucket(e, max_start + s);
     CMLD_TRY(run_step(e, o));
   }
   CMLD_CUDA(cudaEventRecord(e->ev1, e->stream));
@@ -2008,6 +1965,8 @@ int32_t cmld_engine_decode_greedy(cmld_engine *e, int32_t n_seqs, const int32_t 
   CMLD_TRY(settle(e));
   CMLD_CUDA(cudaMemcpyAsync(hist.data(), e->d_history, hist.size() * 4, cudaMemcpyDeviceToHost, e->stream));
   CMLD_TRY(finish(e, "decode_greedy"));
+  if (e->lay) layered_advance(e, n_seqs, seqs, positions, n_steps);
+  e->last_logit_row = n_seqs - 1;
   cudaEventElapsedTime(&e->last_ms, e->ev0, e->ev1);
   e->last_launches = e->launches;
   for (size_t i = 0; i < hist.size(); ++i) tokens_out[i] = (uint32_t)hist[i];

@@ -1,0 +1,509 @@
+// Multi-head attention over latents: a position's cache row is one latent vector c (rank values) and one rotated key
+// part shared by all heads (rot_dim values); per head the unrotated key is W_uk c and the value W_uv c.
+//
+// Decoding and short portions work in latent space: the query is taken through W_uk^T once (q_nope . W_uk c =
+// (W_uk^T q_nope) . c), the cache rows are scored and averaged as they are, and W_uv is applied to the average.
+//   latent_prep_kernel    rotates and transforms the queries; norms, rotates and appends the new cache rows
+//   latent_attn_kernel    a range of positions for eight heads of one row: online softmax, all in 32-bit
+//   latent_output_kernel  merges the ranges, applies W_uv and the sigmoid gate
+// Long portions expand keys and values with two matrix products and run a tiled attention on the tensor cores:
+//   latent_prefill_kernel 64 queries of one head per CTA, 64 keys at a time; scores, weights and sums in 32-bit (the
+//                         weights enter the second product as two bfloat16 terms)
+#include "layered.cuh"
+#include "mma_sync.cuh"
+
+namespace cmld {
+
+namespace {
+
+// ---------------------------------------------------------------- queries into latent space, cache append
+
+constexpr int kPrepThreads = 256, kPrepRanks = 128, kPrepRows = 2;
+
+// The value at index j of a rotated vector whose pairs (2i, 2i + 1), i < dims / 2, turn by the angles behind cs.
+__device__ __forceinline__ float rotated(const float *x, int j, int dims, const float *cs) {
+  if (j >= dims) return x[j];
+  const float c = cs[(j >> 1) * 2], s = cs[(j >> 1) * 2 + 1];
+  const float u = x[j & ~1], v = x[j | 1];
+  return (j & 1) ? v * c + u * s : u * c - v * s;
+}
+
+// grid: x = row groups (appending CTAs: rows), y = head * slices + slice of the latent; the last y appends.
+__global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentArgs a, int slices, int query_ys) {
+  __shared__ float red[kPrepThreads / 32];
+  __shared__ float part[kPrepThreads / 64][kPrepRows][kPrepRanks];
+  extern __shared__ float qn[];  // [kPrepRows][dim]
+  pdl_launch();
+  pdl_wait();
+  const LatentShape &m = a.m;
+  const int tid = threadIdx.x;
+  if ((int)blockIdx.y == query_ys) {
+    // new cache rows
+    for (int r = blockIdx.x; r < a.rows; r += gridDim.x) {
+      const float *low = a.low + (int64_t)r * a.low_ld;
+      const int64_t pos = a.positions[r];
+      const int64_t at = ((int64_t)a.slots[r] * a.max_pos + pos) * a.cache_ld;
+      float s = 0.0f;
+      for (int i = tid; i < m.rank; i += kPrepThreads) s = fmaf(low[i], low[i], s);
+      const float inv = 1.0f / sqrtf(cta_total(s, red) / (float)m.rank + m.eps);
+      for (int i = tid; i < m.rank; i += kPrepThreads) act_store(a.cache, a.cache_half, at + i, low[i] * inv * a.latent_norm[i]);
+      for (int i = tid; i < m.rot_dim; i += kPrepThreads)
+        act_store(a.cache, a.cache_half, at + m.rank + i, rotated(low + m.rank, i, m.rot_dims, a.cs + pos * m.rot_dims));
+    }
+    return;
+  }
+  const int h = blockIdx.y / slices, sl = blockIdx.y % slices, qd = m.dim + m.rot_dim, D = m.rank + m.rot_dim;
+  const int n_groups = (a.rows + kPrepRows - 1) / kPrepRows;
+  for (int g = blockIdx.x; g < n_groups; g += gridDim.x) {
+    const int r0 = g * kPrepRows, nr = min(kPrepRows, a.rows - r0);
+    __syncthreads();
+    for (int i = tid; i < kPrepRows * m.dim; i += kPrepThreads) {
+      const int r = i / m.dim, d = i % m.dim;
+      qn[i] = r < nr ? a.q[((int64_t)(r0 + r) * m.heads + h) * qd + d] : 0.0f;
+    }
+    __syncthreads();
+    // 64 pairs of latent dimensions x 4 shares of the head's dimensions
+    const int pr = tid & 63, sh = tid >> 6, r = sl * kPrepRanks + 2 * pr;
+    float acc[kPrepRows][2] = {};
+    if (r < m.rank) {
+      const bf16 *w = a.uk.w + (int64_t)h * m.dim * a.uk.ld + r;  // rows are zero-padded to a multiple of 8
+#pragma unroll 8
+      for (int d = sh; d < m.dim; d += 4) {
+        const uint32_t v = *reinterpret_cast<const uint32_t *>(w + (int64_t)d * a.uk.ld);
+#pragma unroll
+        for (int i = 0; i < kPrepRows; ++i) {
+          const float qv = qn[i * m.dim + d];
+          acc[i][0] = fmaf(bf16_lo(v), qv, acc[i][0]);
+          acc[i][1] = fmaf(bf16_hi(v), qv, acc[i][1]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kPrepRows; ++i) {
+      part[sh][i][2 * pr] = acc[i][0];
+      part[sh][i][2 * pr + 1] = acc[i][1];
+    }
+    __syncthreads();
+    for (int i = tid; i < kPrepRows * kPrepRanks; i += kPrepThreads) {
+      const int rr = i / kPrepRanks, c = i % kPrepRanks;
+      if (rr < nr && sl * kPrepRanks + c < m.rank)
+        a.qa[((int64_t)(r0 + rr) * m.heads + h) * D + sl * kPrepRanks + c] =
+            m.scale * (part[0][rr][c] + part[1][rr][c] + part[2][rr][c] + part[3][rr][c]);
+    }
+    if (sl == 0)
+      for (int i = tid; i < nr * m.rot_dim; i += kPrepThreads) {
+        const int rr = i / m.rot_dim, j = i % m.rot_dim;
+        const float *x = a.q + ((int64_t)(r0 + rr) * m.heads + h) * qd + m.dim;
+        a.qa[((int64_t)(r0 + rr) * m.heads + h) * D + m.rank + j] =
+            m.scale * rotated(x, j, m.rot_dims, a.cs + (int64_t)a.positions[r0 + rr] * m.rot_dims);
+      }
+  }
+}
+
+// ---------------------------------------------------------------- attention in latent space
+
+constexpr int kAttThreads = 256, kAttHeads = 8, kAttKeys = 32;
+
+__host__ __device__ inline int att_units(int D) {  // 16-byte units of a staged row: an odd count keeps lanes apart
+  const int u = (D + 3) / 4;
+  return u | 1;
+}
+__host__ __device__ inline int att_smem(int D) {
+  return (kAttKeys + kAttHeads) * att_units(D) * 16 + (8 * kAttHeads * kAttKeys + kAttKeys * kAttHeads + kAttHeads) * 4;
+}
+
+// NR: pairs of latent dimensions per thread (rank <= 512 * NR)
+template <int NR>
+__global__ void __launch_bounds__(kAttThreads) latent_attn_kernel(const LatentArgs a) {
+  extern __shared__ __align__(16) float sm[];
+  pdl_launch();
+  pdl_wait();
+  const LatentShape &m = a.m;
+  const int D = m.rank + m.rot_dim, U = att_units(D), ld = U * 4, used = (D + 3) / 4;
+  float *ks = sm, *qs = ks + kAttKeys * ld, *sc = qs + kAttHeads * ld, *pr = sc + 8 * kAttHeads * kAttKeys, *corr = pr + kAttKeys * kAttHeads;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int split = blockIdx.x, h0 = blockIdx.y * kAttHeads, row = blockIdx.z, nh = min(kAttHeads, m.heads - h0);
+  const int n = a.positions[row] + 1;
+  const int tiles = (n + kAttKeys - 1) / kAttKeys, per = (tiles + a.splits - 1) / a.splits;
+  const int lo = min(split * per, tiles) * kAttKeys, hi = min(min((split + 1) * per, tiles) * kAttKeys, n);
+  const int64_t cache0 = (int64_t)a.slots[row] * a.max_pos * a.cache_ld;
+  for (int i = tid; i < kAttHeads * ld; i += kAttThreads) {
+    const int h = i / ld, d = i % ld;
+    qs[i] = h < nh && d < D ? a.qa[((int64_t)row * m.heads + h0 + h) * D + d] : 0.0f;
+  }
+  float acc[kAttHeads][NR][2];
+#pragma unroll
+  for (int h = 0; h < kAttHeads; ++h)
+#pragma unroll
+    for (int j = 0; j < NR; ++j) acc[h][j][0] = acc[h][j][1] = 0.0f;
+  float mx = -INFINITY, sum = 0.0f;  // of head `warp`
+  const bool vec = a.cache_half && a.cache_ld % 8 == 0;
+  for (int k0 = lo; k0 < hi; k0 += kAttKeys) {
+    __syncthreads();
+    if (vec) {
+      const bf16 *c = static_cast<const bf16 *>(a.cache) + cache0;
+      const int u8 = (ld + 7) / 8;
+      for (int i = tid; i < kAttKeys * u8; i += kAttThreads) {
+        const int k = i / u8, d = (i % u8) * 8;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (k0 + k < hi && d < D) v = *reinterpret_cast<const uint4 *>(c + (int64_t)(k0 + k) * a.cache_ld + d);
+        const float f[8] = {bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y), bf16_lo(v.z), bf16_hi(v.z), bf16_lo(v.w), bf16_hi(v.w)};
+        float *o = ks + k * ld + d;
+#pragma unroll
+        for (int q = 0; q < 2; ++q)
+          if (d + 4 * q < ld) {
+            float4 w;
+            w.x = d + 4 * q + 0 < D ? f[4 * q + 0] : 0.0f;
+            w.y = d + 4 * q + 1 < D ? f[4 * q + 1] : 0.0f;
+            w.z = d + 4 * q + 2 < D ? f[4 * q + 2] : 0.0f;
+            w.w = d + 4 * q + 3 < D ? f[4 * q + 3] : 0.0f;
+            *reinterpret_cast<float4 *>(o + 4 * q) = w;
+          }
+      }
+    } else {
+      for (int i = tid; i < kAttKeys * ld; i += kAttThreads) {
+        const int k = i / ld, d = i % ld;
+        ks[i] = k0 + k < hi && d < D ? act_load(a.cache, a.cache_half, cache0 + (int64_t)(k0 + k) * a.cache_ld + d) : 0.0f;
+      }
+    }
+    __syncthreads();
+    // scores: lane = key, a warp takes every eighth 16-byte unit of the dimensions for all heads
+    float s[kAttHeads];
+#pragma unroll
+    for (int h = 0; h < kAttHeads; ++h) s[h] = 0.0f;
+    for (int u = warp; u < used; u += 8) {
+      const float4 k = *reinterpret_cast<const float4 *>(ks + lane * ld + u * 4);
+#pragma unroll
+      for (int h = 0; h < kAttHeads; ++h) {
+        const float4 q = *reinterpret_cast<const float4 *>(qs + h * ld + u * 4);
+        s[h] = fmaf(k.x, q.x, fmaf(k.y, q.y, fmaf(k.z, q.z, fmaf(k.w, q.w, s[h]))));
+      }
+    }
+#pragma unroll
+    for (int h = 0; h < kAttHeads; ++h) sc[(warp * kAttHeads + h) * kAttKeys + lane] = s[h];
+    __syncthreads();
+    {
+      float v = 0.0f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) v += sc[(w * kAttHeads + warp) * kAttKeys + lane];
+      if (k0 + lane >= hi) v = -INFINITY;
+      const float nm = fmaxf(mx, warp_max(v)), c = expf(mx - nm), p = expf(v - nm);
+      sum = fmaf(sum, c, warp_sum(p));
+      mx = nm;
+      pr[lane * kAttHeads + warp] = p;
+      if (lane == 0) corr[warp] = c;
+    }
+    __syncthreads();
+    {
+      float c[kAttHeads];
+#pragma unroll
+      for (int h = 0; h < kAttHeads; ++h) c[h] = corr[h];
+#pragma unroll
+      for (int j = 0; j < NR; ++j)
+#pragma unroll
+        for (int h = 0; h < kAttHeads; ++h) {
+          acc[h][j][0] *= c[h];
+          acc[h][j][1] *= c[h];
+        }
+    }
+    const int nk = min(kAttKeys, hi - k0);
+    if (2 * tid < m.rank) {
+#pragma unroll 4
+      for (int k = 0; k < nk; ++k) {
+        const float4 p0 = *reinterpret_cast<const float4 *>(pr + k * kAttHeads), p1 = *reinterpret_cast<const float4 *>(pr + k * kAttHeads + 4);
+        const float p[8] = {p0.x, p0.y, p0.z, p0.w, p1.x, p1.y, p1.z, p1.w};
+#pragma unroll
+        for (int j = 0; j < NR; ++j) {
+          const int d = 2 * tid + 512 * j;
+          if (NR > 1 && d >= m.rank) break;
+          const float2 v = *reinterpret_cast<const float2 *>(ks + k * ld + d);
+#pragma unroll
+          for (int h = 0; h < kAttHeads; ++h) {
+            acc[h][j][0] = fmaf(p[h], v.x, acc[h][j][0]);
+            acc[h][j][1] = fmaf(p[h], v.y, acc[h][j][1]);
+          }
+        }
+      }
+    }
+  }
+  // partials: maximum, sum, weighted latents
+  const int64_t ps = m.rank + 2;
+  float *out = a.part + (((int64_t)row * m.heads + h0) * a.splits + split) * ps;
+  if (warp < nh && lane == 0) {
+    out[(int64_t)warp * a.splits * ps] = mx;
+    out[(int64_t)warp * a.splits * ps + 1] = sum;
+  }
+#pragma unroll
+  for (int h = 0; h < kAttHeads; ++h)
+    if (h < nh)
+#pragma unroll
+      for (int j = 0; j < NR; ++j) {
+        const int d = 2 * tid + 512 * j;
+        float *o = out + (int64_t)h * a.splits * ps + 2;
+        if (d < m.rank) o[d] = acc[h][j][0];
+        if (d + 1 < m.rank) o[d + 1] = acc[h][j][1];
+      }
+}
+
+// ---------------------------------------------------------------- merge, W_uv, gate
+
+constexpr int kOutThreads = 256, kOutCols = 32;
+
+__global__ void __launch_bounds__(kOutThreads) latent_output_kernel(const LatentArgs a) {
+  extern __shared__ __align__(16) float ctx[];  // [ld of W_uv]
+  __shared__ float wgt[64];
+  pdl_launch();
+  pdl_wait();
+  const LatentShape &m = a.m;
+  const int row = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * kOutCols, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int64_t ps = m.rank + 2;
+  const float *part = a.part + ((int64_t)row * m.heads + h) * a.splits * ps;
+  if (warp == 0) {
+    float m0 = lane < a.splits ? part[lane * ps] : -INFINITY, m1 = lane + 32 < a.splits ? part[(lane + 32) * ps] : -INFINITY;
+    const float mx = warp_max(fmaxf(m0, m1));
+    const float e0 = lane < a.splits ? expf(m0 - mx) : 0.0f, e1 = lane + 32 < a.splits ? expf(m1 - mx) : 0.0f;
+    const float l = warp_sum((lane < a.splits ? e0 * part[lane * ps + 1] : 0.0f) + (lane + 32 < a.splits ? e1 * part[(lane + 32) * ps + 1] : 0.0f));
+    wgt[lane] = e0 / l;
+    wgt[lane + 32] = e1 / l;
+  }
+  __syncthreads();
+  for (int i = tid; i < (int)a.uv.ld; i += kOutThreads) {
+    float c = 0.0f;
+    if (i < m.rank)
+#pragma unroll 4
+      for (int s = 0; s < a.splits; ++s)
+        if (wgt[s] != 0.0f) c = fmaf(wgt[s], part[s * ps + 2 + i], c);  // an empty range has weight 0
+    ctx[i] = c;
+  }
+  __syncthreads();
+  for (int v = v0 + warp; v < min(v0 + kOutCols, m.vdim); v += kOutThreads / 32) {
+    const bf16 *w = a.uv.w + ((int64_t)h * m.vdim + v) * a.uv.ld;
+    float s = 0.0f;
+    for (int k = lane * 8; k < (int)a.uv.ld; k += 256) {
+      const uint4 x = *reinterpret_cast<const uint4 *>(w + k);
+      const float4 c0 = *reinterpret_cast<const float4 *>(ctx + k), c1 = *reinterpret_cast<const float4 *>(ctx + k + 4);
+      s = fmaf(bf16_lo(x.x), c0.x, fmaf(bf16_hi(x.x), c0.y, s));
+      s = fmaf(bf16_lo(x.y), c0.z, fmaf(bf16_hi(x.y), c0.w, s));
+      s = fmaf(bf16_lo(x.z), c1.x, fmaf(bf16_hi(x.z), c1.y, s));
+      s = fmaf(bf16_lo(x.w), c1.z, fmaf(bf16_hi(x.w), c1.w, s));
+    }
+    s = warp_sum(s);
+    if (lane == 0) act_store(a.out.p, a.out.half, row * a.out.ld + h * m.vdim + v, s * sigmoid_f(a.gate[row * a.gate_ld + h * m.vdim + v]));
+  }
+}
+
+// ---------------------------------------------------------------- long portions on the tensor cores
+
+constexpr int kPfThreads = 128, kPfQ = 64, kPfK = 64;
+
+__device__ __forceinline__ void cp16(void *dst, const void *src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+
+__host__ __device__ inline int pf_qd(const LatentShape &m) { return (m.dim + m.rot_dim + 15) & ~15; }
+__host__ __device__ inline int pf_smem(int qd, int dv) { return (kPfQ * (qd + 8) + 2 * kPfK * (qd + 8) + 2 * kPfK * (dv + 8)) * 2; }
+
+// DV: value dimensions, padded to 32, 64, 128 or 256
+template <int DV>
+__global__ void __launch_bounds__(kPfThreads) latent_prefill_kernel(const LatentPrefillArgs a) {
+  extern __shared__ __align__(16) bf16 sh[];
+  const LatentShape &m = a.m;
+  const int qd = pf_qd(m), QS = qd + 8, VS = DV + 8;
+  bf16 *q_s = sh, *k_s = q_s + kPfQ * QS, *v_s = k_s + 2 * kPfK * QS;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y;
+  const int r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kPfQ;  // the longest rows first
+  const int64_t last = a.start + min(r0 + kPfQ, a.rows) - 1;      // the last position this tile's queries see
+  const int n_tiles = (int)(last / kPfK) + 1;
+  pdl_launch();
+  pdl_wait();
+  auto load_tile = [&](int t, int st) {
+    bf16 *kd = k_s + st * kPfK * QS, *vd = v_s + st * kPfK * VS;
+    const int nu = m.dim / 8, ru = m.rot_dim / 8, ku = nu + ru, vu = m.vdim / 8;
+    for (int i = tid; i < kPfK * ku; i += kPfThreads) {
+      const int k = i / ku, u = i % ku;
+      const int64_t p = (int64_t)t * kPfK + k;
+      const bool live = p <= last;
+      const int64_t pc = live ? p : 0;
+      const bf16 *src = u < nu ? a.kv + pc * a.kv_ld + h * m.dim + u * 8 : a.cache + pc * a.cache_ld + m.rank + (u - nu) * 8;
+      cp16(kd + k * QS + u * 8, src, live);
+    }
+    for (int i = tid; i < kPfK * vu; i += kPfThreads) {
+      const int k = i / vu, u = i % vu;
+      const int64_t p = (int64_t)t * kPfK + k;
+      const bool live = p <= last;
+      cp16(vd + k * VS + u * 8, a.kv + (live ? p : 0) * a.kv_ld + m.heads * m.dim + h * m.vdim + u * 8, live);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // columns no copy touches: zero once
+  for (int i = tid; i < 2 * kPfK * (qd - m.dim - m.rot_dim); i += kPfThreads) {
+    const int w = qd - m.dim - m.rot_dim;
+    k_s[(i / w) * QS + m.dim + m.rot_dim + i % w] = __float2bfloat16_rn(0.0f);
+  }
+  for (int i = tid; i < 2 * kPfK * (DV - m.vdim); i += kPfThreads) v_s[(i / (DV - m.vdim)) * VS + m.vdim + i % (DV - m.vdim)] = __float2bfloat16_rn(0.0f);
+  load_tile(0, 0);
+  const int q_ld = m.heads * (m.dim + m.rot_dim);
+  for (int i = tid; i < kPfQ * qd; i += kPfThreads) {
+    const int r = i / qd, d = i % qd;
+    float v = 0.0f;
+    if (r0 + r < a.rows && d < m.dim + m.rot_dim) {
+      const float *x = a.q + (int64_t)(r0 + r) * q_ld + h * (m.dim + m.rot_dim);
+      v = d < m.dim ? x[d] : rotated(x + m.dim, d - m.dim, m.rot_dims, a.cs + (a.start + r0 + r) * m.rot_dims);
+    }
+    q_s[r * QS + d] = __float2bfloat16_rn(v);
+  }
+  float O[DV / 8][4];
+#pragma unroll
+  for (int n = 0; n < DV / 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) O[n][e] = 0.0f;
+  float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};
+  const int tr = lane >> 2, tc = (lane & 3) * 2, i0 = warp * 16;
+  const int64_t pos0 = a.start + r0 + i0 + tr;
+  for (int t = 0; t < n_tiles; ++t) {
+    const int st = t & 1;
+    if (t + 1 < n_tiles) {
+      load_tile(t + 1, st ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const bf16 *kt = k_s + st * kPfK * QS, *vt = v_s + st * kPfK * VS;
+    float P[8][4] = {};
+#pragma unroll 2
+    for (int k = 0; k < qd; k += 16) {
+      uint32_t A[4], B[4];
+      ldsm4(A, q_s + (i0 + (lane & 15)) * QS + k + (lane >> 4) * 8);
+#pragma unroll
+      for (int n = 0; n < 4; ++n) {
+        ldsm4(B, kt + (n * 16 + (lane & 7) + ((lane >> 4) << 3)) * QS + k + ((lane >> 3) & 1) * 8);
+        mma16816(P[2 * n], A, B[0], B[1]);
+        mma16816(P[2 * n + 1], A, B[2], B[3]);
+      }
+    }
+    float nm[2] = {mx[0], mx[1]};
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int64_t key = (int64_t)t * kPfK + n * 8 + tc + (e & 1);
+        P[n][e] = key <= pos0 + (e >> 1) * 8 ? P[n][e] * m.scale : -INFINITY;
+        nm[e >> 1] = fmaxf(nm[e >> 1], P[n][e]);
+      }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      nm[e] = fmaxf(nm[e], __shfl_xor_sync(0xffffffffu, nm[e], 1));
+      nm[e] = fmaxf(nm[e], __shfl_xor_sync(0xffffffffu, nm[e], 2));
+    }
+    // key 0 is visible to every query, so nm is finite from the first tile on
+    const float c0 = expf(mx[0] - nm[0]), c1 = expf(mx[1] - nm[1]);
+    float ts[2] = {0.0f, 0.0f};
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        P[n][e] = expf(P[n][e] - nm[e >> 1]);
+        ts[e >> 1] += P[n][e];
+      }
+    sum[0] = fmaf(sum[0], c0, ts[0]);
+    sum[1] = fmaf(sum[1], c1, ts[1]);
+    mx[0] = nm[0];
+    mx[1] = nm[1];
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n) {
+      O[n][0] *= c0;
+      O[n][1] *= c0;
+      O[n][2] *= c1;
+      O[n][3] *= c1;
+    }
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) {
+      uint32_t H[4], L[4], B[4];
+      split_pair(P[2 * kk][0], P[2 * kk][1], H[0], L[0]);
+      split_pair(P[2 * kk][2], P[2 * kk][3], H[1], L[1]);
+      split_pair(P[2 * kk + 1][0], P[2 * kk + 1][1], H[2], L[2]);
+      split_pair(P[2 * kk + 1][2], P[2 * kk + 1][3], H[3], L[3]);
+#pragma unroll
+      for (int n = 0; n < DV / 16; ++n) {
+        ldsm4t(B, vt + (kk * 16 + (lane & 15)) * VS + n * 16 + (lane >> 4) * 8);
+        mma16816(O[2 * n], H, B[0], B[1]);
+        mma16816(O[2 * n + 1], H, B[2], B[3]);
+        mma16816(O[2 * n], L, B[0], B[1]);
+        mma16816(O[2 * n + 1], L, B[2], B[3]);
+      }
+    }
+    __syncthreads();  // the stage is free for the tile after next
+  }
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 1);
+    sum[e] += __shfl_xor_sync(0xffffffffu, sum[e], 2);
+  }
+#pragma unroll
+  for (int n = 0; n < DV / 8; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = r0 + i0 + tr + (e >> 1) * 8, v = n * 8 + tc + (e & 1);
+      if (r < a.rows && v < m.vdim) {
+        const float g = a.gate[(int64_t)r * a.gate_ld + h * m.vdim + v];
+        a.out[(int64_t)r * a.out_ld + h * m.vdim + v] = __float2bfloat16_rn(O[n][e] / sum[e >> 1] * sigmoid_f(g));
+      }
+    }
+}
+
+template <int DV>
+int32_t prefill(const LatentPrefillArgs &a, bool pdl, cudaStream_t s) {
+  static bool ready = false;
+  if (!ready) {
+    CMLD_TRY(allow_smem(latent_prefill_kernel<DV>, 227 * 1024));
+    ready = true;
+  }
+  return launch_kernel(latent_prefill_kernel<DV>, dim3((a.rows + kPfQ - 1) / kPfQ, a.m.heads), dim3(kPfThreads), pf_smem(pf_qd(a.m), DV), pdl, s, a);
+}
+
+}  // namespace
+
+bool latent_shape_ok(const LatentShape &m) {
+  return m.heads >= 1 && m.dim >= 1 && m.vdim >= 1 && m.rank >= 1 && m.rank <= 1024 && m.rot_dim >= 0 && m.rot_dims >= 0 && m.rot_dims % 2 == 0 &&
+         m.rot_dims <= m.rot_dim && att_smem(m.rank + m.rot_dim) <= 227 * 1024 && m.dim <= 4096;
+}
+
+int32_t launch_latent_prep(const LatentArgs &a, bool queries, bool pdl, cudaStream_t s) {
+  const int slices = (a.m.rank + kPrepRanks - 1) / kPrepRanks, ys = queries ? a.m.heads * slices : 0;
+  const int gx = std::min<int>(queries ? (a.rows + kPrepRows - 1) / kPrepRows : a.rows, 16384);
+  return launch_kernel(latent_prep_kernel, dim3(gx, ys + 1), dim3(kPrepThreads), (size_t)kPrepRows * a.m.dim * 4, pdl, s, a, slices, ys);
+}
+
+int32_t launch_latent_attention(const LatentArgs &a, bool pdl, cudaStream_t s) {
+  static bool ready = false;
+  if (!ready) {
+    CMLD_TRY(allow_smem(latent_attn_kernel<1>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_kernel<2>, 227 * 1024));
+    ready = true;
+  }
+  const dim3 grid(a.splits, (a.m.heads + kAttHeads - 1) / kAttHeads, a.rows);
+  const size_t smem = att_smem(a.m.rank + a.m.rot_dim);
+  if (a.m.rank <= 512) return launch_kernel(latent_attn_kernel<1>, grid, dim3(kAttThreads), smem, pdl, s, a);
+  return launch_kernel(latent_attn_kernel<2>, grid, dim3(kAttThreads), smem, pdl, s, a);
+}
+
+int32_t launch_latent_output(const LatentArgs &a, bool pdl, cudaStream_t s) {
+  if (a.splits > 64) return fail(CMLD_ERR_INVALID, "latent attention: %d ranges, at most 64", a.splits);
+  return launch_kernel(latent_output_kernel, dim3((a.m.vdim + kOutCols - 1) / kOutCols, a.m.heads, a.rows), dim3(kOutThreads), (size_t)a.uv.ld * 4, pdl, s, a);
+}
+
+bool latent_prefill_fits(const LatentShape &m, int64_t cache_ld, int64_t kv_ld) {
+  if (m.dim % 8 || m.rot_dim % 8 || m.vdim % 8 || m.rank % 8 || cache_ld % 8 || kv_ld % 8 || m.vdim > 256) return false;
+  const int dv = m.vdim <= 32 ? 32 : m.vdim <= 64 ? 64 : m.vdim <= 128 ? 128 : 256;
+  return pf_smem(pf_qd(m), dv) <= 227 * 1024;
+}
+
+int32_t launch_latent_prefill(const LatentPrefillArgs &a, bool pdl, cudaStream_t s) {
+  if (a.m.vdim <= 32) return prefill<32>(a, pdl, s);
+  if (a.m.vdim <= 64) return prefill<64>(a, pdl, s);
+  if (a.m.vdim <= 128) return prefill<128>(a, pdl, s);
+  return prefill<256>(a, pdl, s);
+}
+
+}  // namespace cmld

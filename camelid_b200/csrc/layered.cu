@@ -1,0 +1,839 @@
+// Layered designs behind the engine: a model described layer by layer (mixer type and sizes, feed-forward), with a
+// residual held as several streams and, optionally, a run of layers that is passed several times.
+//
+// The engine's own parts stay in charge: the token-driven calls, rows and slots, CUDA graphs of decode steps, argmax
+// and sampling (csrc/engine.cu).  This file owns the description, the named tensors, the caches and states, and the
+// step: which kernels run for `rows` rows.
+//
+// Three forms of a step share the kernels between the linear layers:
+//   one or two rows    fused matrix-vector products (csrc/lin_mv.cu), 32-bit activations
+//   more rows, bf16    tcgen05 products (csrc/lin_tc5.cu), bfloat16 activations, 32-bit residual, norms and scores
+//   more rows, f32     FP32 products (csrc/lin_f32.cu)
+//
+// Cache and state: per layer run (a looped layer counts once per pass) and slot, a latent layer keeps max_pos rows, a
+// lightning layer one state.  A sequence that starts at position 0 starts from nothing, whatever the slot held before;
+// any other start must be where the slot's sequence ends, because a state cannot be rewound.
+#include <cmath>
+
+#include "engine.cuh"
+#include "layered.cuh"
+
+namespace cmld {
+
+namespace {
+
+struct HyperW {
+  float *in = nullptr, *out = nullptr, *mix = nullptr;
+};
+struct NormW {
+  float *w = nullptr, *b = nullptr;
+};
+struct LayerDef {
+  cmld_layer_desc d{};
+  LinW in, uq, ukv, uk, uv, o, up, down;  // in: the projections that read the mixer's input, stacked
+  NormW norm1, norm2;
+  float *dq_norm = nullptr, *dkv_norm = nullptr, *mix_norm = nullptr;
+  HyperW hc[2];
+  float *powers = nullptr, *cs = nullptr;
+  LatentShape lat{};
+};
+struct Named {
+  std::string name;
+  int64_t rows = 0, cols = 0;  // rows == 0: a vector of cols f32 values (cols may itself be a product)
+  bf16 *m = nullptr;           // matrix destination, row stride ld
+  int64_t ld = 0;
+  float *v = nullptr;
+  bool set = false;
+};
+
+constexpr int kLatentRows = 256;    // rows whose queries are in latent space at a time
+constexpr int kExpandRows = 32;     // portions of this many rows expand keys and values
+constexpr int kPortionRows = 2048;  // rows of one step of a portion
+
+}  // namespace
+
+struct LayeredModel {
+  cmld_layered_config cfg{};
+  bool f32 = false;
+  std::vector<LayerDef> layers;
+  std::vector<int> order;       // layer of every run
+  std::vector<void *> store;    // per run: cache or state
+  LinW embed, head;
+  NormW embed_norm, final_norm;
+  std::vector<Named> named;
+  std::vector<int64_t> filled;  // per slot: tokens its sequence holds; -1: a call on it failed half-way
+  int64_t part_floats = 0;
+  // scratch, f32 unless noted
+  float *x[2] = {}, *y = nullptr, *proj = nullptr, *q = nullptr, *qa = nullptr, *part = nullptr, *taps = nullptr;
+  void *act = nullptr, *wide = nullptr, *mixed = nullptr, *hidden = nullptr;  // bf16 or f32
+  bf16 *kv = nullptr;
+  int32_t *row_map = nullptr;
+};
+
+namespace {
+
+int64_t cache_ld(const LayerDef &L) { return (L.d.kv_rank + L.d.rot_dim + 7) & ~7; }
+
+struct Builder {
+  cmld_engine *e;
+  LayeredModel *m;
+  int32_t rc = CMLD_OK;
+  void matrix(LinW &w, int64_t rows, int64_t cols) {
+    if (rc != CMLD_OK) return;
+    bf16 *p = nullptr;
+    w.rows = (int32_t)rows;
+    w.cols = (int32_t)cols;
+    w.ld = lin_ld(cols);
+    rc = dev_alloc(e, &p, rows * w.ld);  // zeroed: the padding stays zero
+    w.w = p;
+  }
+  // rows [row0, row0 + rows) of w under `name`
+  void name_rows(const std::string &name, const LinW &w, int64_t row0, int64_t rows) {
+    Named n;
+    n.name = name;
+    n.rows = rows;
+    n.cols = w.cols;
+    n.m = const_cast<bf16 *>(w.w) + row0 * w.ld;
+    n.ld = w.ld;
+    m->named.push_back(n);
+  }
+  void named_matrix(const std::string &name, LinW &w, int64_t rows, int64_t cols) {
+    matrix(w, rows, cols);
+    if (rc == CMLD_OK) name_rows(name, w, 0, rows);
+  }
+  void vector(const std::string &name, float *&v, int64_t n) {
+    if (rc != CMLD_OK) return;
+    rc = dev_alloc(e, &v, n);
+    Named d;
+    d.name = name;
+    d.cols = n;
+    d.v = v;
+    m->named.push_back(d);
+  }
+  void norm(const std::string &name, NormW &n) {
+    vector(name, n.w, m->cfg.width);
+    vector(name + ".b", n.b, m->cfg.width);
+  }
+  void hyper(const std::string &name, HyperW &h) {
+    vector(name + ".in", h.in, m->cfg.streams);
+    vector(name + ".out", h.out, m->cfg.streams);
+    vector(name + ".mix", h.mix, (int64_t)m->cfg.streams * m->cfg.streams);
+  }
+};
+
+int32_t check_layer(const cmld_layer_desc &d, int i) {
+  if (d.type == CMLD_LAYER_LATENT) {
+    const LatentShape s{d.heads, d.dim, d.rot_dim, d.rot_dims, d.vdim, d.kv_rank, d.scale, 0.0f};
+    if (d.q_rank < 1 || !latent_shape_ok(s)) return fail(CMLD_ERR_SHAPE, "layer %d: latent attention sizes not supported", i);
+    if (d.rot_dims > 0 && !(d.rot_base > 0.0)) return fail(CMLD_ERR_INVALID, "layer %d: rotation base must be positive", i);
+  } else if (d.type == CMLD_LAYER_LIGHTNING) {
+    if (!lightning_shape_ok(d.heads, d.dim, d.vdim)) return fail(CMLD_ERR_SHAPE, "layer %d: lightning attention sizes not supported", i);
+    if (!d.decay) return fail(CMLD_ERR_INVALID, "layer %d: decays are missing", i);
+  } else {
+    return fail(CMLD_ERR_UNSUPPORTED, "layer %d: mixer type %d", i, d.type);
+  }
+  if (d.ff < 0) return fail(CMLD_ERR_SHAPE, "layer %d: feed-forward width %d", i, d.ff);
+  return CMLD_OK;
+}
+
+// Angles position * base^(-2i / dims) in 32-bit, their cosine and sine: [position][pair][2].
+int32_t rotation_table(cmld_engine *e, int64_t max_pos, int dims, double base, float **out) {
+  const int half = dims / 2;
+  std::vector<float> f(half), t((size_t)max_pos * dims);
+  for (int i = 0; i < half; ++i) f[i] = (float)std::pow(base, -2.0 * i / dims);
+  for (int64_t p = 0; p < max_pos; ++p)
+    for (int i = 0; i < half; ++i) {
+      const float a = (float)p * f[i];
+      t[(size_t)p * dims + 2 * i] = (float)std::cos((double)a);
+      t[(size_t)p * dims + 2 * i + 1] = (float)std::sin((double)a);
+    }
+  CMLD_TRY(dev_alloc(e, out, (int64_t)t.size(), false));
+  CMLD_CUDA(cudaMemcpyAsync(*out, t.data(), t.size() * 4, cudaMemcpyHostToDevice, e->stream));
+  CMLD_CUDA(cudaStreamSynchronize(e->stream));
+  return CMLD_OK;
+}
+
+int32_t build(cmld_engine *e, LayeredModel *m) {
+  const cmld_layered_config &c = m->cfg;
+  Builder b{e, m};
+  b.named_matrix("embed", m->embed, c.vocab, c.width);
+  b.norm("embed.norm", m->embed_norm);
+  std::map<std::pair<int, double>, float *> tables;
+  for (int i = 0; i < c.n_layers; ++i) {
+    LayerDef &L = m->layers[i];
+    const cmld_layer_desc &d = L.d;
+    const std::string p = "l" + std::to_string(i) + ".", mx = p + "mix.";
+    const int64_t H = d.heads;
+    b.norm(p + "norm1", L.norm1);
+    if (d.type == CMLD_LAYER_LATENT) {
+      b.matrix(L.in, d.q_rank + d.kv_rank + d.rot_dim + H * d.vdim, c.width);
+      b.matrix(L.ukv, H * (d.dim + d.vdim), d.kv_rank);
+      CMLD_TRY(b.rc);
+      b.name_rows(mx + "dq", L.in, 0, d.q_rank);
+      b.name_rows(mx + "dkv", L.in, d.q_rank, d.kv_rank + d.rot_dim);
+      b.name_rows(mx + "g", L.in, d.q_rank + d.kv_rank + d.rot_dim, H * d.vdim);
+      b.vector(mx + "dq.norm", L.dq_norm, d.q_rank);
+      b.vector(mx + "dkv.norm", L.dkv_norm, d.kv_rank);
+      b.named_matrix(mx + "uq", L.uq, H * (d.dim + d.rot_dim), d.q_rank);
+      b.name_rows(mx + "uk", L.ukv, 0, H * d.dim);
+      b.name_rows(mx + "uv", L.ukv, H * d.dim, H * d.vdim);
+      L.uk = L.uv = L.ukv;
+      L.uk.rows = (int32_t)(H * d.dim);
+      L.uv.rows = (int32_t)(H * d.vdim);
+      L.uv.w = L.ukv.w + H * d.dim * L.ukv.ld;
+      L.lat = LatentShape{d.heads, d.dim, d.rot_dim, d.rot_dims, d.vdim, d.kv_rank, d.scale, c.eps};
+      if (d.rot_dims > 0) {
+        float *&t = tables[{d.rot_dims, d.rot_base}];
+        if (!t) CMLD_TRY(rotation_table(e, c.max_pos, d.rot_dims, d.rot_base, &t));
+        L.cs = t;
+      }
+    } else {
+      b.matrix(L.in, H * (2 * d.dim + 2 * d.vdim), c.width);
+      CMLD_TRY(b.rc);
+      b.name_rows(mx + "q", L.in, 0, H * d.dim);
+      b.name_rows(mx + "k", L.in, H * d.dim, H * d.dim);
+      b.name_rows(mx + "v", L.in, 2 * H * d.dim, H * d.vdim);
+      b.name_rows(mx + "g", L.in, 2 * H * d.dim + H * d.vdim, H * d.vdim);
+      b.vector(mx + "norm", L.mix_norm, H * d.vdim);
+      std::vector<float> pw((size_t)H * (kLightningChunk + 1));
+      for (int h = 0; h < d.heads; ++h)
+        for (int j = 0; j <= kLightningChunk; ++j) pw[(size_t)h * (kLightningChunk + 1) + j] = (float)std::pow((double)d.decay[h], (double)j);
+      CMLD_TRY(dev_alloc(e, &L.powers, (int64_t)pw.size(), false));
+      CMLD_CUDA(cudaMemcpyAsync(L.powers, pw.data(), pw.size() * 4, cudaMemcpyHostToDevice, e->stream));
+      CMLD_CUDA(cudaStreamSynchronize(e->stream));
+    }
+    b.named_matrix(mx + "o", L.o, c.width, H * d.vdim);
+    b.hyper(p + "hc1", L.hc[0]);
+    if (d.ff > 0) {
+      b.norm(p + "norm2", L.norm2);
+      b.named_matrix(p + "mlp.up", L.up, d.ff, c.width);
+      b.named_matrix(p + "mlp.down", L.down, c.width, d.ff);
+      b.hyper(p + "hc2", L.hc[1]);
+    }
+    L.d.decay = nullptr;  // the caller's memory
+    CMLD_TRY(b.rc);
+  }
+  b.norm("final.norm", m->final_norm);
+  b.named_matrix("head", m->head, c.vocab, c.width);
+  CMLD_TRY(b.rc);
+
+  // order of runs
+  const int times = std::max(1, c.loop_times);
+  for (int i = 0; i < c.loop_start; ++i) m->order.push_back(i);
+  for (int t = 0; t < times; ++t)
+    for (int i = c.loop_start; i < c.loop_stop; ++i) m->order.push_back(i);
+  for (int i = c.loop_stop; i < c.n_layers; ++i) m->order.push_back(i);
+
+  // caches and states
+  const int64_t slots = std::max(1, c.max_seqs);
+  m->filled.assign(slots, 0);
+  const int64_t es = m->f32 ? 4 : 2;
+  for (int li : m->order) {
+    const LayerDef &L = m->layers[li];
+    uint8_t *p = nullptr;
+    const int64_t bytes = L.d.type == CMLD_LAYER_LATENT ? slots * c.max_pos * cache_ld(L) * es : slots * L.d.heads * (int64_t)L.d.dim * L.d.vdim * 4;
+    CMLD_TRY(dev_alloc(e, &p, bytes));
+    m->store.push_back(p);
+  }
+
+  // scratch for the widest layer
+  const int64_t R = std::max<int64_t>(slots, std::min<int64_t>(c.max_pos, kPortionRows));
+  CMLD_TRY(init_rows(e, R, std::max<int64_t>(slots, 32), c.vocab));
+  int64_t proj = 1, q = 1, wide = 1, mixed = 1, ff = 1, kv = 0, qa = 1, part = 1;
+  for (const LayerDef &L : m->layers) {
+    const cmld_layer_desc &d = L.d;
+    const int64_t H = d.heads;
+    mixed = std::max(mixed, lin_ld(H * d.vdim));
+    ff = std::max(ff, lin_ld(std::max(d.ff, 1)));
+    if (d.type == CMLD_LAYER_LATENT) {
+      proj = std::max<int64_t>(proj, L.in.rows);
+      q = std::max(q, H * (d.dim + d.rot_dim));
+      wide = std::max(wide, lin_ld(d.q_rank));
+      const int64_t kv_ld = lin_ld(H * (d.dim + d.vdim));
+      if (!m->f32 && latent_prefill_fits(L.lat, cache_ld(L), kv_ld)) kv = std::max(kv, kv_ld);
+      qa = std::max(qa, H * (d.kv_rank + d.rot_dim));
+      const int64_t groups = (H + 7) / 8;
+      part = std::max(part, (int64_t)(2 * e->sm_count * 8 + std::min<int64_t>(R, kLatentRows) * groups * 8) * (d.kv_rank + 2));
+    } else {
+      wide = std::max(wide, lin_ld(L.in.rows));
+      proj = std::max<int64_t>(proj, H * d.vdim);
+    }
+  }
+  m->part_floats = part;
+  for (float *&x : m->x) CMLD_TRY(dev_alloc(e, &x, R * c.streams * c.width));
+  CMLD_TRY(dev_alloc(e, &m->y, R * c.width));
+  CMLD_TRY(dev_alloc(e, &m->proj, R * proj));
+  CMLD_TRY(dev_alloc(e, &m->q, R * q));
+  CMLD_TRY(dev_alloc(e, &m->qa, std::min<int64_t>(R, kLatentRows) * qa));
+  CMLD_TRY(dev_alloc(e, &m->part, part));
+  float *f = nullptr;  // sized for f32 rows: steps of one or two rows keep 32-bit activations in either precision
+  CMLD_TRY(dev_alloc(e, &f, R * lin_ld(c.width)));
+  m->act = f;
+  CMLD_TRY(dev_alloc(e, &f, R * wide));
+  m->wide = f;
+  CMLD_TRY(dev_alloc(e, &f, R * mixed));
+  m->mixed = f;
+  CMLD_TRY(dev_alloc(e, &f, R * ff));
+  m->hidden = f;
+  if (kv > 0) CMLD_TRY(dev_alloc(e, &m->kv, c.max_pos * kv));
+  CMLD_TRY(dev_alloc(e, &m->row_map, std::max<int64_t>(slots, 32)));
+  CMLD_CUDA(cudaStreamSynchronize(e->stream));
+  return CMLD_OK;
+}
+
+int32_t validate(const cmld_layered_config &c) {
+  if (c.n_layers < 1 || c.streams < 1 || c.width < 1 || c.vocab < 1 || c.max_pos < 1 || !c.layers) return fail(CMLD_ERR_SHAPE, "layered model: dimensions must be positive");
+  if (c.max_pos > (1 << 24)) return fail(CMLD_ERR_SHAPE, "max_pos too large");
+  if (c.width > 16384) return fail(CMLD_ERR_SHAPE, "width %d, at most 16384", c.width);
+  if (c.loop_start < 0 || c.loop_stop < c.loop_start || c.loop_stop > c.n_layers || c.loop_times < 0)
+    return fail(CMLD_ERR_INVALID, "loop %d..%d x %d does not fit %d layers", c.loop_start, c.loop_stop, c.loop_times, c.n_layers);
+  if (c.dtype != CMLD_BF16 && c.dtype != CMLD_F32) return fail(CMLD_ERR_UNSUPPORTED, "layered models compute in bfloat16 or 32-bit");
+  for (int i = 0; i < c.n_layers; ++i) CMLD_TRY(check_layer(c.layers[i], i));
+  return CMLD_OK;
+}
+
+// ---------------------------------------------------------------- the step
+
+struct Step {
+  cmld_engine *e;
+  LayeredModel *m;
+  const StepOpts &o;
+  int32_t R;
+  bool mv, pdl, half;        // matrix-vector form; programmatic dependent launches; bf16 activations
+  int cur = 0;
+  const HyperW *pending = nullptr;
+
+  StreamMix boundary(const float *in, const NormW &n) {
+    StreamMix s{};
+    s.streams = m->cfg.streams;
+    s.width = m->cfg.width;
+    s.eps = m->cfg.eps;
+    s.in = in;
+    s.norm_w = n.w;
+    s.norm_b = n.b;
+    if (!pending) {
+      s.embed = m->embed.w;
+      s.embed_ld = m->embed.ld;
+      s.tokens = e->d_tokens;
+      s.enorm_w = m->embed_norm.w;
+      s.enorm_b = m->embed_norm.b;
+    } else {
+      s.x_in = m->x[cur];
+      s.y = m->y;
+      s.mix = pending->mix;
+      s.out = pending->out;
+    }
+    s.x_out = m->x[cur ^ 1];
+    cur ^= 1;
+    return s;
+  }
+  ActBuf buf(void *p, int64_t cols) const { return ActBuf{p, half ? 1 : 0, lin_ld(cols)}; }
+
+  int32_t vec(LinMvArgs a) {
+    a.batch = R;
+    e->launches += 1;
+    return launch_lin_mv(a, pdl, e->stream);
+  }
+  int32_t lin(const LinW &w, ActBuf x, void *out, bool out_half, int64_t out_ld, int act = kActNone, int act_rows = 0, int32_t rows = -1) {
+    LinArgs a{};
+    a.w = w;
+    a.x = x.p;
+    a.x_ld = x.ld;
+    a.rows = rows < 0 ? R : rows;
+    a.out = out;
+    a.out_half = out_half;
+    a.out_ld = out_ld;
+    a.act = act;
+    a.act_rows = act_rows;
+    e->launches += 1;
+    return x.half ? launch_lin_tc5(a, e->sm_count, e->d_status, pdl, e->stream) : launch_lin_f32(a, e->stream);
+  }
+  // The sublayer boundary followed by the linear layer that reads it.
+  int32_t read_in(const StreamMix &s, const LinW &w, void *out, bool out_half, int64_t out_ld, int act, int act_rows) {
+    if (mv) {
+      LinMvArgs a{};
+      a.w = w;
+      a.prologue = kProStreams;
+      a.mix = s;
+      a.y = static_cast<float *>(out);
+      a.y_ld = out_ld;
+      a.act = act;
+      a.act_rows = act_rows;
+      return vec(a);
+    }
+    const ActBuf h = buf(m->act, m->cfg.width);
+    e->launches += 1;
+    CMLD_TRY(launch_stream_mix(s, R, h, pdl, e->stream));
+    return lin(w, h, out, out_half, out_ld, act, act_rows);
+  }
+  int32_t vec_plain(const LinW &w, const float *x, int64_t x_ld, float *y, int64_t y_ld) {
+    LinMvArgs a{};
+    a.w = w;
+    a.x = x;
+    a.x_ld = x_ld;
+    a.y = y;
+    a.y_ld = y_ld;
+    return vec(a);
+  }
+
+  int32_t latent(const LayerDef &L, void *store, const StreamMix &s) {
+    const cmld_layer_desc &d = L.d;
+    const int64_t pl = L.in.rows, kv0 = d.q_rank, g0 = d.q_rank + d.kv_rank + d.rot_dim, ql = L.uq.rows, ov = (int64_t)d.heads * d.vdim;
+    CMLD_TRY(read_in(s, L.in, m->proj, false, pl, kActNone, 0));
+    if (mv) {
+      LinMvArgs a{};
+      a.w = L.uq;
+      a.prologue = kProRms;
+      a.x = m->proj;
+      a.x_ld = pl;
+      a.norm_w = L.dq_norm;
+      a.eps = m->cfg.eps;
+      a.y = m->q;
+      a.y_ld = ql;
+      CMLD_TRY(vec(a));
+    } else {
+      const ActBuf cq = buf(m->wide, d.q_rank);
+      CMLD_TRY(launch_rms_rows(m->proj, pl, L.dq_norm, d.q_rank, m->cfg.eps, ActBuf{}, cq, R, pdl, e->stream));
+      e->launches += 1;
+      CMLD_TRY(lin(L.uq, cq, m->q, false, ql));
+    }
+    LatentArgs a{};
+    a.m = L.lat;
+    a.cs = L.cs;
+    a.cache = store;
+    a.cache_half = m->f32 ? 0 : 1;
+    a.cache_ld = cache_ld(L);
+    a.max_pos = m->cfg.max_pos;
+    a.low_ld = pl;
+    a.latent_norm = L.dkv_norm;
+    a.uk = L.uk;
+    a.uv = L.uv;
+    a.qa = m->qa;
+    a.part = m->part;
+    a.gate_ld = pl;
+    const ActBuf out = buf(m->mixed, ov);
+    const int64_t kv_ld = lin_ld(L.ukv.rows);
+    const bool expand = half && o.shared_slots && R >= kExpandRows && latent_prefill_fits(L.lat, a.cache_ld, kv_ld);
+    // every row's cache entry goes in before any row attends
+    const bool append_first = expand || R > kLatentRows;
+    auto rows_from = [&](int r0, int n) {
+      a.rows = n;
+      a.positions = e->d_positions + r0;
+      a.slots = e->d_slots + r0;
+      a.low = m->proj + (int64_t)r0 * pl + kv0;
+      a.q = m->q + (int64_t)r0 * ql;
+      a.gate = m->proj + (int64_t)r0 * pl + g0;
+      a.out = out;
+      a.out.p = static_cast<uint8_t *>(out.p) + (int64_t)r0 * out.ld * (out.half ? 2 : 4);
+    };
+    if (append_first) {
+      rows_from(0, R);
+      CMLD_TRY(launch_latent_prep(a, false, pdl, e->stream));
+      e->launches += 1;
+    }
+    if (expand) {
+      const int64_t total = o.seq_start + R;
+      const bf16 *c = static_cast<const bf16 *>(store) + (int64_t)o.seq_slot * a.max_pos * a.cache_ld;
+      CMLD_TRY(lin(L.ukv, ActBuf{const_cast<bf16 *>(c), 1, a.cache_ld}, m->kv, true, kv_ld, kActNone, 0, (int32_t)total));
+      LatentPrefillArgs p{};
+      p.m = L.lat;
+      p.rows = R;
+      p.start = o.seq_start;
+      p.cs = L.cs;
+      p.cache = c;
+      p.cache_ld = a.cache_ld;
+      p.kv = m->kv;
+      p.kv_ld = kv_ld;
+      p.q = m->q;
+      p.gate = m->proj + g0;
+      p.gate_ld = pl;
+      p.out = static_cast<bf16 *>(out.p);
+      p.out_ld = out.ld;
+      CMLD_TRY(launch_latent_prefill(p, pdl, e->stream));
+      e->launches += 1;
+    } else {
+      const int groups = (d.heads + 7) / 8;
+      const int64_t cap = o.attn_cap > 0 ? o.attn_cap : m->cfg.max_pos;
+      for (int r0 = 0; r0 < R; r0 += kLatentRows) {
+        const int n = std::min(kLatentRows, R - r0);
+        rows_from(r0, n);
+        a.splits = (int)std::max<int64_t>(1, std::min<int64_t>({64, (2 * e->sm_count) / (n * groups), cap / 64}));
+        if ((int64_t)n * d.heads * a.splits * (d.kv_rank + 2) > m->part_floats) return fail(CMLD_ERR_STATE, "latent attention: partials exceed the scratch");
+        CMLD_TRY(launch_latent_prep(a, true, pdl, e->stream));
+        CMLD_TRY(launch_latent_attention(a, pdl, e->stream));
+        CMLD_TRY(launch_latent_output(a, pdl, e->stream));
+        e->launches += 3;
+      }
+    }
+    if (mv) return vec_plain(L.o, static_cast<float *>(out.p), out.ld, m->y, m->cfg.width);
+    return lin(L.o, out, m->y, false, m->cfg.width);
+  }
+
+  int32_t lightning(const LayerDef &L, void *store, const StreamMix &s) {
+    const cmld_layer_desc &d = L.d;
+    const int64_t ld = lin_ld(L.in.rows), ov = (int64_t)d.heads * d.vdim, g0 = (int64_t)d.heads * (2 * d.dim + d.vdim);
+    CMLD_TRY(read_in(s, L.in, m->wide, half, ld, kActSilu, (int)g0));
+    LightningArgs a{};
+    a.heads = d.heads;
+    a.dim = d.dim;
+    a.vdim = d.vdim;
+    a.powers = L.powers;
+    a.state = static_cast<float *>(store);
+    a.qkv = m->wide;
+    a.half = half;
+    a.ld = ld;
+    a.out = m->proj;
+    a.positions = e->d_positions;
+    a.slots = e->d_slots;
+    a.rows = R;
+    a.one_sequence = o.shared_slots;
+    e->launches += 1;
+    if (R >= kLightningChunk / 4 && lightning_chunk_fits(a)) CMLD_TRY(launch_lightning_chunks(a, pdl, e->stream));
+    else CMLD_TRY(launch_lightning_steps(a, pdl, e->stream));
+    if (mv) {
+      LinMvArgs v{};
+      v.w = L.o;
+      v.prologue = kProRmsGate;
+      v.x = m->proj;
+      v.x_ld = ov;
+      v.norm_w = L.mix_norm;
+      v.eps = m->cfg.eps;
+      v.gate = static_cast<float *>(m->wide) + g0;
+      v.gate_ld = ld;
+      v.y = m->y;
+      v.y_ld = m->cfg.width;
+      return vec(v);
+    }
+    const ActBuf out = buf(m->mixed, ov);
+    ActBuf gate{static_cast<uint8_t *>(m->wide) + g0 * (half ? 2 : 4), half ? 1 : 0, ld};
+    CMLD_TRY(launch_rms_rows(m->proj, ov, L.mix_norm, (int)ov, m->cfg.eps, gate, out, R, pdl, e->stream));
+    e->launches += 1;
+    return lin(L.o, out, m->y, false, m->cfg.width);
+  }
+
+  int32_t mlp(const LayerDef &L, const StreamMix &s) {
+    const ActBuf h = buf(m->hidden, L.d.ff);
+    CMLD_TRY(read_in(s, L.up, h.p, half, h.ld, kActRelu2, 0));
+    if (mv) return vec_plain(L.down, static_cast<float *>(h.p), h.ld, m->y, m->cfg.width);
+    return lin(L.down, h, m->y, false, m->cfg.width);
+  }
+
+  int32_t head() {
+    StreamMix s = boundary(nullptr, m->final_norm);
+    s.x_out = nullptr;
+    const int32_t n = o.n_want < 0 ? R : o.n_want;
+    if (o.n_want >= 0) s.row_map = m->row_map;
+    if (n <= 2 && lin_mv_fits(m->cfg.width, n)) {
+      LinMvArgs a{};
+      a.w = m->head;
+      a.batch = n;
+      a.prologue = kProStreams;
+      a.mix = s;
+      a.y = e->logits;
+      a.y_ld = m->cfg.vocab;
+      e->launches += 1;
+      return launch_lin_mv(a, pdl, e->stream);
+    }
+    const ActBuf h{m->act, m->f32 ? 0 : 1, lin_ld(m->cfg.width)};
+    CMLD_TRY(launch_stream_mix(s, n, h, pdl, e->stream));
+    e->launches += 1;
+    return lin(m->head, h, e->logits, false, m->cfg.vocab, kActNone, 0, n);
+  }
+};
+
+bool all_fit_mv(const LayeredModel *m, int32_t R) {
+  if (!lin_mv_fits(m->cfg.width, R)) return false;
+  for (const LayerDef &L : m->layers)
+    for (int64_t cols : {(int64_t)L.d.heads * L.d.vdim, (int64_t)L.d.ff, (int64_t)L.d.q_rank})
+      if (cols > 0 && !lin_mv_fits((int32_t)cols, R)) return false;
+  return true;
+}
+
+}  // namespace
+
+int32_t layered_step(cmld_engine *e, const StepOpts &o) {
+  LayeredModel *m = e->lay;
+  const int32_t R = o.batch;
+  if (R < 1 || R > e->max_rows) return fail(CMLD_ERR_INVALID, "step of %d rows exceeds the engine's %d", R, e->max_rows);
+  const int32_t n_logits = !o.logits ? 0 : o.n_want < 0 ? R : o.n_want;
+  if (n_logits > e->logit_rows) return fail(CMLD_ERR_INVALID, "logits of %d rows exceed the engine's %d", n_logits, e->logit_rows);
+  const bool mv = all_fit_mv(m, R);
+  Step st{e, m, o, R, mv, !(e->cfg.flags & CMLD_FLAG_NO_PDL), !mv && !m->f32};
+  const int64_t W = m->cfg.width;
+  for (size_t run = 0; run < m->order.size(); ++run) {
+    const LayerDef &L = m->layers[m->order[run]];
+    const StreamMix s = st.boundary(L.hc[0].in, L.norm1);
+    CMLD_TRY(L.d.type == CMLD_LAYER_LATENT ? st.latent(L, m->store[run], s) : st.lightning(L, m->store[run], s));
+    st.pending = &L.hc[0];
+    if (L.d.ff > 0) {
+      CMLD_TRY(st.mlp(L, st.boundary(L.hc[1].in, L.norm2)));
+      st.pending = &L.hc[1];
+    }
+    if (o.taps_out) {
+      const int cur = st.cur;
+      StreamMix t = st.boundary(nullptr, NormW{});
+      t.x_out = nullptr;
+      st.cur = cur;
+      CMLD_TRY(launch_stream_tap(t, R, o.taps_out + (int64_t)run * R * W, e->stream));
+    }
+  }
+  if (n_logits > 0) {
+    CMLD_TRY(st.head());
+    if (o.argmax) {
+      CMLD_TRY(launch_argmax(e->logits, m->cfg.vocab, n_logits, e->am_val, e->am_idx, e->am_ticket, e->out_idx, o.feed_back ? e->d_tokens : nullptr,
+                             e->d_positions, e->d_history, e->stream));
+      e->launches += 1;
+    }
+  }
+  return CMLD_OK;
+}
+
+int32_t layered_ready(const cmld_engine *e, bool report) {
+  for (const Named &n : e->lay->named)
+    if (!n.set) {
+      if (report) fail(CMLD_ERR_STATE, "tensor %s is not set", n.name.c_str());
+      return 0;
+    }
+  return 1;
+}
+
+// Before a call touches the rows' slots: each row starts a sequence (position 0) or continues the slot's, one row per slot.
+int32_t layered_claim(cmld_engine *e, int32_t n, const int32_t *seqs, const int64_t *positions) {
+  LayeredModel *m = e->lay;
+  for (int i = 0; i < n; ++i) {
+    for (int j = 0; j < i; ++j)
+      if (seqs[i] == seqs[j]) return fail(CMLD_ERR_INVALID, "slot %d appears twice in a step (use cmld_engine_extend for several tokens of a sequence)", seqs[i]);
+    if (positions[i] != 0 && m->filled[seqs[i]] != positions[i])
+      return fail(CMLD_ERR_STATE, "slot %d holds %lld tokens: its sequence cannot continue at position %lld", seqs[i], (long long)m->filled[seqs[i]],
+                  (long long)positions[i]);
+  }
+  for (int i = 0; i < n; ++i) m->filled[seqs[i]] = -1;  // until the call has succeeded
+  return CMLD_OK;
+}
+
+void layered_advance(cmld_engine *e, int32_t n, const int32_t *seqs, const int64_t *positions, int64_t steps) {
+  for (int i = 0; i < n; ++i) e->lay->filled[seqs[i]] = positions[i] + steps;
+}
+
+int32_t layered_extend(cmld_engine *e, int32_t seq, const int32_t *tokens, int64_t n, int64_t start, const int32_t *want, int32_t n_want,
+                       float *logits_out, float *taps_out) {
+  LayeredModel *m = e->lay;
+  const cmld_layered_config &c = m->cfg;
+  if (seq < 0 || seq >= (int32_t)m->filled.size()) return fail(CMLD_ERR_INVALID, "sequence slot %d out of range (max_seqs %zu)", seq, m->filled.size());
+  if (start < 0 || start + n > c.max_pos) return fail(CMLD_ERR_STATE, "positions %lld..%lld exceed max_pos %d", (long long)start, (long long)(start + n - 1), c.max_pos);
+  for (int64_t i = 0; i < n; ++i)
+    if (tokens[i] < 0 || tokens[i] >= c.vocab) return fail(CMLD_ERR_INVALID, "token id %d out of range", tokens[i]);
+  CMLD_TRY(layered_claim(e, 1, &seq, &start));
+  const int64_t runs = (int64_t)m->order.size();
+  int32_t w = 0;
+  for (int64_t i = 0; i < n; i += e->max_rows) {
+    const int rows = (int)std::min<int64_t>(e->max_rows, n - i);
+    std::vector<int32_t> pos(rows), slots(rows, seq);
+    for (int r = 0; r < rows; ++r) pos[r] = (int32_t)(start + i + r);
+    CMLD_TRY(stage_rows(e, rows, tokens + i, pos.data(), slots.data()));
+    StepOpts o;
+    o.batch = rows;
+    o.shared_slots = rows > 1;
+    o.from_tokens = true;
+    o.seq_start = start + i;
+    o.seq_slot = seq;
+    o.attn_cap = 512;
+    while (o.attn_cap <= start + i + rows - 1) o.attn_cap *= 2;
+    float *taps = nullptr;
+    if (taps_out) {
+      CMLD_CUDA(cudaMalloc(&taps, (size_t)runs * rows * c.width * 4));
+      o.taps_out = taps;
+    }
+    // The rows whose logits are wanted, as many at a time as the logits buffer holds; after the last token always its own.
+    const bool last = i + rows >= n;
+    std::vector<int32_t> ask;
+    while (w + (int32_t)ask.size() < n_want && want[w + ask.size()] < i + rows) ask.push_back((int32_t)(want[w + ask.size()] - i));
+    const int32_t live = (int32_t)ask.size();
+    if (last && (ask.empty() || ask.back() != rows - 1)) ask.push_back(rows - 1);
+    if (rows == 1 && !taps && last) {
+      // the shape of a decode step, and its graph
+      CMLD_TRY(run_step(e, o));
+      e->last_logit_row = 0;
+      if (live) CMLD_CUDA(cudaMemcpyAsync(logits_out + (int64_t)w * c.vocab, e->logits, (size_t)c.vocab * 4, cudaMemcpyDeviceToHost, e->stream));
+    } else {
+      o.logits = false;
+      int32_t rc = layered_step(e, o);
+      // the stream after the last layer is still in place: read it out for the rows asked for
+      Step st{e, m, o, rows, all_fit_mv(m, rows), !(e->cfg.flags & CMLD_FLAG_NO_PDL), false};
+      int flips = 0;
+      for (int li : m->order) flips += m->layers[li].d.ff > 0 ? 2 : 1;
+      const LayerDef &tail = m->layers[m->order.back()];
+      for (size_t a = 0; a < ask.size() && rc == CMLD_OK; a += e->logit_rows) {
+        const int32_t k = (int32_t)std::min<size_t>(e->logit_rows, ask.size() - a);
+        cudaError_t ce = cudaMemcpyAsync(m->row_map, ask.data() + a, (size_t)k * 4, cudaMemcpyHostToDevice, e->stream);
+        o.n_want = k;
+        st.pending = &tail.hc[tail.d.ff > 0 ? 1 : 0];
+        st.cur = flips & 1;
+        if (ce == cudaSuccess) rc = st.head();
+        if (rc == CMLD_OK && ce == cudaSuccess)
+          rc = launch_argmax(e->logits, c.vocab, k, e->am_val, e->am_idx, e->am_ticket, e->out_idx, nullptr, e->d_positions, e->d_history, e->stream);
+        const int32_t give = std::max(0, std::min<int32_t>(k, live - (int32_t)a));
+        if (rc == CMLD_OK && ce == cudaSuccess && give > 0)
+          ce = cudaMemcpyAsync(logits_out + (int64_t)(w + a) * c.vocab, e->logits, (size_t)give * c.vocab * 4, cudaMemcpyDeviceToHost, e->stream);
+        if (ce != cudaSuccess) rc = fail(CMLD_ERR_CUDA, "extend: %s", cudaGetErrorString(ce));
+        e->launches += 1;
+        e->last_logit_row = k - 1;
+      }
+      if (taps && rc == CMLD_OK) {
+        for (int64_t r = 0; r < runs && rc == CMLD_OK; ++r)
+          if (cudaMemcpyAsync(taps_out + (r * n + i) * c.width, taps + r * rows * c.width, (size_t)rows * c.width * 4, cudaMemcpyDeviceToHost, e->stream) != cudaSuccess)
+            rc = fail(CMLD_ERR_CUDA, "extend: copying the residual stream failed");
+      }
+      if (taps) {
+        cudaStreamSynchronize(e->stream);
+        cudaFree(taps);
+      }
+      CMLD_TRY(rc);
+    }
+    w += live;
+  }
+  return CMLD_OK;
+}
+
+void layered_free(cmld_engine *e) {
+  delete e->lay;
+  e->lay = nullptr;
+}
+
+// f32 or bfloat16 values -> a padded bfloat16 matrix, or an f32 vector
+__global__ void named_from_f32_kernel(const float *src, int64_t rows, int64_t cols, bf16 *m, int64_t ld, float *v, float add) {
+  for (int64_t i = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; i < rows * cols; i += (int64_t)gridDim.x * blockDim.x) {
+    if (m) m[i / cols * ld + i % cols] = __float2bfloat16_rn(src[i] + add);
+    else v[i] = __bfloat162float(__float2bfloat16_rn(src[i] + add));
+  }
+}
+
+static Named *find_named(cmld_engine *e, const char *name) {
+  for (Named &n : e->lay->named)
+    if (n.name == name) return &n;
+  return nullptr;
+}
+
+}  // namespace cmld
+
+using namespace cmld;
+
+extern "C" {
+
+int32_t cmld_engine_create_layered(const cmld_layered_config *cfg, cmld_engine **out) {
+  if (!cfg || !out) return fail(CMLD_ERR_INVALID, "config or out pointer is null");
+  *out = nullptr;
+  CMLD_TRY(validate(*cfg));
+  int ndev = 0;
+  if (cudaGetDeviceCount(&ndev) != cudaSuccess || ndev == 0) {
+    cudaGetLastError();
+    return fail(CMLD_ERR_CUDA, "no CUDA device: this engine has no CPU path");
+  }
+  int dev = cfg->device;
+  if (dev < 0) CMLD_CUDA(cudaGetDevice(&dev));
+  if (dev >= ndev) return fail(CMLD_ERR_INVALID, "device %d out of range (%d present)", dev, ndev);
+  cudaDeviceProp prop{};
+  CMLD_CUDA(cudaGetDeviceProperties(&prop, dev));
+  if (prop.major != 10) return fail(CMLD_ERR_UNSUPPORTED, "device %d is sm_%d%d; this library is built for sm_100a only", dev, prop.major, prop.minor);
+  DeviceGuard guard(dev);
+  if (!guard.ok) return fail(CMLD_ERR_CUDA, "cannot select CUDA device %d", dev);
+  cmld_engine *e = new cmld_engine();
+  e->lay = new LayeredModel();
+  e->lay->cfg = *cfg;
+  e->lay->f32 = cfg->dtype == CMLD_F32;
+  e->lay->layers.resize(cfg->n_layers);
+  for (int i = 0; i < cfg->n_layers; ++i) e->lay->layers[i].d = cfg->layers[i];
+  e->lay->cfg.layers = nullptr;
+  e->cfg.n_layers = cfg->n_layers;
+  e->cfg.hidden = cfg->width;
+  e->cfg.head_dim = 1;
+  e->cfg.vocab = cfg->vocab;
+  e->cfg.max_pos = cfg->max_pos;
+  e->cfg.max_seqs = std::max(1, cfg->max_seqs);
+  e->cfg.eps = cfg->eps;
+  e->cfg.flags = cfg->flags;
+  e->full = e->cfg;
+  e->vocab_local = cfg->vocab;
+  e->device = dev;
+  int32_t rc = engine_open(e, dev);
+  if (rc == CMLD_OK) rc = build(e, e->lay);
+  if (rc != CMLD_OK) {
+    cmld_engine_destroy(e);
+    return rc;
+  }
+  *out = e;
+  return CMLD_OK;
+}
+
+int32_t cmld_engine_named_count(const cmld_engine *e) { return e && e->lay ? (int32_t)e->lay->named.size() : 0; }
+
+int32_t cmld_engine_named_info(const cmld_engine *e, int32_t i, const char **name, int64_t *rows, int64_t *cols) {
+  if (!e || !e->lay || i < 0 || i >= (int32_t)e->lay->named.size() || !name || !rows || !cols) return fail(CMLD_ERR_INVALID, "named_info: bad argument");
+  const Named &n = e->lay->named[i];
+  *name = n.name.c_str();
+  *rows = n.rows;
+  *cols = n.cols;
+  return CMLD_OK;
+}
+
+int32_t cmld_engine_set_named(cmld_engine *e, const char *name, int32_t dtype, const void *data, uint64_t nbytes) {
+  CMLD_ENGINE_ENTER(e);
+  if (!e->lay) return fail(CMLD_ERR_UNSUPPORTED, "set_named: a llama-shaped engine takes its weights by layer");
+  if (!name || !data) return fail(CMLD_ERR_INVALID, "set_named: null argument");
+  Named *n = find_named(e, name);
+  if (!n) return fail(CMLD_ERR_INVALID, "set_named: this model has no tensor %s", name);
+  const int64_t rows = std::max<int64_t>(1, n->rows), count = rows * n->cols, es = dtype == CMLD_F32 ? 4 : 2;
+  if (dtype != CMLD_BF16 && dtype != CMLD_F32) return fail(CMLD_ERR_UNSUPPORTED, "set_named(%s): type %d", name, dtype);
+  if ((int64_t)nbytes != count * es)
+    return fail(CMLD_ERR_SHAPE, "set_named(%s): %lld x %lld values need %lld bytes, got %llu", name, (long long)rows, (long long)n->cols, (long long)(count * es),
+                (unsigned long long)nbytes);
+  if (n->m && dtype == CMLD_BF16) {
+    CMLD_CUDA(cudaMemcpy2DAsync(n->m, (size_t)n->ld * 2, data, (size_t)n->cols * 2, (size_t)n->cols * 2, (size_t)rows, cudaMemcpyDefault, e->stream));
+  } else if (n->m) {
+    return fail(CMLD_ERR_UNSUPPORTED, "set_named(%s): matrices are bfloat16", name);
+  } else if (dtype == CMLD_F32) {
+    CMLD_CUDA(cudaMemcpyAsync(n->v, data, (size_t)count * 4, cudaMemcpyDefault, e->stream));
+  } else {
+    std::vector<uint16_t> h(count);
+    CMLD_CUDA(cudaMemcpy(h.data(), data, (size_t)count * 2, cudaMemcpyDefault));
+    std::vector<uint32_t> f(count);
+    for (int64_t i = 0; i < count; ++i) f[i] = (uint32_t)h[i] << 16;
+    CMLD_CUDA(cudaMemcpyAsync(n->v, f.data(), (size_t)count * 4, cudaMemcpyHostToDevice, e->stream));
+  }
+  CMLD_CUDA(cudaStreamSynchronize(e->stream));
+  n->set = true;
+  return CMLD_OK;
+}
+
+int32_t cmld_engine_synth_named(cmld_engine *e, const char *name, uint64_t seed, uint64_t stream, float mean, float sigma) {
+  CMLD_ENGINE_ENTER(e);
+  if (!e->lay || !name) return fail(CMLD_ERR_INVALID, "synth_named: bad argument");
+  Named *n = find_named(e, name);
+  if (!n) return fail(CMLD_ERR_INVALID, "synth_named: this model has no tensor %s", name);
+  const int64_t rows = std::max<int64_t>(1, n->rows);
+  // 64 Mi values at a time through an f32 slab
+  const int64_t slab = std::max<int64_t>(1, std::min<int64_t>(rows, (64ll << 20) / n->cols));
+  Weight w;
+  CMLD_TRY(weight_alloc(w, CMLD_F32, slab, n->cols));
+  int32_t rc = CMLD_OK;
+  for (int64_t r0 = 0; r0 < rows && rc == CMLD_OK; r0 += slab) {
+    w.rows = std::min(slab, rows - r0);
+    rc = launch_synth(w, seed, stream, r0, sigma, e->stream);
+    if (rc != CMLD_OK) break;
+    named_from_f32_kernel<<<1024, 256, 0, e->stream>>>(reinterpret_cast<const float *>(w.data), w.rows, n->cols, n->m ? n->m + r0 * n->ld : nullptr, n->ld,
+                                                       n->v, mean);
+    if (cudaGetLastError() != cudaSuccess || cudaStreamSynchronize(e->stream) != cudaSuccess) rc = fail(CMLD_ERR_CUDA, "synth_named failed");
+  }
+  weight_free(w);
+  if (rc == CMLD_OK) n->set = true;
+  return rc;
+}
+
+int32_t cmld_engine_slot_filled(const cmld_engine *e, int32_t slot, int64_t *tokens) {
+  if (!e || !e->lay || !tokens) return fail(CMLD_ERR_INVALID, "slot_filled: bad argument");
+  if (slot < 0 || slot >= (int32_t)e->lay->filled.size()) return fail(CMLD_ERR_INVALID, "sequence slot %d out of range", slot);
+  *tokens = e->lay->filled[slot];
+  return CMLD_OK;
+}
+
+}  // extern "C"

@@ -1,0 +1,312 @@
+// Building blocks of layered models: designs described layer by layer (mixer type, sizes, feed-forward) instead of by
+// the one llama shape.  Weights are bfloat16 matrices; activations are bfloat16 or 32-bit, sums always 32-bit.
+// One launcher per mechanism, its sizes and constants as arguments; csrc/layered.cu strings them together.
+#pragma once
+
+#include <cuda_bf16.h>
+
+#include "common.cuh"
+
+namespace cmld {
+
+typedef __nv_bfloat16 bf16;
+
+// A bfloat16 matrix [rows][cols], row stride ld elements (a multiple of 8; the padding is zero).
+struct LinW {
+  const bf16 *w = nullptr;
+  int32_t rows = 0, cols = 0;
+  int64_t ld = 0;
+};
+inline int64_t lin_ld(int64_t cols) { return (cols + 7) & ~int64_t(7); }
+
+// Activation rows: bf16 (half = 1) or f32.
+struct ActBuf {
+  void *p = nullptr;
+  int32_t half = 0;
+  int64_t ld = 0;  // elements
+};
+
+// What a linear layer does to its sums: SiLU on output rows below act_rows, the square of ReLU on all, or nothing.
+enum LinAct { kActNone = 0, kActSilu = 1, kActRelu2 = 2 };
+
+// One boundary between two sublayers of a residual held as `streams` parallel copies (hyper-connections): the update of
+// the sublayer that has just produced y, then the read-out and layer norm that feed the next one.
+//   x'_t = sum_s mix[s][t] x_s + out[t] y;   u = sum_t in[t] x'_t (in == null: the plain sum);   result = LN(u)
+// embed != null: the first boundary instead: x' = LN_embed(embed[token]) in every stream.
+// All of it in 32-bit.
+struct StreamMix {
+  const float *x_in = nullptr;  // [row][streams][width]
+  float *x_out = nullptr;       // same layout, another buffer; null: the updated streams are not kept
+  const float *y = nullptr;     // [row][width]
+  const float *mix = nullptr, *out = nullptr, *in = nullptr;
+  const float *norm_w = nullptr, *norm_b = nullptr;  // null: no norm
+  float eps = 0.0f;
+  const bf16 *embed = nullptr;
+  int64_t embed_ld = 0;
+  const int32_t *tokens = nullptr;
+  const float *enorm_w = nullptr, *enorm_b = nullptr;
+  int32_t streams = 1, width = 0;
+  const int32_t *row_map = nullptr;  // result row r comes from row row_map[r]; null: r
+};
+
+// stream_mix.cu
+int32_t launch_stream_mix(const StreamMix &m, int32_t rows, ActBuf out, bool pdl, cudaStream_t s);
+// residual after a layer, [rows][width] f32: the sum of the updated streams
+int32_t launch_stream_tap(const StreamMix &m, int32_t rows, float *out, cudaStream_t s);
+// out[r] = x[r] / rms(x[r]) * w (* sigmoid(gate[r])), x f32 [rows][x_ld]; gate f32 or bf16
+int32_t launch_rms_rows(const float *x, int64_t x_ld, const float *w, int32_t cols, float eps, ActBuf gate, ActBuf out, int32_t rows,
+                        bool pdl, cudaStream_t s);
+
+// lin_mv.cu: up to two activation rows, one pass over the weights at HBM speed, with the operand's preparation fused
+// into the prologue of every CTA.
+enum LinPrologue { kProPlain = 0, kProRms = 1, kProRmsGate = 2, kProStreams = 3 };
+struct LinMvArgs {
+  LinW w;
+  int32_t batch = 1;
+  int32_t prologue = kProPlain;
+  StreamMix mix;              // kProStreams
+  const float *x = nullptr;   // the others: f32 rows
+  int64_t x_ld = 0;
+  const float *norm_w = nullptr;
+  float eps = 0.0f;
+  const float *gate = nullptr;  // kProRmsGate: f32 rows, multiplied by their sigmoid
+  int64_t gate_ld = 0;
+  float *y = nullptr;
+  int64_t y_ld = 0;
+  int32_t act = kActNone, act_rows = 0;
+};
+bool lin_mv_fits(int32_t cols, int32_t batch);
+int32_t launch_lin_mv(const LinMvArgs &a, bool pdl, cudaStream_t s);
+
+// lin_tc5.cu / lin_f32.cu: any number of rows.  out[r][o] = act(sum_k w[o][k] x[r][k])
+struct LinArgs {
+  LinW w;
+  const void *x = nullptr;  // bf16 rows (tcgen05) or f32 rows (f32 kernel), x_ld elements apart
+  int64_t x_ld = 0;
+  int32_t rows = 0;
+  void *out = nullptr;
+  int32_t out_half = 0;
+  int64_t out_ld = 0;
+  int32_t act = kActNone, act_rows = 0;
+};
+int32_t launch_lin_tc5(const LinArgs &a, int32_t sm_count, int32_t *status, bool pdl, cudaStream_t s);
+int32_t launch_lin_f32(const LinArgs &a, cudaStream_t s);
+
+// latent_attn.cu: attention over a cache of one latent vector and one shared rotated key part per position.
+struct LatentShape {
+  int32_t heads, dim, rot_dim, rot_dims, vdim, rank;
+  float scale, eps;
+};
+struct LatentArgs {
+  LatentShape m;
+  int32_t rows = 0;
+  const int32_t *positions = nullptr, *slots = nullptr;  // per row
+  const float *cs = nullptr;    // [position][rot_dims / 2][cos, sin]
+  void *cache = nullptr;        // [slot][max_pos][cache_ld]: latent | rotated key part
+  int32_t cache_half = 0;
+  int64_t cache_ld = 0, max_pos = 0;
+  const float *low = nullptr;   // [row][low_ld]: latent before its norm | key part before its rotation
+  int64_t low_ld = 0;
+  const float *latent_norm = nullptr;
+  const float *q = nullptr;     // [row][heads * (dim + rot_dim)]
+  LinW uk, uv;
+  float *qa = nullptr;          // [row][heads][rank + rot_dim]: queries in latent space, scaled
+  float *part = nullptr;        // [row][heads][splits][rank + 2]
+  int32_t splits = 1;
+  const float *gate = nullptr;  // [row][gate_ld]
+  int64_t gate_ld = 0;
+  ActBuf out;                   // [row][heads * vdim]
+};
+// Appends the rows' latents to the cache; with queries, also brings the queries into latent space.
+int32_t launch_latent_prep(const LatentArgs &a, bool queries, bool pdl, cudaStream_t s);
+int32_t launch_latent_attention(const LatentArgs &a, bool pdl, cudaStream_t s);
+int32_t launch_latent_output(const LatentArgs &a, bool pdl, cudaStream_t s);
+bool latent_shape_ok(const LatentShape &m);
+// A long portion of one sequence: keys and values already expanded to kv[position][heads * dim | heads * vdim] (bf16).
+struct LatentPrefillArgs {
+  LatentShape m;
+  int32_t rows = 0;
+  int64_t start = 0;            // position of row 0
+  const float *cs = nullptr;
+  const bf16 *cache = nullptr;  // this slot's cache rows, for the rotated key part
+  int64_t cache_ld = 0;
+  const bf16 *kv = nullptr;
+  int64_t kv_ld = 0;
+  const float *q = nullptr;
+  const float *gate = nullptr;
+  int64_t gate_ld = 0;
+  bf16 *out = nullptr;
+  int64_t out_ld = 0;
+};
+bool latent_prefill_fits(const LatentShape &m, int64_t cache_ld, int64_t kv_ld);
+int32_t launch_latent_prefill(const LatentPrefillArgs &a, bool pdl, cudaStream_t s);
+
+// lightning.cu: linear attention with a fixed decay per head, state [slot][heads][dim][vdim] in f32.
+struct LightningArgs {
+  int32_t heads, dim, vdim;
+  const float *powers = nullptr;   // [heads][kLightningChunk + 1]: decay^0, decay^1, ...
+  float *state = nullptr;
+  const void *qkv = nullptr;       // [row][ld]: q (heads x dim) | k (heads x dim) | v (heads x vdim), f32 or bf16
+  int32_t half = 0;
+  int64_t ld = 0;
+  float *out = nullptr;            // [row][heads * vdim]
+  const int32_t *positions = nullptr, *slots = nullptr;
+  int32_t rows = 0;
+  int32_t one_sequence = 0;        // 1: the rows are consecutive tokens of one sequence; 0: one token of each row's own
+};
+constexpr int kLightningChunk = 64;
+bool lightning_shape_ok(int32_t heads, int32_t dim, int32_t vdim);
+int32_t launch_lightning_steps(const LightningArgs &a, bool pdl, cudaStream_t s);   // token after token
+bool lightning_chunk_fits(const LightningArgs &a);
+int32_t launch_lightning_chunks(const LightningArgs &a, bool pdl, cudaStream_t s);  // 64 tokens at a time on the tensor cores
+
+#ifdef __CUDACC__
+
+template <typename... KA, typename... A>
+inline int32_t launch_kernel(void (*k)(KA...), dim3 grid, dim3 block, size_t smem, bool pdl, cudaStream_t s, A &&...args) {
+  cudaLaunchConfig_t cfg{};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = s;
+  cudaLaunchAttribute attr[1];
+  attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[0].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = pdl ? 1 : 0;
+  CMLD_CUDA(cudaLaunchKernelEx(&cfg, k, static_cast<KA>(args)...));
+  return CMLD_OK;
+}
+// Once per kernel: full shared memory.
+template <typename K>
+inline int32_t allow_smem(K k, size_t bytes) {
+  CMLD_CUDA(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes));
+  return CMLD_OK;
+}
+
+__device__ __forceinline__ void pdl_launch() { asm volatile("griddepcontrol.launch_dependents;"); }
+__device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float lin_activate(float v, int act, bool in_range) {
+  if (act == kActSilu && in_range) return v * sigmoid_f(v);
+  if (act == kActRelu2) {
+    const float p = fmaxf(v, 0.0f);
+    return p * p;
+  }
+  return v;
+}
+__device__ __forceinline__ float bf16_lo(uint32_t w) { return __uint_as_float(w << 16); }
+__device__ __forceinline__ float bf16_hi(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
+__device__ __forceinline__ float act_load(const void *p, int half, int64_t i) {
+  return half ? __bfloat162float(static_cast<const bf16 *>(p)[i]) : static_cast<const float *>(p)[i];
+}
+__device__ __forceinline__ void act_store(void *p, int half, int64_t i, float v) {
+  if (half) static_cast<bf16 *>(p)[i] = __float2bfloat16_rn(v);
+  else static_cast<float *>(p)[i] = v;
+}
+
+// Sum over the CTA; every thread gets it.  `red` holds at least blockDim.x / 32 floats.
+__device__ __forceinline__ float cta_total(float v, float *red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, n = (blockDim.x + 31) >> 5;
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) red[warp] = v;
+  __syncthreads();
+  float t = 0.0f;
+  for (int i = 0; i < n; ++i) t += red[i];
+  return t;
+}
+
+template <int S>
+__device__ __forceinline__ void stream_update(const StreamMix &m, int64_t row, float *u, bool store) {
+  float mix[S][S], out[S], in[S];
+#pragma unroll
+  for (int s = 0; s < S; ++s) {
+    const bool live = s < m.streams;
+    out[s] = live ? m.out[s] : 0.0f;
+    in[s] = live ? (m.in ? m.in[s] : 1.0f) : 0.0f;
+#pragma unroll
+    for (int t = 0; t < S; ++t) mix[s][t] = live && t < m.streams ? m.mix[s * m.streams + t] : 0.0f;
+  }
+  const float *x = m.x_in + row * m.streams * m.width, *y = m.y + row * m.width;
+  float *xo = m.x_out ? m.x_out + row * m.streams * m.width : nullptr;
+  for (int i = threadIdx.x; i < m.width; i += blockDim.x) {
+    float xs[S];
+#pragma unroll
+    for (int s = 0; s < S; ++s) xs[s] = s < m.streams ? x[(int64_t)s * m.width + i] : 0.0f;
+    const float yi = y[i];
+    float acc = 0.0f;
+#pragma unroll
+    for (int t = 0; t < S; ++t) {
+      float v = out[t] * yi;
+#pragma unroll
+      for (int s = 0; s < S; ++s) v = fmaf(mix[s][t], xs[s], v);
+      if (store && xo && t < m.streams) xo[(int64_t)t * m.width + i] = v;
+      acc = fmaf(in[t], v, acc);
+    }
+    u[i] = acc;
+  }
+}
+
+// Any number of streams: one updated stream at a time.
+__device__ __forceinline__ void stream_update_many(const StreamMix &m, int64_t row, float *u, bool store) {
+  const float *x = m.x_in + row * m.streams * m.width, *y = m.y + row * m.width;
+  float *xo = store && m.x_out ? m.x_out + row * m.streams * m.width : nullptr;
+  for (int i = threadIdx.x; i < m.width; i += blockDim.x) {
+    const float yi = y[i];
+    float acc = 0.0f;
+    for (int t = 0; t < m.streams; ++t) {
+      float v = m.out[t] * yi;
+      for (int s = 0; s < m.streams; ++s) v = fmaf(m.mix[s * m.streams + t], x[(int64_t)s * m.width + i], v);
+      if (xo) xo[(int64_t)t * m.width + i] = v;
+      acc = fmaf(m.in ? m.in[t] : 1.0f, v, acc);
+    }
+    u[i] = acc;
+  }
+}
+
+// (u - mean) / sqrt(var + eps) * w + b in place over the CTA (u in shared memory).
+__device__ __forceinline__ void layer_norm_cta(float *u, int n, const float *w, const float *b, float eps, float *red) {
+  float s = 0.0f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) s += u[i];
+  const float mean = cta_total(s, red) / (float)n;
+  s = 0.0f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) {
+    const float d = u[i] - mean;
+    s = fmaf(d, d, s);
+  }
+  const float r = 1.0f / sqrtf(cta_total(s, red) / (float)n + eps);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) u[i] = (u[i] - mean) * r * w[i] + b[i];
+}
+
+// The whole boundary for one row; the result is left in u[width] (shared memory; each thread holds its own stride).
+__device__ __forceinline__ void stream_mix_row(const StreamMix &m, int r, float *u, float *red, bool store) {
+  const int64_t row = m.row_map ? m.row_map[r] : r;
+  if (m.embed) {
+    const bf16 *e = m.embed + (int64_t)m.tokens[row] * m.embed_ld;
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = __bfloat162float(e[i]);
+    layer_norm_cta(u, m.width, m.enorm_w, m.enorm_b, m.eps, red);
+    float in = 0.0f;
+    for (int s = 0; s < m.streams; ++s) in += m.in ? m.in[s] : 1.0f;
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) {
+      const float x = u[i];
+      if (store && m.x_out)
+        for (int s = 0; s < m.streams; ++s) m.x_out[(row * m.streams + s) * m.width + i] = x;
+      u[i] = in * x;
+    }
+  } else {
+    switch (m.streams) {
+      case 1: stream_update<1>(m, row, u, store); break;
+      case 2: stream_update<2>(m, row, u, store); break;
+      case 3: stream_update<3>(m, row, u, store); break;
+      case 4: stream_update<4>(m, row, u, store); break;
+      default: stream_update_many(m, row, u, store); break;
+    }
+  }
+  if (m.norm_w) layer_norm_cta(u, m.width, m.norm_w, m.norm_b, m.eps, red);
+}
+
+#endif  // __CUDACC__
+
+}  // namespace cmld

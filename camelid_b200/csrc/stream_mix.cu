@@ -1,0 +1,64 @@
+// Row operations of layered models: the hyper-connection boundary (stream update, read-out, layer norm), the embedding
+// with its norm, RMS norm with an optional gate.
+#include "layered.cuh"
+
+namespace cmld {
+
+namespace {
+
+constexpr int kMixThreads = 256;
+
+__global__ void __launch_bounds__(kMixThreads) stream_mix_kernel(const StreamMix m, ActBuf out) {
+  extern __shared__ float u[];
+  __shared__ float red[kMixThreads / 32];
+  pdl_launch();
+  pdl_wait();
+  const int r = blockIdx.x;
+  stream_mix_row(m, r, u, red, true);
+  for (int i = threadIdx.x; i < m.width; i += blockDim.x) act_store(out.p, out.half, r * out.ld + i, u[i]);
+}
+
+__global__ void __launch_bounds__(kMixThreads) stream_tap_kernel(const StreamMix m, float *out) {
+  extern __shared__ float u[];
+  __shared__ float red[kMixThreads / 32];
+  pdl_wait();
+  stream_mix_row(m, blockIdx.x, u, red, false);
+  for (int i = threadIdx.x; i < m.width; i += blockDim.x) out[(int64_t)blockIdx.x * m.width + i] = u[i];
+}
+
+__global__ void __launch_bounds__(kMixThreads) rms_rows_kernel(const float *x, int64_t x_ld, const float *w, int cols, float eps, ActBuf gate, ActBuf out) {
+  __shared__ float red[kMixThreads / 32];
+  pdl_launch();
+  pdl_wait();
+  const int64_t r = blockIdx.x;
+  const float *xr = x + r * x_ld;
+  float s = 0.0f;
+  for (int i = threadIdx.x; i < cols; i += blockDim.x) s = fmaf(xr[i], xr[i], s);
+  const float inv = 1.0f / sqrtf(cta_total(s, red) / (float)cols + eps);
+  for (int i = threadIdx.x; i < cols; i += blockDim.x) {
+    float v = xr[i] * inv * w[i];
+    if (gate.p) v *= sigmoid_f(act_load(gate.p, gate.half, r * gate.ld + i));
+    act_store(out.p, out.half, r * out.ld + i, v);
+  }
+}
+
+}  // namespace
+
+int32_t launch_stream_mix(const StreamMix &m, int32_t rows, ActBuf out, bool pdl, cudaStream_t s) {
+  const size_t smem = (size_t)m.width * 4;
+  if (smem > 48 * 1024) CMLD_TRY(allow_smem(stream_mix_kernel, smem));
+  return launch_kernel(stream_mix_kernel, dim3(rows), dim3(kMixThreads), smem, pdl, s, m, out);
+}
+
+int32_t launch_stream_tap(const StreamMix &m, int32_t rows, float *out, cudaStream_t s) {
+  const size_t smem = (size_t)m.width * 4;
+  if (smem > 48 * 1024) CMLD_TRY(allow_smem(stream_tap_kernel, smem));
+  return launch_kernel(stream_tap_kernel, dim3(rows), dim3(kMixThreads), smem, false, s, m, out);
+}
+
+int32_t launch_rms_rows(const float *x, int64_t x_ld, const float *w, int32_t cols, float eps, ActBuf gate, ActBuf out, int32_t rows,
+                        bool pdl, cudaStream_t s) {
+  return launch_kernel(rms_rows_kernel, dim3(rows), dim3(kMixThreads), 0, pdl, s, x, x_ld, w, cols, eps, gate, out);
+}
+
+}  // namespace cmld

@@ -16,7 +16,7 @@ import numpy as np
 
 from ._lib import Config, Tensor, check, lib
 
-F32, Q8_0, Q4_K, Q6_K, Q8_0_HOST36 = 0, 8, 12, 14, 108
+F32, Q8_0, Q4_K, Q6_K, BF16, Q8_0_HOST36 = 0, 8, 12, 14, 30, 108
 ACT_Q8_0, ACT_Q8_K = 1, 2
 QT_NAMES = {"F32": F32, "Q8_0": Q8_0, "Q4_K": Q4_K, "Q6_K": Q6_K}
 PROJ_NAMES = ("q", "k", "v", "o", "gate", "up", "down")
@@ -196,7 +196,86 @@ class EngineConfig:
         return d
 
 
-class ResidentDecode:
+class TokenEngine:
+    """What every engine answers, whatever its design: sequences in slots, driven by token ids."""
+
+    _h = None
+    cfg = None  # has vocab, hidden, max_pos, max_seqs
+
+    def close(self):
+        if getattr(self, "_h", None):
+            lib().cmld_engine_destroy(self._h)
+            self._h = None
+
+    def __del__(self):
+        try:
+            self.close()
+        except Exception:
+            pass
+
+    def weights_ready(self) -> bool:
+        return bool(lib().cmld_engine_weights_ready(self._h))
+
+    def max_pos(self) -> int:
+        return int(lib().cmld_engine_max_pos(self._h))
+
+    def n_layers(self) -> int:
+        return int(lib().cmld_engine_n_layers(self._h))
+
+    def extend(self, seq: int, tokens, start_pos: int, want=(), taps: int = 0):
+        """Feeds a portion of a sequence.  Returns (greedy token after it, logits [len(want), vocab] at the places
+        `want` of the portion); with ``taps`` = the number of layer runs also the residual stream after each of them,
+        [taps, len(tokens), width] (layered designs)."""
+        t = np.ascontiguousarray(tokens, np.int32)
+        w = np.ascontiguousarray(want, np.int32)
+        logits = np.empty((w.size, self.cfg.vocab), np.float32)
+        stream = np.empty((taps, t.size, self.cfg.hidden), np.float32) if taps else None
+        nxt = C.c_uint32(0)
+        check(lib().cmld_engine_extend(self._h, seq, _np_ptr(t), t.size, start_pos, _np_ptr(w), w.size, _np_ptr(logits),
+                                       _np_ptr(stream) if taps else None, C.byref(nxt)))
+        return (int(nxt.value), logits, stream) if taps else (int(nxt.value), logits)
+
+    def sample(self, temperature: float, seed: int, min_p: float = 0.0, row: int = -1):
+        """Draws from logits the engine still holds (row of the last step_batch; -1: the last token of the last call).
+        None when the min-p filter cannot decide on the device."""
+        tok = C.c_uint32(0)
+        check(lib().cmld_engine_sample_row(self._h, row, temperature, min_p, seed, C.byref(tok)))
+        return None if tok.value == 0xFFFFFFFF else int(tok.value)
+
+    def prefill_tokens(self, seq: int, tokens, start_pos: int = 0) -> int:
+        t = np.ascontiguousarray(tokens, np.int32)
+        nxt = C.c_uint32(0)
+        check(lib().cmld_engine_prefill_tokens(self._h, seq, _np_ptr(t), t.size, start_pos, C.byref(nxt)))
+        return int(nxt.value)
+
+    def decode_greedy(self, seqs, tokens_in, positions, n_steps: int) -> np.ndarray:
+        s = np.ascontiguousarray(seqs, np.int32)
+        t = np.ascontiguousarray(tokens_in, np.int32)
+        p = np.ascontiguousarray(positions, np.int64)
+        out = np.empty((n_steps, s.size), np.uint32)
+        check(lib().cmld_engine_decode_greedy(self._h, s.size, _np_ptr(s), _np_ptr(t), _np_ptr(p), n_steps, _np_ptr(out)))
+        return out
+
+    def step_batch(self, seqs, tokens_in, positions, want_logits=False, want_hidden=False):
+        s = np.ascontiguousarray(seqs, np.int32)
+        t = np.ascontiguousarray(tokens_in, np.int32)
+        p = np.ascontiguousarray(positions, np.int64)
+        toks = np.empty(s.size, np.uint32)
+        logits = np.empty((s.size, self.cfg.vocab), np.float32) if want_logits else None
+        hidden = np.empty((s.size, self.cfg.hidden), np.float32) if want_hidden else None
+        check(lib().cmld_engine_step_batch(self._h, s.size, _np_ptr(s), _np_ptr(t), _np_ptr(p), _np_ptr(toks),
+                                           _np_ptr(logits) if want_logits else None,
+                                           _np_ptr(hidden) if want_hidden else None))
+        return toks, logits, hidden
+
+    def last_timing(self):
+        ms = C.c_float(0)
+        n = C.c_int64(0)
+        check(lib().cmld_engine_last_timing(self._h, C.byref(ms), C.byref(n)))
+        return float(ms.value), int(n.value)
+
+
+class ResidentDecode(TokenEngine):
     """CudaResidentDecode (src/cuda_resident.rs:15093) over the C ABI."""
 
     def __init__(self, cfg: EngineConfig):
@@ -205,11 +284,6 @@ class ResidentDecode:
         c = cfg.to_c()
         check(lib().cmld_engine_create(C.byref(c), C.byref(h)))
         self._h = h.value
-
-    def close(self):
-        if getattr(self, "_h", None):
-            lib().cmld_engine_destroy(self._h)
-            self._h = None
 
     # -- sharded engines ---------------------------------------------------------
     @staticmethod
@@ -223,12 +297,6 @@ class ResidentDecode:
         """Collective over the ranks of the tensor- or expert-parallel group."""
         buf = (C.c_uint8 * 128).from_buffer_copy(unique_id)
         check(lib().cmld_engine_comm_init(self._h, buf, rank, world))
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
 
     # -- weights ---------------------------------------------------------------
     def set_layer(self, layer: int, projs: dict, attn_norm, ffn_norm):
@@ -292,20 +360,11 @@ class ResidentDecode:
         token_embd._h = None
 
     # -- bookkeeping -----------------------------------------------------------
-    def weights_ready(self) -> bool:
-        return bool(lib().cmld_engine_weights_ready(self._h))
-
     def filled(self) -> int:
         return int(lib().cmld_engine_filled(self._h))
 
     def set_filled(self, n: int):
         check(lib().cmld_engine_set_filled(self._h, n))
-
-    def max_pos(self) -> int:
-        return int(lib().cmld_engine_max_pos(self._h))
-
-    def n_layers(self) -> int:
-        return int(lib().cmld_engine_n_layers(self._h))
 
     # -- forward_token family ----------------------------------------------------
     def _f(self, a):
@@ -407,36 +466,3 @@ class ResidentDecode:
         ck, cv = np.empty(shape, np.float32), np.empty(shape, np.float32)
         check(lib().cmld_engine_read_kv_layer(self._h, layer, n_positions, _np_ptr(ck), _np_ptr(cv)))
         return ck, cv
-
-    # -- token-id driven ---------------------------------------------------------
-    def prefill_tokens(self, seq: int, tokens, start_pos: int = 0) -> int:
-        t = np.ascontiguousarray(tokens, np.int32)
-        nxt = C.c_uint32(0)
-        check(lib().cmld_engine_prefill_tokens(self._h, seq, _np_ptr(t), t.size, start_pos, C.byref(nxt)))
-        return int(nxt.value)
-
-    def decode_greedy(self, seqs, tokens_in, positions, n_steps: int) -> np.ndarray:
-        s = np.ascontiguousarray(seqs, np.int32)
-        t = np.ascontiguousarray(tokens_in, np.int32)
-        p = np.ascontiguousarray(positions, np.int64)
-        out = np.empty((n_steps, s.size), np.uint32)
-        check(lib().cmld_engine_decode_greedy(self._h, s.size, _np_ptr(s), _np_ptr(t), _np_ptr(p), n_steps, _np_ptr(out)))
-        return out
-
-    def step_batch(self, seqs, tokens_in, positions, want_logits=False, want_hidden=False):
-        s = np.ascontiguousarray(seqs, np.int32)
-        t = np.ascontiguousarray(tokens_in, np.int32)
-        p = np.ascontiguousarray(positions, np.int64)
-        toks = np.empty(s.size, np.uint32)
-        logits = np.empty((s.size, self.cfg.vocab), np.float32) if want_logits else None
-        hidden = np.empty((s.size, self.cfg.hidden), np.float32) if want_hidden else None
-        check(lib().cmld_engine_step_batch(self._h, s.size, _np_ptr(s), _np_ptr(t), _np_ptr(p), _np_ptr(toks),
-                                           _np_ptr(logits) if want_logits else None,
-                                           _np_ptr(hidden) if want_hidden else None))
-        return toks, logits, hidden
-
-    def last_timing(self):
-        ms = C.c_float(0)
-        n = C.c_int64(0)
-        check(lib().cmld_engine_last_timing(self._h, C.byref(ms), C.byref(n)))
-        return float(ms.value), int(n.value)

@@ -43,6 +43,7 @@ typedef enum {
   CMLD_Q8_0 = 8,          /* 34-byte wire blocks: f16 d + 32 x i8 */
   CMLD_Q4_K = 12,         /* 144-byte superblocks */
   CMLD_Q6_K = 14,         /* 210-byte superblocks */
+  CMLD_BF16 = 30,         /* layered designs' matrices (cmld_engine_set_named) */
   CMLD_Q8_0_HOST36 = 108  /* Camelid's host block {f32 scale; i8[32]} (src/tensor/mod.rs:105-118),
                              what q8_0_raw_bytes hands to set_layer (src/inference.rs:16387) */
 } cmld_qtype;
@@ -233,6 +234,49 @@ CMLD_API int32_t cmld_engine_seed_layer(cmld_engine *e, int32_t layer, const flo
 CMLD_API int32_t cmld_engine_read_kv_layer(cmld_engine *e, int32_t layer, int64_t n_positions, float *ck_out,
                                            float *cv_out);
 
+/* ---- layered designs: models described layer by layer (no counterpart in the reference) ----
+ *
+ * An engine made by cmld_engine_create_layered answers the token-driven calls below (prefill_tokens, extend,
+ * decode_greedy, step_batch without hidden_out, sample_row, last_timing) and weights_ready / max_pos / n_layers;
+ * the calls that speak of llama-shaped layers return CMLD_ERR_UNSUPPORTED.
+ *
+ * The residual is held as `streams` parallel copies x_s.  For each sublayer, with its vectors in, out and matrix mix:
+ *   u = sum_s in[s] x_s;  y = sublayer(layernorm(u));  x_t <- sum_s mix[s][t] x_s + out[t] y.
+ * Layers loop_start .. loop_stop-1 run loop_times times in a row with the same weights, each pass with its own cache
+ * or state.  A sequence slot holds rows and states that belong together: a call either starts a sequence (position 0) or
+ * continues it where it ends (cmld_engine_slot_filled). */
+typedef enum {
+  CMLD_LAYER_LATENT = 1,    /* attention over a cached latent and a rotated key part shared by the heads */
+  CMLD_LAYER_LIGHTNING = 2  /* linear attention with a fixed decay per head, RMS-normed and gated */
+} cmld_layer_type;
+typedef struct {
+  int32_t type;
+  int32_t heads, dim, vdim;
+  int32_t q_rank, kv_rank, rot_dim, rot_dims; /* latent: rot_dims of the rot_dim values turn, in pairs (2i, 2i + 1) */
+  int32_t ff;                                 /* width of the squared-ReLU feed-forward; 0 = none */
+  float scale;                                /* latent: factor of the scores */
+  double rot_base;                            /* latent: pair i turns by position * rot_base^(-2i / rot_dims) */
+  const float *decay;                         /* lightning: [heads]; borrowed for the duration of the call */
+} cmld_layer_desc;
+typedef struct {
+  int32_t n_layers, loop_start, loop_stop, loop_times; /* loop_times 0 or 1: every layer once */
+  int32_t streams, width, vocab, max_pos, max_seqs;
+  int32_t dtype;  /* CMLD_BF16: bfloat16 products with 32-bit sums, residual, norms, scores and states; CMLD_F32: all 32-bit */
+  int32_t device, flags;
+  float eps;
+  const cmld_layer_desc *layers;
+} cmld_layered_config;
+CMLD_API int32_t cmld_engine_create_layered(const cmld_layered_config *cfg, cmld_engine **out);
+/* The tensors the model needs, by name: matrices [rows][cols] (bfloat16), or rows == 0: vectors of cols values. */
+CMLD_API int32_t cmld_engine_named_count(const cmld_engine *e);
+CMLD_API int32_t cmld_engine_named_info(const cmld_engine *e, int32_t i, const char **name, int64_t *rows, int64_t *cols);
+/* Values in host or device memory, row-major without padding; dtype CMLD_BF16, or CMLD_F32 for vectors. */
+CMLD_API int32_t cmld_engine_set_named(cmld_engine *e, const char *name, int32_t dtype, const void *data, uint64_t nbytes);
+/* Seeded values mean + N(0, sigma), made on the device and rounded to bfloat16 (benchmarks, tests). */
+CMLD_API int32_t cmld_engine_synth_named(cmld_engine *e, const char *name, uint64_t seed, uint64_t stream, float mean, float sigma);
+/* Tokens the sequence in `slot` holds; -1 after a call on it failed half-way (start again at position 0). */
+CMLD_API int32_t cmld_engine_slot_filled(const cmld_engine *e, int32_t slot, int64_t *tokens);
+
 /* ---- on-device token loop (forward_token_device, src/cuda_resident.rs:19671-19834, there
  * for one architecture only; here for all).  Needs cmld_engine_set_token_embd. ---- */
 
@@ -254,6 +298,18 @@ CMLD_API int32_t cmld_engine_decode_greedy(cmld_engine *e, int32_t n_seqs, const
 CMLD_API int32_t cmld_engine_step_batch(cmld_engine *e, int32_t n_seqs, const int32_t *seqs,
                                         const int32_t *tokens_in, const int64_t *positions,
                                         uint32_t *tokens_out, float *logits_out, float *hidden_out);
+/* Feeds `n` tokens of sequence slot `seq` at positions start_pos.. (a portion of a prompt, or one token) and returns
+ * the logits at chosen places: want[n_want] are rising indices into `tokens`, logits_out[n_want][vocab]; either may be
+ * empty.  *next_token_out (may be NULL) = the greedy id after the last token.  taps_out (layered designs only, may be
+ * NULL): [layer runs][n][width], the residual stream (sum of the streams) after every layer run.
+ * cmld_engine_prefill_tokens is this call without places. */
+CMLD_API int32_t cmld_engine_extend(cmld_engine *e, int32_t seq, const int32_t *tokens, int64_t n, int64_t start_pos,
+                                    const int32_t *want, int32_t n_want, float *logits_out, float *taps_out,
+                                    uint32_t *next_token_out);
+/* Draws a token from logits the engine still holds: row `row` of the last step_batch, or (row < 0) the row of the last
+ * token of the last call.  Temperature, min_p and the 0xffffffff answer as in cmld_engine_forward_token_sample. */
+CMLD_API int32_t cmld_engine_sample_row(cmld_engine *e, int32_t row, float temperature, float min_p, uint64_t seed,
+                                        uint32_t *token_out);
 /* Device time of the last decode_greedy / step_batch call, from CUDA events on the engine's
  * stream (milliseconds), and the number of kernel launches it made. */
 CMLD_API int32_t cmld_engine_last_timing(const cmld_engine *e, float *ms_out, int64_t *launches_out);
