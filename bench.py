@@ -558,6 +558,74 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
+def design_case(eng, vocab, batch, n_prompt, steps, warmup, local_rank):
+    """Prompts one after the other, then greedy decode of all of them: device times (CUDA events in the engine)."""
+    first, prefill_ms = [], []
+    for s in range(batch):
+        first.append(eng.prefill_tokens(s, prompt_tokens(vocab, n_prompt, s), 0))
+        prefill_ms.append(eng.last_timing()[0])
+    if batch == 1:  # warm: the same prompt again into the same slot
+        for _ in range(3):
+            eng.prefill_tokens(0, prompt_tokens(vocab, n_prompt, 0), 0)
+            prefill_ms.append(eng.last_timing()[0])
+    prefill_ms = prefill_ms[-3:]
+    seqs, pos = list(range(batch)), [n_prompt] * batch
+    w = eng.decode_greedy(seqs, first, pos, max(3, warmup))
+    pos = [p + w.shape[0] for p in pos]
+    sampler = clock_sampler(local_rank)
+    sampler.start()
+    eng.decode_greedy(seqs, [int(t) for t in w[-1]], pos, steps)
+    ms, launches = eng.last_timing()
+    return {"batch": batch, "prompt_tokens": n_prompt, "steps": steps, "ms_per_step": ms / steps, "decode_tokens_per_s": batch * steps / (ms * 1e-3),
+            "launches_per_step": launches / steps, "prefill_ms": min(prefill_ms), "prefill_tokens_per_s": n_prompt / (min(prefill_ms) * 1e-3),
+            "context": pos[0] + steps / 2, "clocks": sampler.stop()}
+
+
+def run_design(args):
+    """--design losarax: the layered design at several sizes beside the llama shape of equal width, depth, feed-forward width
+    and vocabulary (Q4_K_M, this library's closest model).  Weights are random; one JSON line."""
+    import camelid_b200 as cm
+    from camelid_b200 import synth
+
+    if cm.device_count() < 1:
+        raise SystemExit("bench.py needs a CUDA device: the engine has no CPU path")
+    hbm, kind = measured_peaks()
+    p = ROOT / "MEASURED_PEAKS.json"
+    tflops = float(json.loads(p.read_text())["bf16_tflops"]) if p.exists() else 1590.0
+    rows = []
+    n_prompt = args.prompt or 1024
+    steps, warmup = args.steps, max(3, args.warmup)
+    shapes = [s for s in (args.design_shapes or "losarax-2k,losarax-4k").split(",") if s]
+    for shape in shapes:
+        peer = synth.LOSARAX_PEER[shape]
+        for batch in [int(b) for b in args.design_batches.split(",")]:
+            spec = synth.losarax_spec(shape, args.design_layers or None)
+            ctx = n_prompt + steps + warmup + 8
+            eng = synth.build_layered(spec, SEED, ctx, batch)
+            r = design_case(eng, spec.vocab, batch, n_prompt, steps, warmup, 0)
+            wb = synth.layered_bytes(eng)
+            by = wb + synth.layered_context_bytes(eng, r["context"], batch)
+            flops = wb * n_prompt  # two per bfloat16 weight; the head runs for one row
+            flops -= 2 * (n_prompt - 1) * spec.vocab * spec.width
+            r.update(model=shape, layers=len(spec.layers), dtype="bf16", weight_bytes=wb, decode_frac_of_hbm=by / (r["ms_per_step"] * 1e-3) / 1e9 / hbm,
+                     prefill_linear_tflops=flops / (r["prefill_ms"] * 1e-3) / 1e12, prefill_frac_of_bf16=flops / (r["prefill_ms"] * 1e-3) / 1e12 / tflops)
+            rows.append(r)
+            eng.close()
+            cfg = synth.engine_config(peer, max_pos=ctx, max_seqs=batch, n_layers=len(spec.layers))
+            eng = synth.build_engine(cfg, "q4_k_m", SEED)
+            r = design_case(eng, cfg.vocab, batch, n_prompt, steps, warmup, 0)
+            wb = synth.weight_bytes_per_token(cfg, "q4_k_m")
+            by = wb + batch * synth.kv_bytes_per_position(cfg) * r["context"]
+            sh = synth.proj_shapes(cfg)
+            flops = 2 * n_prompt * cfg.n_layers * sum(a * b for a, b in sh.values())
+            r.update(model=peer, layers=cfg.n_layers, dtype="q4_k_m", weight_bytes=wb, decode_frac_of_hbm=by / (r["ms_per_step"] * 1e-3) / 1e9 / hbm,
+                     prefill_linear_tflops=flops / (r["prefill_ms"] * 1e-3) / 1e12, prefill_frac_of_bf16=flops / (r["prefill_ms"] * 1e-3) / 1e12 / tflops)
+            rows.append(r)
+            eng.close()
+    print(json.dumps({"design": args.design, "steps": steps, "warmup": warmup, "data": "synthetic (random weights)", "hbm_gbs": hbm, "bf16_tflops": tflops,
+                      "peak_kind": kind, "l2": "inputs larger than L2: every step streams the model's weights from HBM", "results": rows}), flush=True)
+
+
 def run_e2e(cm, eng, cfg, synth, mix, cur, pos, device_tokens, n_steps):
     """K steps through cmld_engine_forward_token with host buffers, timed on the host clock
     (each call ends with the device-to-host read of the token)."""
@@ -600,6 +668,11 @@ def main():
                     help="profiling runs only: start decoding at the prompt length over an all-zero KV cache instead of ingesting a prompt")
     ap.add_argument("--prompt", type=int, default=0, help="override the workload's prompt length (profiling runs)")
     ap.add_argument("--engine-flags", type=int, default=0, help="CMLD_FLAG_* bits: 1 no CUDA graph, 2 direct-load matvec, 4 no PDL, 8 separate prep kernels, 16 plain reference-order kernels, 32 NCCL-only sums, 64 tensor-core matvec from 5 rows, 128 lane-parallel f32 sums")
+    ap.add_argument("--design", default="", choices=["", "losarax"],
+                    help="measure a layered design at --design-shapes beside the llama shapes of equal size, instead of the workload")
+    ap.add_argument("--design-shapes", default="", help="comma-separated names from synth.LOSARAX_SHAPES")
+    ap.add_argument("--design-layers", type=int, default=0, help="layers instead of the shape's own number (profiling runs)")
+    ap.add_argument("--design-batches", default="1,32")
     ap.add_argument("--watchdog", type=int, default=-1,
                     help="seconds after which a stuck run dumps its Python stacks and exits (default: 1500 when N > 1, off at N = 1)")
     args = ap.parse_args()
@@ -610,6 +683,8 @@ def main():
         faulthandler.dump_traceback_later(wd, exit=True)  # a rank waiting for a peer that died must not wait for ever
     if args.impl == "reference":
         run_reference(args)
+    elif args.design:
+        run_design(args)
     else:
         run_ours(args)
 

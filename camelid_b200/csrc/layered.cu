@@ -829,6 +829,86 @@ int32_t cmld_engine_synth_named(cmld_engine *e, const char *name, uint64_t seed,
   return rc;
 }
 
+int32_t cmld_linear(int32_t kernel, const void *w_dev, int64_t rows, int64_t cols, const void *x_dev, int32_t n, void *out_dev, int32_t out_bf16,
+                    int32_t act, int32_t act_rows, int32_t n_copies, int32_t iters, float *ms_out) {
+  if (!w_dev || !x_dev || !out_dev || rows < 1 || cols < 1 || n < 1) return fail(CMLD_ERR_INVALID, "linear: bad argument");
+  if (kernel < 0 || kernel > 2 || (kernel == 0 && (out_bf16 || !lin_mv_fits((int32_t)cols, n)))) return fail(CMLD_ERR_SHAPE, "linear: the kernel does not take this");
+  cudaStream_t s = nullptr;
+  int32_t *status = nullptr;
+  CMLD_CUDA(cudaStreamCreateWithFlags(&s, cudaStreamNonBlocking));
+  int32_t rc = CMLD_OK;
+  cudaGraph_t graph = nullptr;
+  cudaGraphExec_t exec = nullptr;
+  cudaEvent_t e0 = nullptr, e1 = nullptr;
+  auto cuda = [&](cudaError_t ce) {
+    if (rc == CMLD_OK && ce != cudaSuccess) rc = fail(CMLD_ERR_CUDA, "linear: %s", cudaGetErrorString(ce));
+  };
+  cuda(cudaMalloc(&status, 4));
+  if (rc == CMLD_OK) cuda(cudaMemsetAsync(status, 0, 4, s));
+  int sms = 148, dev = 0;
+  cudaGetDevice(&dev);
+  cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+  auto once = [&](int i, bool pdl) -> int32_t {
+    const int64_t ld = lin_ld(cols);
+    const LinW w{static_cast<const bf16 *>(w_dev) + (int64_t)(i % std::max(1, n_copies)) * rows * ld, (int32_t)rows, (int32_t)cols, ld};
+    if (kernel == 0) {
+      LinMvArgs a{};
+      a.w = w;
+      a.batch = n;
+      a.x = static_cast<const float *>(x_dev);
+      a.x_ld = ld;
+      a.y = static_cast<float *>(out_dev);
+      a.y_ld = rows;
+      a.act = act;
+      a.act_rows = act_rows;
+      return launch_lin_mv(a, pdl, s);
+    }
+    LinArgs a{};
+    a.w = w;
+    a.x = x_dev;
+    a.x_ld = ld;
+    a.rows = n;
+    a.out = out_dev;
+    a.out_half = out_bf16;
+    a.out_ld = rows;
+    a.act = act;
+    a.act_rows = act_rows;
+    return kernel == 1 ? launch_lin_tc5(a, sms, status, pdl, s) : launch_lin_f32(a, s);
+  };
+  if (rc == CMLD_OK) rc = once(0, false);
+  if (rc == CMLD_OK && iters > 0) {
+    cuda(cudaEventCreate(&e0));
+    cuda(cudaEventCreate(&e1));
+    for (int i = 0; i < 3 && rc == CMLD_OK; ++i) rc = once(i, true);
+    cuda(cudaStreamBeginCapture(s, cudaStreamCaptureModeThreadLocal));
+    for (int i = 0; i < iters && rc == CMLD_OK; ++i) rc = once(i, true);
+    cuda(cudaStreamEndCapture(s, &graph));
+    if (rc == CMLD_OK) cuda(cudaGraphInstantiate(&exec, graph, 0));
+    for (int i = 0; i < 2 && rc == CMLD_OK; ++i) {  // the first replay warms up
+      cuda(cudaEventRecord(e0, s));
+      cuda(cudaGraphLaunch(exec, s));
+      cuda(cudaEventRecord(e1, s));
+      cuda(cudaStreamSynchronize(s));
+    }
+    float ms = 0.0f;
+    if (rc == CMLD_OK) cuda(cudaEventElapsedTime(&ms, e0, e1));
+    if (ms_out) *ms_out = ms / (float)iters;
+  }
+  int32_t st = 0;
+  if (rc == CMLD_OK) {
+    cuda(cudaMemcpyAsync(&st, status, 4, cudaMemcpyDeviceToHost, s));
+    cuda(cudaStreamSynchronize(s));
+    if (rc == CMLD_OK && st != 0) rc = fail(st, "linear: a bounded device-side wait gave up");
+  }
+  if (exec) cudaGraphExecDestroy(exec);
+  if (graph) cudaGraphDestroy(graph);
+  if (e0) cudaEventDestroy(e0);
+  if (e1) cudaEventDestroy(e1);
+  cudaFree(status);
+  cudaStreamDestroy(s);
+  return rc;
+}
+
 int32_t cmld_engine_slot_filled(const cmld_engine *e, int32_t slot, int64_t *tokens) {
   if (!e || !e->lay || !tokens) return fail(CMLD_ERR_INVALID, "slot_filled: bad argument");
   if (slot < 0 || slot >= (int32_t)e->lay->filled.size()) return fail(CMLD_ERR_INVALID, "sequence slot %d out of range", slot);

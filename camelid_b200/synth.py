@@ -124,6 +124,77 @@ def build_engine(cfg: EngineConfig, mix: str, seed: int, tap=None, sigma: float 
     return eng
 
 
+# ---------------------------------------------------------------- layered designs
+
+LOSARAX_SHAPES = {
+    # name: (width, layers, heads, dim, vdim, q_rank, kv_rank, rot_dim, ff, vocab, streams); layers alternate latent
+    # attention (with a feed-forward) and lightning attention (every other one with a feed-forward)
+    "losarax-tiny": (256, 2, 4, 32, 32, 96, 64, 16, 512, 512, 2),
+    "losarax-2k": (2048, 8, 16, 128, 128, 768, 256, 64, 8192, 128256, 4),
+    "losarax-4k": (4096, 8, 32, 128, 128, 1536, 512, 64, 14336, 128256, 4),
+}
+# the llama shape of equal width, feed-forward width and vocabulary
+LOSARAX_PEER = {"losarax-tiny": "tiny", "losarax-2k": "llama-1b", "losarax-4k": "llama-8b"}
+
+
+def losarax_spec(shape: str, n_layers: int | None = None):
+    from .layered import LATENT, LIGHTNING, LayerSpec, LayeredSpec
+
+    width, layers, heads, dim, vdim, qr, kr, rot, ff, vocab, streams = LOSARAX_SHAPES[shape]
+    out = []
+    for i in range(n_layers or layers):
+        if i % 2 == 0:
+            out.append(LayerSpec(LATENT, heads, dim, vdim, ff, q_rank=qr, kv_rank=kr, rot_dim=rot, rot_dims=rot, rot_base=500000.0,
+                                 scale=float((dim + rot) ** -0.5)))
+        else:
+            out.append(LayerSpec(LIGHTNING, heads, dim, vdim, ff, decay=[1.0 - 2.0 ** -(3 + 6.0 * h / heads) for h in range(heads)]))
+    return LayeredSpec(vocab=vocab, width=width, eps=1e-5, layers=out, streams=streams)
+
+
+def build_layered(spec, seed: int, max_pos: int, max_seqs: int = 1, dtype: str = "bfloat16", **kw):
+    """A layered engine with seeded random weights: matrices N(0, 1/cols), norms around 1, streams that stay bounded."""
+    from .layered import LayeredEngine
+
+    eng = LayeredEngine(spec, max_pos, max_seqs, dtype, **kw)
+    for i, (name, shape) in enumerate(eng.tensors().items()):
+        if name.endswith(".mix"):
+            m = np.eye(spec.streams, dtype=np.float32)
+            eng.set_tensor(name, m.reshape(-1))
+        elif len(shape) == 2:
+            eng.synth_tensor(name, seed, i, 0.0, 1.0 if name == "embed" else float(shape[1]) ** -0.5)
+        elif name.endswith((".b", ".out")):
+            eng.synth_tensor(name, seed, i, 0.0, 0.1)
+        elif name.endswith(".in"):
+            eng.synth_tensor(name, seed, i, 1.0 / spec.streams, 0.1)
+        else:
+            eng.synth_tensor(name, seed, i, 1.0, 0.1)
+    return eng
+
+
+def layered_bytes(eng) -> int:
+    """bfloat16 bytes of every matrix one decode step reads once per pass (the embedding: one row)."""
+    total = 0
+    for name, shape in eng.tensors().items():
+        if len(shape) < 2:
+            continue
+        passes = 1
+        if name[0] == "l" and name[1].isdigit():
+            passes = eng.spec.runs.count(int(name[1:name.index(".")]))
+        total += 2 * passes * (shape[1] if name == "embed" else shape[0] * shape[1])
+    return total
+
+
+def layered_context_bytes(eng, context: int, batch: int = 1) -> int:
+    """Cache rows read (bfloat16) and states read and written (f32) by one decode step at that context."""
+    from .layered import LATENT
+
+    total = 0
+    for i in eng.spec.runs:
+        s = eng.spec.layers[i]
+        total += 2 * context * (s.kv_rank + s.rot_dim) if s.type == LATENT else 8 * s.heads * s.dim * s.vdim
+    return total * batch
+
+
 def weight_bytes_per_token(cfg: EngineConfig, mix: str) -> int:
     """Wire bytes of every weight one decode step reads once (the roofline numerator's weight
     term): all layer projections (top-k experts for MoE), norms, the output matrix and one

@@ -422,6 +422,14 @@ CMLD_API int32_t cmld_attention_decode_ordered(const float *q_dev, const void *k
 CMLD_API int32_t cmld_attention_decode_noalloc(const float *q_dev, const void *k_cache_dev, const void *v_cache_dev,
                                                int32_t n_heads, int32_t n_kv_heads, int32_t head_dim, int64_t max_pos,
                                                int64_t n_pos, float scale, float *out_dev);
+/* The linear layer of layered designs as an operator: out[r][o] = act(sum_k w[o][k] x[r][k]) for n rows of x.
+ * kernel 0: matrix-vector form (n <= 2, x f32, out f32); 1: tcgen05 (x bfloat16); 2: FP32 units (x f32).
+ * w_dev: bfloat16 [rows][ld], ld = cols rounded up to 8 with zero padding; x_dev rows of the same ld; out_dev [n][rows]
+ * bfloat16 if out_bf16 else f32.  act 0 none, 1 SiLU on the first act_rows outputs, 2 square of ReLU.
+ * iters > 0: afterwards iters launches are timed (one CUDA-graph replay, CUDA events), the weights visited round-robin
+ * through n_copies matrices w_dev + i * rows * ld; *ms_out = mean milliseconds per launch. */
+CMLD_API int32_t cmld_linear(int32_t kernel, const void *w_dev, int64_t rows, int64_t cols, const void *x_dev, int32_t n, void *out_dev,
+                             int32_t out_bf16, int32_t act, int32_t act_rows, int32_t n_copies, int32_t iters, float *ms_out);
 /* Time `iters` back-to-back launches of cmld_gemv with CUDA events around one CUDA-graph replay of
  * them (so the host's enqueue rate is not measured); the weights are `n_copies` distinct matrices
  * visited round-robin so that the stream comes from HBM when their total exceeds the L2.
