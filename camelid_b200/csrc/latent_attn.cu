@@ -4,7 +4,8 @@
 // Decoding and short portions work in latent space: the query is taken through W_uk^T once (q_nope . W_uk c =
 // (W_uk^T q_nope) . c), the cache rows are scored and averaged as they are, and W_uv is applied to the average.
 //   latent_prep_kernel    rotates and transforms the queries; norms, rotates and appends the new cache rows
-//   latent_attn_kernel    a range of positions for eight heads of one row: online softmax, all in 32-bit
+//   latent_attn_kernel    a range of positions for eight heads of one row: online softmax, all in 32-bit (f32 cache)
+//   latent_attn_mma_kernel  the same for 16 heads on the tensor cores (bfloat16 cache)
 //   latent_output_kernel  merges the ranges, applies W_uv and the sigmoid gate
 // Long portions expand keys and values with two matrix products and run a tiled attention on the tensor cores:
 //   latent_prefill_kernel 64 queries of one head per CTA, 64 keys at a time; scores, weights and sums in 32-bit (the
@@ -18,7 +19,7 @@ namespace {
 
 // ---------------------------------------------------------------- queries into latent space, cache append
 
-constexpr int kPrepThreads = 256, kPrepRanks = 128, kPrepRows = 2;
+constexpr int kPrepThreads = 256, kPrepRanks = 128;
 
 // The value at index j of a rotated vector whose pairs (2i, 2i + 1), i < dims / 2, turn by the angles behind cs.
 __device__ __forceinline__ float rotated(const float *x, int j, int dims, const float *cs) {
@@ -29,14 +30,24 @@ __device__ __forceinline__ float rotated(const float *x, int j, int dims, const 
 }
 
 // grid: x = row groups (appending CTAs: rows), y = head * slices + slice of the latent; the last y appends.
+// ROWS: rows that share a CTA's pass over its weights.
+template <int ROWS>
 __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentArgs a, int slices, int query_ys) {
   __shared__ float red[kPrepThreads / 32];
-  __shared__ float part[kPrepThreads / 64][kPrepRows][kPrepRanks];
-  extern __shared__ float qn[];  // [kPrepRows][dim]
+  extern __shared__ float prep_sm[];
+  float *qn = prep_sm, *part = prep_sm + ROWS * ((a.m.dim + 3) & ~3);  // [ROWS][dim]; [16][kPrepRanks], one row at a time
   pdl_launch();
-  pdl_wait();
   const LatentShape &m = a.m;
-  const int tid = threadIdx.x;
+  const int tid = threadIdx.x, h = blockIdx.y / slices, sl = blockIdx.y % slices;
+  // eight latent dimensions per thread, the head's dimensions over 16 groups of threads; the first 128 of them are asked
+  // for before the predecessor's results (weights depend on no earlier kernel)
+  const int dg = tid >> 4, r = sl * kPrepRanks + (tid & 15) * 8;
+  const bf16 *w = a.uk.w + (int64_t)h * m.dim * a.uk.ld + r;
+  const bool in = (int)blockIdx.y < query_ys && r < (int)a.uk.ld;
+  uint4 pre[8];
+#pragma unroll
+  for (int j = 0; j < 8; ++j) pre[j] = in && dg + 16 * j < m.dim ? ld_stream16(w + (int64_t)(dg + 16 * j) * a.uk.ld) : make_uint4(0, 0, 0, 0);
+  pdl_wait();
   if ((int)blockIdx.y == query_ys) {
     // new cache rows
     for (int r = blockIdx.x; r < a.rows; r += gridDim.x) {
@@ -52,43 +63,49 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
     }
     return;
   }
-  const int h = blockIdx.y / slices, sl = blockIdx.y % slices, qd = m.dim + m.rot_dim, D = m.rank + m.rot_dim;
-  const int n_groups = (a.rows + kPrepRows - 1) / kPrepRows;
+  const int qd = m.dim + m.rot_dim, D = m.rank + m.rot_dim;
+  const int n_groups = (a.rows + ROWS - 1) / ROWS;
   for (int g = blockIdx.x; g < n_groups; g += gridDim.x) {
-    const int r0 = g * kPrepRows, nr = min(kPrepRows, a.rows - r0);
+    const int r0 = g * ROWS, nr = min(ROWS, a.rows - r0);
     __syncthreads();
-    for (int i = tid; i < kPrepRows * m.dim; i += kPrepThreads) {
-      const int r = i / m.dim, d = i % m.dim;
-      qn[i] = r < nr ? a.q[((int64_t)(r0 + r) * m.heads + h) * qd + d] : 0.0f;
+    for (int i = tid; i < ROWS * m.dim; i += kPrepThreads) {
+      const int rr = i / m.dim, d = i % m.dim;
+      qn[i] = rr < nr ? a.q[((int64_t)(r0 + rr) * m.heads + h) * qd + d] : 0.0f;
     }
     __syncthreads();
-    // 64 pairs of latent dimensions x 4 shares of the head's dimensions
-    const int pr = tid & 63, sh = tid >> 6, r = sl * kPrepRanks + 2 * pr;
-    float acc[kPrepRows][2] = {};
-    if (r < m.rank) {
-      const bf16 *w = a.uk.w + (int64_t)h * m.dim * a.uk.ld + r;  // rows are zero-padded to a multiple of 8
-#pragma unroll 8
-      for (int d = sh; d < m.dim; d += 4) {
-        const uint32_t v = *reinterpret_cast<const uint32_t *>(w + (int64_t)d * a.uk.ld);
+    float acc[ROWS][8] = {};
+    auto take = [&](uint4 v, int d) {
+      const float f[8] = {bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y), bf16_lo(v.z), bf16_hi(v.z), bf16_lo(v.w), bf16_hi(v.w)};
 #pragma unroll
-        for (int i = 0; i < kPrepRows; ++i) {
-          const float qv = qn[i * m.dim + d];
-          acc[i][0] = fmaf(bf16_lo(v), qv, acc[i][0]);
-          acc[i][1] = fmaf(bf16_hi(v), qv, acc[i][1]);
-        }
+      for (int i = 0; i < ROWS; ++i) {
+        const float qv = qn[i * m.dim + d];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[i][e] = fmaf(f[e], qv, acc[i][e]);
       }
-    }
+    };
 #pragma unroll
-    for (int i = 0; i < kPrepRows; ++i) {
-      part[sh][i][2 * pr] = acc[i][0];
-      part[sh][i][2 * pr + 1] = acc[i][1];
-    }
-    __syncthreads();
-    for (int i = tid; i < kPrepRows * kPrepRanks; i += kPrepThreads) {
-      const int rr = i / kPrepRanks, c = i % kPrepRanks;
-      if (rr < nr && sl * kPrepRanks + c < m.rank)
-        a.qa[((int64_t)(r0 + rr) * m.heads + h) * D + sl * kPrepRanks + c] =
-            m.scale * (part[0][rr][c] + part[1][rr][c] + part[2][rr][c] + part[3][rr][c]);
+    for (int j = 0; j < 8; ++j)
+      if (dg + 16 * j < m.dim) take(pre[j], dg + 16 * j);
+    if (in)
+      for (int d = dg + 128; d < m.dim; d += 16) take(ld_stream16(w + (int64_t)d * a.uk.ld), d);
+    for (int i = 0; i < nr; ++i) {
+      __syncthreads();
+      float4 *o = reinterpret_cast<float4 *>(part + dg * kPrepRanks + (tid & 15) * 8);
+      float f[8];
+#pragma unroll
+      for (int k = 0; k < ROWS; ++k)
+        if (k == i)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[e] = acc[k][e];
+      o[0] = make_float4(f[0], f[1], f[2], f[3]);
+      o[1] = make_float4(f[4], f[5], f[6], f[7]);
+      __syncthreads();
+      if (tid < kPrepRanks && sl * kPrepRanks + tid < m.rank) {
+        float t = 0.0f;
+#pragma unroll
+        for (int k = 0; k < 16; ++k) t += part[k * kPrepRanks + tid];
+        a.qa[((int64_t)(r0 + i) * m.heads + h) * D + sl * kPrepRanks + tid] = m.scale * t;
+      }
     }
     if (sl == 0)
       for (int i = tid; i < nr * m.rot_dim; i += kPrepThreads) {
@@ -127,9 +144,10 @@ __global__ void __launch_bounds__(kAttThreads) latent_attn_kernel(const LatentAr
   const int tiles = (n + kAttKeys - 1) / kAttKeys, per = (tiles + a.splits - 1) / a.splits;
   const int lo = min(split * per, tiles) * kAttKeys, hi = min(min((split + 1) * per, tiles) * kAttKeys, n);
   const int64_t cache0 = (int64_t)a.slots[row] * a.max_pos * a.cache_ld;
-  for (int i = tid; i < kAttHeads * ld; i += kAttThreads) {
-    const int h = i / ld, d = i % ld;
-    qs[i] = h < nh && d < D ? a.qa[((int64_t)row * m.heads + h0 + h) * D + d] : 0.0f;
+  {
+    const float *q = a.qa + ((int64_t)row * m.heads + h0 + warp) * D;  // a warp brings one head's query
+#pragma unroll 4
+    for (int d = lane; d < ld; d += 32) qs[warp * ld + d] = warp < nh && d < D ? q[d] : 0.0f;
   }
   float acc[kAttHeads][NR][2];
 #pragma unroll
@@ -143,22 +161,22 @@ __global__ void __launch_bounds__(kAttThreads) latent_attn_kernel(const LatentAr
     if (vec) {
       const bf16 *c = static_cast<const bf16 *>(a.cache) + cache0;
       const int u8 = (ld + 7) / 8;
-      for (int i = tid; i < kAttKeys * u8; i += kAttThreads) {
-        const int k = i / u8, d = (i % u8) * 8;
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (k0 + k < hi && d < D) v = *reinterpret_cast<const uint4 *>(c + (int64_t)(k0 + k) * a.cache_ld + d);
-        const float f[8] = {bf16_lo(v.x), bf16_hi(v.x), bf16_lo(v.y), bf16_hi(v.y), bf16_lo(v.z), bf16_hi(v.z), bf16_lo(v.w), bf16_hi(v.w)};
-        float *o = ks + k * ld + d;
+      // a warp takes every eighth key, its lanes 16 bytes each; the cache row's padding beyond D is zero
+      for (int u = lane; u < u8; u += 32) {
+        const int d = u * 8;
+        uint4 v[kAttKeys / 8];
 #pragma unroll
-        for (int q = 0; q < 2; ++q)
-          if (d + 4 * q < ld) {
-            float4 w;
-            w.x = d + 4 * q + 0 < D ? f[4 * q + 0] : 0.0f;
-            w.y = d + 4 * q + 1 < D ? f[4 * q + 1] : 0.0f;
-            w.z = d + 4 * q + 2 < D ? f[4 * q + 2] : 0.0f;
-            w.w = d + 4 * q + 3 < D ? f[4 * q + 3] : 0.0f;
-            *reinterpret_cast<float4 *>(o + 4 * q) = w;
-          }
+        for (int j = 0; j < kAttKeys / 8; ++j) {
+          const int k = warp + 8 * j;
+          v[j] = make_uint4(0, 0, 0, 0);
+          if (k0 + k < hi && d < (int)a.cache_ld) v[j] = *reinterpret_cast<const uint4 *>(c + (int64_t)(k0 + k) * a.cache_ld + d);
+        }
+#pragma unroll
+        for (int j = 0; j < kAttKeys / 8; ++j) {
+          float *o = ks + (warp + 8 * j) * ld + d;
+          *reinterpret_cast<float4 *>(o) = make_float4(bf16_lo(v[j].x), bf16_hi(v[j].x), bf16_lo(v[j].y), bf16_hi(v[j].y));
+          if (d + 4 < ld) *reinterpret_cast<float4 *>(o + 4) = make_float4(bf16_lo(v[j].z), bf16_hi(v[j].z), bf16_lo(v[j].w), bf16_hi(v[j].w));
+        }
       }
     } else {
       for (int i = tid; i < kAttKeys * ld; i += kAttThreads) {
@@ -245,50 +263,206 @@ __global__ void __launch_bounds__(kAttThreads) latent_attn_kernel(const LatentAr
       }
 }
 
+// ---- the same on the tensor cores, for a bfloat16 cache: 16 heads, 32 keys at a time.  Queries and weights enter as two
+// bfloat16 terms each, the cache rows as they are.
+
+constexpr int kMmaHeads = 16, kMmaKeys = 32, kMmaThreads = 256;
+
+__host__ __device__ inline int mma_dp(int D) { return (D + 31) & ~31; }
+__host__ __device__ inline int mma_smem(int D) {
+  const int ds = mma_dp(D) + 8;
+  return (2 * kMmaHeads + 2 * kMmaKeys) * ds * 2 + 2 * kMmaHeads * (kMmaKeys + 1) * 4 + 2 * kMmaHeads * (kMmaKeys + 8) * 2 + kMmaHeads * 4;
+}
+
+// NT: 8-wide tiles of the latent per warp (rank <= 64 * NT)
+template <int NT>
+__global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentArgs a) {
+  extern __shared__ __align__(16) uint8_t mraw[];
+  const LatentShape &m = a.m;
+  const int D = m.rank + m.rot_dim, DP = mma_dp(D), DS = DP + 8, PS = kMmaKeys + 8;
+  bf16 *qh = reinterpret_cast<bf16 *>(mraw), *ql = qh + kMmaHeads * DS, *ks = ql + kMmaHeads * DS;
+  float *sc = reinterpret_cast<float *>(ks + 2 * kMmaKeys * DS);          // [2 halves of D][16][33]
+  bf16 *ph = reinterpret_cast<bf16 *>(sc + 2 * kMmaHeads * (kMmaKeys + 1)), *pl = ph + kMmaHeads * PS;
+  float *corr = reinterpret_cast<float *>(pl + kMmaHeads * PS);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int split = blockIdx.x, h0 = blockIdx.y * kMmaHeads, row = blockIdx.z, nh = min(kMmaHeads, m.heads - h0);
+  pdl_launch();
+  pdl_wait();
+  const int n = a.positions[row] + 1;
+  const int tiles = (n + kMmaKeys - 1) / kMmaKeys, per = (tiles + a.splits - 1) / a.splits;
+  const int t_lo = min(split * per, tiles), t_hi = min(t_lo + per, tiles);
+  const bf16 *cache = static_cast<const bf16 *>(a.cache) + (int64_t)a.slots[row] * a.max_pos * a.cache_ld;
+  // the cache row's padding up to a multiple of eight is zero; beyond it the staged row is zero-filled
+  auto load = [&](int t, bf16 *dst) {
+    for (int u = lane; u < DP / 8; u += 32) {
+#pragma unroll
+      for (int k = warp; k < kMmaKeys; k += kMmaThreads / 32) {
+        const int p = t * kMmaKeys + k;
+        const bool live = p < n && u * 8 < (int)a.cache_ld;
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst + k * DS + u * 8)),
+                     "l"(cache + (live ? (int64_t)p * a.cache_ld + u * 8 : 0)), "r"(live ? 16 : 0)
+                     : "memory");
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (t_lo < t_hi) load(t_lo, ks);
+  for (int h = warp; h < kMmaHeads; h += kMmaThreads / 32) {
+    const float *q = a.qa + ((int64_t)row * m.heads + h0 + h) * D;
+#pragma unroll 4
+    for (int d = lane; d < DP; d += 32) {
+      const float v = h < nh && d < D ? q[d] : 0.0f;
+      const bf16 hi = __float2bfloat16_rn(v);
+      qh[h * DS + d] = hi;
+      ql[h * DS + d] = __float2bfloat16_rn(v - __bfloat162float(hi));
+    }
+  }
+  float O[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) O[i][e] = 0.0f;
+  float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};  // of heads 2 * warp, 2 * warp + 1
+  const int tr = lane >> 2, tc = (lane & 3) * 2;
+  const int dh = warp >> 2, kt = (warp & 3) * 8;                // this warp's half of D and its eight keys
+  for (int t = t_lo; t < t_hi; ++t) {
+    bf16 *k_s = ks + ((t - t_lo) & 1) * kMmaKeys * DS;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    if (t + 1 < t_hi) load(t + 1, ks + ((t + 1 - t_lo) & 1) * kMmaKeys * DS);
+    float P[4] = {};
+    const int d0 = dh * (DP / 2);
+    for (int k = d0; k < d0 + DP / 2; k += 16) {
+      uint32_t A[4], L[4], b0, b1;
+      ldsm4(A, qh + (lane & 15) * DS + k + (lane >> 4) * 8);
+      ldsm4(L, ql + (lane & 15) * DS + k + (lane >> 4) * 8);
+      asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
+                   : "=r"(b0), "=r"(b1)
+                   : "r"((uint32_t)__cvta_generic_to_shared(k_s + (kt + (lane & 7)) * DS + k + ((lane >> 3) & 1) * 8))
+                   : "memory");
+      mma16816(P, A, b0, b1);
+      mma16816(P, L, b0, b1);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) sc[(dh * kMmaHeads + tr + (e >> 1) * 8) * (kMmaKeys + 1) + kt + tc + (e & 1)] = P[e];
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int h = 2 * warp + i;
+      float v = sc[h * (kMmaKeys + 1) + lane] + sc[(kMmaHeads + h) * (kMmaKeys + 1) + lane];
+      if (t * kMmaKeys + lane >= n) v = -INFINITY;
+      const float nm = fmaxf(mx[i], warp_max(v)), c = expf(mx[i] - nm), p = expf(v - nm);
+      sum[i] = fmaf(sum[i], c, warp_sum(p));
+      mx[i] = nm;
+      const bf16 hi = __float2bfloat16_rn(p);
+      ph[h * PS + lane] = hi;
+      pl[h * PS + lane] = __float2bfloat16_rn(p - __bfloat162float(hi));
+      if (lane == 0) corr[h] = c;
+    }
+    __syncthreads();
+    const float c0 = corr[tr], c1 = corr[tr + 8];
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      O[i][0] *= c0;
+      O[i][1] *= c0;
+      O[i][2] *= c1;
+      O[i][3] *= c1;
+    }
+#pragma unroll
+    for (int k = 0; k < kMmaKeys; k += 16) {
+      uint32_t A[4], L[4], B[4];
+      ldsm4(A, ph + (lane & 15) * PS + k + (lane >> 4) * 8);
+      ldsm4(L, pl + (lane & 15) * PS + k + (lane >> 4) * 8);
+#pragma unroll
+      for (int i = 0; i < NT; i += 2) {
+        const int r = (warp * NT + i) * 8;
+        if (r >= DP) break;  // a warp whose tiles lie past the latent
+        ldsm4t(B, k_s + (k + (lane & 15)) * DS + min(r + (lane >> 4) * 8, DP - 8));
+        mma16816(O[i], A, B[0], B[1]);
+        mma16816(O[i + 1], A, B[2], B[3]);
+        mma16816(O[i], L, B[0], B[1]);
+        mma16816(O[i + 1], L, B[2], B[3]);
+      }
+    }
+  }
+  const int64_t ps = m.rank + 2;
+  float *out = a.part + (((int64_t)row * m.heads + h0) * a.splits + split) * ps;
+  if (lane == 0)
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+      if (2 * warp + i < nh) {
+        out[(int64_t)(2 * warp + i) * a.splits * ps] = mx[i];
+        out[(int64_t)(2 * warp + i) * a.splits * ps + 1] = sum[i];
+      }
+#pragma unroll
+  for (int i = 0; i < NT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int h = tr + (e >> 1) * 8, r = (warp * NT + i) * 8 + tc + (e & 1);
+      if (h < nh && r < m.rank) out[(int64_t)h * a.splits * ps + 2 + r] = O[i][e];
+    }
+}
+
 // ---------------------------------------------------------------- merge, W_uv, gate
 
-constexpr int kOutThreads = 256, kOutCols = 32;
+constexpr int kOutThreads = 512, kOutCols = 32, kOutRows = 4;
 
-__global__ void __launch_bounds__(kOutThreads) latent_output_kernel(const LatentArgs a) {
+// grid: x = slices of a head's value dimensions, y = head, z = groups of rows (they share the weights in registers)
+__global__ void __launch_bounds__(kOutThreads) latent_output_kernel(const LatentArgs a, int keys_per_tile) {
   extern __shared__ __align__(16) float ctx[];  // [ld of W_uv]
   __shared__ float wgt[64];
   pdl_launch();
-  pdl_wait();
   const LatentShape &m = a.m;
-  const int row = blockIdx.z, h = blockIdx.y, v0 = blockIdx.x * kOutCols, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int64_t ps = m.rank + 2;
-  const float *part = a.part + ((int64_t)row * m.heads + h) * a.splits * ps;
-  if (warp == 0) {
-    float m0 = lane < a.splits ? part[lane * ps] : -INFINITY, m1 = lane + 32 < a.splits ? part[(lane + 32) * ps] : -INFINITY;
-    const float mx = warp_max(fmaxf(m0, m1));
-    const float e0 = lane < a.splits ? expf(m0 - mx) : 0.0f, e1 = lane + 32 < a.splits ? expf(m1 - mx) : 0.0f;
-    const float l = warp_sum((lane < a.splits ? e0 * part[lane * ps + 1] : 0.0f) + (lane + 32 < a.splits ? e1 * part[(lane + 32) * ps + 1] : 0.0f));
-    wgt[lane] = e0 / l;
-    wgt[lane + 32] = e1 / l;
-  }
-  __syncthreads();
-  for (int i = tid; i < (int)a.uv.ld; i += kOutThreads) {
-    float c = 0.0f;
-    if (i < m.rank)
-#pragma unroll 4
-      for (int s = 0; s < a.splits; ++s)
-        if (wgt[s] != 0.0f) c = fmaf(wgt[s], part[s * ps + 2 + i], c);  // an empty range has weight 0
-    ctx[i] = c;
-  }
-  __syncthreads();
-  for (int v = v0 + warp; v < min(v0 + kOutCols, m.vdim); v += kOutThreads / 32) {
-    const bf16 *w = a.uv.w + ((int64_t)h * m.vdim + v) * a.uv.ld;
-    float s = 0.0f;
-    for (int k = lane * 8; k < (int)a.uv.ld; k += 256) {
-      const uint4 x = *reinterpret_cast<const uint4 *>(w + k);
-      const float4 c0 = *reinterpret_cast<const float4 *>(ctx + k), c1 = *reinterpret_cast<const float4 *>(ctx + k + 4);
-      s = fmaf(bf16_lo(x.x), c0.x, fmaf(bf16_hi(x.x), c0.y, s));
-      s = fmaf(bf16_lo(x.y), c0.z, fmaf(bf16_hi(x.y), c0.w, s));
-      s = fmaf(bf16_lo(x.z), c1.x, fmaf(bf16_hi(x.z), c1.y, s));
-      s = fmaf(bf16_lo(x.w), c1.z, fmaf(bf16_hi(x.w), c1.w, s));
+  const int h = blockIdx.y, v0 = blockIdx.x * kOutCols, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  constexpr int kPer = kOutCols / (kOutThreads / 32);  // value dimensions per warp
+  uint4 w[kPer][2];  // the first 512 weights of each: they depend on no earlier kernel
+#pragma unroll
+  for (int j = 0; j < kPer; ++j)
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+      const int v = v0 + warp + j * (kOutThreads / 32), k = lane * 8 + q * 256;
+      w[j][q] = v < m.vdim && k < (int)a.uv.ld ? ld_stream16(a.uv.w + ((int64_t)h * m.vdim + v) * a.uv.ld + k) : make_uint4(0, 0, 0, 0);
     }
-    s = warp_sum(s);
-    if (lane == 0) act_store(a.out.p, a.out.half, row * a.out.ld + h * m.vdim + v, s * sigmoid_f(a.gate[row * a.gate_ld + h * m.vdim + v]));
+  pdl_wait();
+  const int64_t ps = m.rank + 2;
+  for (int row = blockIdx.z * kOutRows; row < min(((int)blockIdx.z + 1) * kOutRows, a.rows); ++row) {
+    const float *part = a.part + ((int64_t)row * m.heads + h) * a.splits * ps;
+    // the ranges that hold keys (the others are empty)
+    const int tiles = a.positions[row] / keys_per_tile + 1, per = (tiles + a.splits - 1) / a.splits, live = (tiles + per - 1) / per;
+    __syncthreads();
+    if (warp == 0) {
+      const float m0 = lane < live ? part[lane * ps] : -INFINITY, m1 = lane + 32 < live ? part[(lane + 32) * ps] : -INFINITY;
+      const float mx = warp_max(fmaxf(m0, m1));
+      const float e0 = lane < live ? expf(m0 - mx) : 0.0f, e1 = lane + 32 < live ? expf(m1 - mx) : 0.0f;
+      const float l = warp_sum((lane < live ? e0 * part[lane * ps + 1] : 0.0f) + (lane + 32 < live ? e1 * part[(lane + 32) * ps + 1] : 0.0f));
+      wgt[lane] = e0 / l;
+      wgt[lane + 32] = e1 / l;
+    }
+    __syncthreads();
+    for (int i = tid; i < (int)a.uv.ld; i += kOutThreads) {
+      float c = 0.0f;
+      if (i < m.rank)
+#pragma unroll 16
+        for (int s = 0; s < live; ++s) c = fmaf(wgt[s], part[s * ps + 2 + i], c);
+      ctx[i] = c;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int j = 0; j < kPer; ++j) {
+      const int v = v0 + warp + j * (kOutThreads / 32);
+      if (v >= m.vdim) break;
+      float s = 0.0f;
+      for (int k = lane * 8, q = 0; k < (int)a.uv.ld; k += 256, ++q) {
+        const uint4 x = q == 0 ? w[j][0] : q == 1 ? w[j][1] : ld_stream16(a.uv.w + ((int64_t)h * m.vdim + v) * a.uv.ld + k);
+        const float4 c0 = *reinterpret_cast<const float4 *>(ctx + k), c1 = *reinterpret_cast<const float4 *>(ctx + k + 4);
+        s = fmaf(bf16_lo(x.x), c0.x, fmaf(bf16_hi(x.x), c0.y, s));
+        s = fmaf(bf16_lo(x.y), c0.z, fmaf(bf16_hi(x.y), c0.w, s));
+        s = fmaf(bf16_lo(x.z), c1.x, fmaf(bf16_hi(x.z), c1.y, s));
+        s = fmaf(bf16_lo(x.w), c1.z, fmaf(bf16_hi(x.w), c1.w, s));
+      }
+      s = warp_sum(s);
+      if (lane == 0) act_store(a.out.p, a.out.half, row * a.out.ld + h * m.vdim + v, s * sigmoid_f(a.gate[row * a.gate_ld + h * m.vdim + v]));
+    }
   }
 }
 
@@ -319,19 +493,18 @@ __global__ void __launch_bounds__(kPfThreads) latent_prefill_kernel(const Latent
   auto load_tile = [&](int t, int st) {
     bf16 *kd = k_s + st * kPfK * QS, *vd = v_s + st * kPfK * VS;
     const int nu = m.dim / 8, ru = m.rot_dim / 8, ku = nu + ru, vu = m.vdim / 8;
-    for (int i = tid; i < kPfK * ku; i += kPfThreads) {
-      const int k = i / ku, u = i % ku;
-      const int64_t p = (int64_t)t * kPfK + k;
-      const bool live = p <= last;
-      const int64_t pc = live ? p : 0;
-      const bf16 *src = u < nu ? a.kv + pc * a.kv_ld + h * m.dim + u * 8 : a.cache + pc * a.cache_ld + m.rank + (u - nu) * 8;
-      cp16(kd + k * QS + u * 8, src, live);
-    }
-    for (int i = tid; i < kPfK * vu; i += kPfThreads) {
-      const int k = i / vu, u = i % vu;
-      const int64_t p = (int64_t)t * kPfK + k;
-      const bool live = p <= last;
-      cp16(vd + k * VS + u * 8, a.kv + (live ? p : 0) * a.kv_ld + m.heads * m.dim + h * m.vdim + u * 8, live);
+    // a warp takes every fourth key, its lanes the key's 16-byte units: unrotated, rotated, values
+    for (int u = lane; u < ku + vu; u += 32) {
+      const bf16 *src = u < nu ? a.kv + h * m.dim + u * 8 : u < ku ? a.cache + m.rank + (u - nu) * 8 : a.kv + m.heads * m.dim + h * m.vdim + (u - ku) * 8;
+      const int64_t ld = u >= nu && u < ku ? a.cache_ld : a.kv_ld;
+      bf16 *dst = u < ku ? kd + u * 8 : vd + (u - ku) * 8;
+      const int ds = u < ku ? QS : VS;
+      const int64_t p0 = (int64_t)t * kPfK;
+#pragma unroll 8
+      for (int k = warp; k < kPfK; k += kPfThreads / 32) {
+        const bool live = p0 + k <= last;
+        cp16(dst + k * ds, src + (live ? p0 + k : 0) * ld, live);
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -343,14 +516,32 @@ __global__ void __launch_bounds__(kPfThreads) latent_prefill_kernel(const Latent
   for (int i = tid; i < 2 * kPfK * (DV - m.vdim); i += kPfThreads) v_s[(i / (DV - m.vdim)) * VS + m.vdim + i % (DV - m.vdim)] = __float2bfloat16_rn(0.0f);
   load_tile(0, 0);
   const int q_ld = m.heads * (m.dim + m.rot_dim);
-  for (int i = tid; i < kPfQ * qd; i += kPfThreads) {
-    const int r = i / qd, d = i % qd;
-    float v = 0.0f;
-    if (r0 + r < a.rows && d < m.dim + m.rot_dim) {
-      const float *x = a.q + (int64_t)(r0 + r) * q_ld + h * (m.dim + m.rot_dim);
-      v = d < m.dim ? x[d] : rotated(x + m.dim, d - m.dim, m.rot_dims, a.cs + (a.start + r0 + r) * m.rot_dims);
+  {
+    // queries, eight dimensions at a time (dim and rot_dim are multiples of eight; pairs do not straddle)
+    const int units = qd / 8, live = (m.dim + m.rot_dim) / 8;
+#pragma unroll 4
+    for (int i = tid; i < kPfQ * units; i += kPfThreads) {
+      const int r = i / units, u = i % units;
+      float f[8] = {};
+      if (r0 + r < a.rows && u < live) {
+        const float4 *x = reinterpret_cast<const float4 *>(a.q + (int64_t)(r0 + r) * q_ld + h * (m.dim + m.rot_dim) + u * 8);
+        const float4 x0 = x[0], x1 = x[1];
+        f[0] = x0.x, f[1] = x0.y, f[2] = x0.z, f[3] = x0.w, f[4] = x1.x, f[5] = x1.y, f[6] = x1.z, f[7] = x1.w;
+        const int j = u * 8 - m.dim;  // place in the rotated part
+        if (j >= 0) {
+          const float *cs = a.cs + (a.start + r0 + r) * m.rot_dims + j;
+#pragma unroll
+          for (int e = 0; e < 8; e += 2)
+            if (j + e < m.rot_dims) {
+              const float c = cs[e], s = cs[e + 1], x = f[e], y = f[e + 1];
+              f[e] = x * c - y * s;
+              f[e + 1] = y * c + x * s;
+            }
+        }
+      }
+      *reinterpret_cast<uint4 *>(q_s + r * QS + u * 8) =
+          make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
     }
-    q_s[r * QS + d] = __float2bfloat16_rn(v);
   }
   float O[DV / 8][4];
 #pragma unroll
@@ -471,8 +662,24 @@ bool latent_shape_ok(const LatentShape &m) {
 
 int32_t launch_latent_prep(const LatentArgs &a, bool queries, bool pdl, cudaStream_t s) {
   const int slices = (a.m.rank + kPrepRanks - 1) / kPrepRanks, ys = queries ? a.m.heads * slices : 0;
-  const int gx = std::min<int>(queries ? (a.rows + kPrepRows - 1) / kPrepRows : a.rows, 16384);
-  return launch_kernel(latent_prep_kernel, dim3(gx, ys + 1), dim3(kPrepThreads), (size_t)kPrepRows * a.m.dim * 4, pdl, s, a, slices, ys);
+  const int rows = queries && a.rows > 2 ? 8 : queries ? 2 : 1;
+  const int gx = std::min<int>((a.rows + rows - 1) / rows, 16384);
+  const size_t smem = (size_t)(rows * ((a.m.dim + 3) & ~3) + 16 * kPrepRanks) * 4;
+  static bool ready = false;
+  if (!ready) {
+    CMLD_TRY(allow_smem(latent_prep_kernel<8>, 160 * 1024));
+    CMLD_TRY(allow_smem(latent_prep_kernel<2>, 160 * 1024));
+    ready = true;
+  }
+  if (rows == 8) return launch_kernel(latent_prep_kernel<8>, dim3(gx, ys + 1), dim3(kPrepThreads), smem, pdl, s, a, slices, ys);
+  return launch_kernel(latent_prep_kernel<2>, dim3(gx, ys + 1), dim3(kPrepThreads), (size_t)(2 * ((a.m.dim + 3) & ~3) + 16 * kPrepRanks) * 4, pdl, s, a, slices, ys);
+}
+
+bool latent_attention_mma(const LatentArgs &a) { return a.cache_half && mma_smem(a.m.rank + a.m.rot_dim) <= 227 * 1024; }
+
+int latent_attention_groups(const LatentArgs &a) {
+  const int g = latent_attention_mma(a) ? kMmaHeads : kAttHeads;
+  return (a.m.heads + g - 1) / g;
 }
 
 int32_t launch_latent_attention(const LatentArgs &a, bool pdl, cudaStream_t s) {
@@ -480,17 +687,30 @@ int32_t launch_latent_attention(const LatentArgs &a, bool pdl, cudaStream_t s) {
   if (!ready) {
     CMLD_TRY(allow_smem(latent_attn_kernel<1>, 227 * 1024));
     CMLD_TRY(allow_smem(latent_attn_kernel<2>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<2>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<4>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<8>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<16>, 227 * 1024));
     ready = true;
   }
-  const dim3 grid(a.splits, (a.m.heads + kAttHeads - 1) / kAttHeads, a.rows);
-  const size_t smem = att_smem(a.m.rank + a.m.rot_dim);
-  if (a.m.rank <= 512) return launch_kernel(latent_attn_kernel<1>, grid, dim3(kAttThreads), smem, pdl, s, a);
-  return launch_kernel(latent_attn_kernel<2>, grid, dim3(kAttThreads), smem, pdl, s, a);
+  const dim3 grid(a.splits, latent_attention_groups(a), a.rows);
+  const int D = a.m.rank + a.m.rot_dim;
+  if (latent_attention_mma(a)) {
+    const dim3 block(kMmaThreads);
+    if (a.m.rank <= 128) return launch_kernel(latent_attn_mma_kernel<2>, grid, block, mma_smem(D), pdl, s, a);
+    if (a.m.rank <= 256) return launch_kernel(latent_attn_mma_kernel<4>, grid, block, mma_smem(D), pdl, s, a);
+    if (a.m.rank <= 512) return launch_kernel(latent_attn_mma_kernel<8>, grid, block, mma_smem(D), pdl, s, a);
+    return launch_kernel(latent_attn_mma_kernel<16>, grid, block, mma_smem(D), pdl, s, a);
+  }
+  if (a.m.rank <= 512) return launch_kernel(latent_attn_kernel<1>, grid, dim3(kAttThreads), att_smem(D), pdl, s, a);
+  return launch_kernel(latent_attn_kernel<2>, grid, dim3(kAttThreads), att_smem(D), pdl, s, a);
 }
 
 int32_t launch_latent_output(const LatentArgs &a, bool pdl, cudaStream_t s) {
   if (a.splits > 64) return fail(CMLD_ERR_INVALID, "latent attention: %d ranges, at most 64", a.splits);
-  return launch_kernel(latent_output_kernel, dim3((a.m.vdim + kOutCols - 1) / kOutCols, a.m.heads, a.rows), dim3(kOutThreads), (size_t)a.uv.ld * 4, pdl, s, a);
+  static_assert(kMmaKeys == kAttKeys, "both attention kernels cut a range at the same keys");
+  return launch_kernel(latent_output_kernel, dim3((a.m.vdim + kOutCols - 1) / kOutCols, a.m.heads, (a.rows + kOutRows - 1) / kOutRows), dim3(kOutThreads),
+                       (size_t)a.uv.ld * 4, pdl, s, a, kMmaKeys);
 }
 
 bool latent_prefill_fits(const LatentShape &m, int64_t cache_ld, int64_t kv_ld) {

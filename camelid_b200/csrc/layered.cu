@@ -252,8 +252,7 @@ int32_t build(cmld_engine *e, LayeredModel *m) {
       const int64_t kv_ld = lin_ld(H * (d.dim + d.vdim));
       if (!m->f32 && latent_prefill_fits(L.lat, cache_ld(L), kv_ld)) kv = std::max(kv, kv_ld);
       qa = std::max(qa, H * (d.kv_rank + d.rot_dim));
-      const int64_t groups = (H + 7) / 8;
-      part = std::max(part, (int64_t)(2 * e->sm_count * 8 + std::min<int64_t>(R, kLatentRows) * groups * 8) * (d.kv_rank + 2));
+      part = std::max(part, (int64_t)(2 * e->sm_count * 16 + std::min<int64_t>(R, kLatentRows) * H) * (d.kv_rank + 2));
     } else {
       wide = std::max(wide, lin_ld(L.in.rows));
       proj = std::max<int64_t>(proj, H * d.vdim);
@@ -452,12 +451,12 @@ struct Step {
       CMLD_TRY(launch_latent_prefill(p, pdl, e->stream));
       e->launches += 1;
     } else {
-      const int groups = (d.heads + 7) / 8;
+      const int groups = latent_attention_groups(a);
       const int64_t cap = o.attn_cap > 0 ? o.attn_cap : m->cfg.max_pos;
       for (int r0 = 0; r0 < R; r0 += kLatentRows) {
         const int n = std::min(kLatentRows, R - r0);
         rows_from(r0, n);
-        a.splits = (int)std::max<int64_t>(1, std::min<int64_t>({64, (2 * e->sm_count) / (n * groups), cap / 64}));
+        a.splits = (int)std::max<int64_t>(1, std::min<int64_t>({64, (2 * e->sm_count) / (n * groups), cap / 32}));
         if ((int64_t)n * d.heads * a.splits * (d.kv_rank + 2) > m->part_floats) return fail(CMLD_ERR_STATE, "latent attention: partials exceed the scratch");
         CMLD_TRY(launch_latent_prep(a, true, pdl, e->stream));
         CMLD_TRY(launch_latent_attention(a, pdl, e->stream));

@@ -119,6 +119,7 @@ struct LatentArgs {
 };
 // Appends the rows' latents to the cache; with queries, also brings the queries into latent space.
 int32_t launch_latent_prep(const LatentArgs &a, bool queries, bool pdl, cudaStream_t s);
+int latent_attention_groups(const LatentArgs &a);  // CTAs the heads of a row are spread over
 int32_t launch_latent_attention(const LatentArgs &a, bool pdl, cudaStream_t s);
 int32_t launch_latent_output(const LatentArgs &a, bool pdl, cudaStream_t s);
 bool latent_shape_ok(const LatentShape &m);

@@ -66,9 +66,14 @@ __global__ void __launch_bounds__(kStepThreads) lightning_steps_kernel(const Lig
 
 constexpr int kC = kLightningChunk, kChunkCols = 32, kChunkThreads = 128;
 
-// shared memory: Q, K [64][dim + 8], V, V' hi, V' lo [64][40], S hi, S lo [dim][40] (all bf16), powers [65]
+// shared memory: two stages of Q, K [64][dim + 8] and V [64][40]; V' hi, V' lo [64][40], S hi, S lo [dim][40] (all bf16);
+// powers [65]
 __host__ __device__ inline int chunk_smem(int dp) {
-  return 2 * kC * (dp + 8) * 2 + 3 * kC * (kChunkCols + 8) * 2 + 2 * dp * (kChunkCols + 8) * 2 + (kC + 1) * 4 + 16;
+  return 2 * (2 * kC * (dp + 8) + kC * (kChunkCols + 8)) * 2 + 2 * kC * (kChunkCols + 8) * 2 + 2 * dp * (kChunkCols + 8) * 2 + (kC + 1) * 4 + 16;
+}
+
+__device__ __forceinline__ void cp16(void *dst, const void *src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
 }
 
 // MT: 16-row tiles of the state per warp (dim <= 64 * MT)
@@ -76,8 +81,8 @@ template <int MT>
 __global__ void __launch_bounds__(kChunkThreads) lightning_chunk_kernel(const LightningArgs a) {
   extern __shared__ __align__(16) uint8_t raw[];
   constexpr int DP = 64 * MT, QS = DP + 8, VS = kChunkCols + 8;
-  bf16 *q_s = reinterpret_cast<bf16 *>(raw), *k_s = q_s + kC * QS, *v_s = k_s + kC * QS, *vh_s = v_s + kC * VS, *vl_s = vh_s + kC * VS,
-       *sh_s = vl_s + kC * VS, *sl_s = sh_s + DP * VS;
+  constexpr int kStage = 2 * kC * QS + kC * VS;  // elements: Q, K, V of one chunk
+  bf16 *stage = reinterpret_cast<bf16 *>(raw), *vh_s = stage + 2 * kStage, *vl_s = vh_s + kC * VS, *sh_s = vl_s + kC * VS, *sl_s = sh_s + DP * VS;
   float *pw = reinterpret_cast<float *>(sl_s + DP * VS);
   pdl_launch();
   pdl_wait();
@@ -100,9 +105,49 @@ __global__ void __launch_bounds__(kChunkThreads) lightning_chunk_kernel(const Li
         S[m][n][e] = !fresh && d < a.dim && c < a.vdim ? st[(int64_t)d * a.vdim + c] : 0.0f;
       }
   const bool vec = a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0;
-  for (int c0 = 0; c0 < a.rows; c0 += kC) {
+  // a chunk's rows into a stage; rows past the end and columns past the sizes are zero
+  auto load = [&](int c0, bf16 *q_s) {
+    bf16 *k_s = q_s + kC * QS, *v_s = k_s + kC * QS;
     const int len = min(kC, a.rows - c0);
-    __syncthreads();  // the previous chunk's readers are done
+    const bf16 *x0 = x + (int64_t)c0 * a.ld;
+    if (vec) {
+#pragma unroll 4
+      for (int i = tid; i < kC * (DP / 8); i += kChunkThreads) {
+        const int r = i / (DP / 8), d = (i % (DP / 8)) * 8;
+        const bool live = r < len && d < a.dim;
+        const bf16 *p = live ? x0 + (int64_t)r * a.ld + h * a.dim + d : x;
+        cp16(q_s + r * QS + d, p, live);
+        cp16(k_s + r * QS + d, live ? p + hd : x, live);
+      }
+#pragma unroll
+      for (int i = tid; i < kC * (kChunkCols / 8); i += kChunkThreads) {
+        const int r = i / (kChunkCols / 8), c = (i % (kChunkCols / 8)) * 8;
+        const bool live = r < len && col0 + c < a.vdim;
+        cp16(v_s + r * VS + c, live ? x0 + (int64_t)r * a.ld + 2 * hd + h * a.vdim + col0 + c : x, live);
+      }
+    } else {
+      const bf16 zero = __float2bfloat16_rn(0.0f);
+      for (int i = tid; i < kC * DP; i += kChunkThreads) {
+        const int r = i / DP, d = i % DP;
+        const bool live = r < len && d < a.dim;
+        const bf16 *p = x0 + (int64_t)r * a.ld + h * a.dim + d;
+        q_s[r * QS + d] = live ? p[0] : zero;
+        k_s[r * QS + d] = live ? p[hd] : zero;
+      }
+      for (int i = tid; i < kC * kChunkCols; i += kChunkThreads) {
+        const int r = i / kChunkCols, c = i % kChunkCols;
+        v_s[r * VS + c] = r < len && col0 + c < a.vdim ? x0[(int64_t)r * a.ld + 2 * hd + h * a.vdim + col0 + c] : zero;
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load(0, stage);
+  for (int c0 = 0; c0 < a.rows; c0 += kC) {
+    const int len = min(kC, a.rows - c0), st = (c0 / kC) & 1;
+    const bf16 *q_s = stage + st * kStage, *k_s = q_s + kC * QS, *v_s = k_s + kC * QS;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();  // this chunk has landed, and the previous one's readers are done
+    if (c0 + kC < a.rows) load(c0 + kC, stage + (st ^ 1) * kStage);
     // the state as two bf16 terms, for Q S
 #pragma unroll
     for (int m = 0; m < MT; ++m)
@@ -116,35 +161,16 @@ __global__ void __launch_bounds__(kChunkThreads) lightning_chunk_kernel(const Li
           *reinterpret_cast<uint32_t *>(sh_s + o) = hi;
           *reinterpret_cast<uint32_t *>(sl_s + o) = lo;
         }
-    if (vec) {
-      for (int i = tid; i < kC * (DP / 8); i += kChunkThreads) {
-        const int r = i / (DP / 8), d = (i % (DP / 8)) * 8;
-        uint4 qv = make_uint4(0, 0, 0, 0), kv = qv;
-        if (r < len && d < a.dim) {
-          const bf16 *p = x + (int64_t)(c0 + r) * a.ld + h * a.dim + d;
-          qv = *reinterpret_cast<const uint4 *>(p);
-          kv = *reinterpret_cast<const uint4 *>(p + hd);
-        }
-        *reinterpret_cast<uint4 *>(q_s + r * QS + d) = qv;
-        *reinterpret_cast<uint4 *>(k_s + r * QS + d) = kv;
-      }
-    } else {
-      for (int i = tid; i < kC * DP; i += kChunkThreads) {
-        const int r = i / DP, d = i % DP;
-        const bool in = r < len && d < a.dim;
-        const bf16 *p = x + (int64_t)(c0 + r) * a.ld + h * a.dim + d;
-        q_s[r * QS + d] = in ? p[0] : __float2bfloat16_rn(0.0f);
-        k_s[r * QS + d] = in ? p[hd] : __float2bfloat16_rn(0.0f);
-      }
-    }
-    for (int i = tid; i < kC * kChunkCols; i += kChunkThreads) {
-      const int r = i / kChunkCols, c = i % kChunkCols;
-      const bf16 v = r < len && col0 + c < a.vdim ? x[(int64_t)(c0 + r) * a.ld + 2 * hd + h * a.vdim + col0 + c] : __float2bfloat16_rn(0.0f);
-      v_s[r * VS + c] = v;
-      const float w = r < len ? __bfloat162float(v) * pw[len - 1 - r] : 0.0f;
-      const bf16 wh = __float2bfloat16_rn(w);
-      vh_s[r * VS + c] = wh;
-      vl_s[r * VS + c] = __float2bfloat16_rn(w - __bfloat162float(wh));
+    // V' = diag(decay^(len-1-j)) V as two terms
+#pragma unroll
+    for (int i = tid; i < kC * kChunkCols / 2; i += kChunkThreads) {
+      const int r = i / (kChunkCols / 2), c = (i % (kChunkCols / 2)) * 2;
+      const uint32_t v = *reinterpret_cast<const uint32_t *>(v_s + r * VS + c);
+      const float w = r < len ? pw[len - 1 - r] : 0.0f;
+      uint32_t hi, lo;
+      split_pair(bf16_lo(v) * w, bf16_hi(v) * w, hi, lo);
+      *reinterpret_cast<uint32_t *>(vh_s + r * VS + c) = hi;
+      *reinterpret_cast<uint32_t *>(vl_s + r * VS + c) = lo;
     }
     __syncthreads();
 

@@ -5,8 +5,8 @@
 // and brought by TMA in 128-byte-swizzled boxes of 64 columns.  Persistent CTAs, one per SM; warp roles:
 //   warp 0      TMA: operand stages (one elected lane)
 //   warp 1      MMA issue (one elected lane), tensor-memory allocation
-//   warps 2-5   epilogue: tcgen05.ld, activation, stores; two accumulator slots, so that a tile's epilogue overlaps the
-//               next tile's products
+//   warps 2-9   epilogue: tcgen05.ld, activation, stores, two warps for each quarter of the accumulator lanes (every
+//               other 16 columns); two accumulator slots, so that a tile's epilogue overlaps the next tile's products
 // Few rows leave few tiles: then `split` CTAs of a thread-block cluster share a tile's inner dimension, leave their
 // partial accumulators in shared memory, and each of them adds the partials of its share of the columns in rank order.
 // The first weight boxes are asked for before the kernel waits for its predecessor.
@@ -20,7 +20,7 @@ namespace cmld {
 
 namespace {
 
-constexpr int kThreads = 192, kBM = 128, kBK = 64;
+constexpr int kEpiWarps = 8, kThreads = (2 + kEpiWarps) * 32, kBM = 128, kBK = 64;
 constexpr uint32_t kSpin = 1u << 22;
 constexpr int kABytes = kBM * kBK * 2;
 
@@ -100,6 +100,9 @@ __device__ __forceinline__ float ld_peer(uint32_t local_addr, uint32_t rank) {
   return v;
 }
 
+__device__ __forceinline__ void put(float *p, float v) { *p = v; }
+__device__ __forceinline__ void put(bf16 *p, float v) { *p = __float2bfloat16_rn(v); }
+
 template <int BN, typename OutT>
 __global__ void __launch_bounds__(kThreads, 1)
     lin_tc5_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const TcLinArgs a) {
@@ -128,7 +131,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     }
     for (int i = 0; i < 2; ++i) {
       bar_init(acc_full(i), 1);
-      bar_init(acc_empty(i), 4);
+      bar_init(acc_empty(i), kEpiWarps);
     }
     *abort_flag = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -190,7 +193,7 @@ __global__ void __launch_bounds__(kThreads, 1)
     }
     __syncwarp();
   } else {
-    const int quarter = warp & 3;  // the 32 accumulator lanes this warp may read
+    const int quarter = warp & 3, half = (warp - 2) >> 2;  // the 32 accumulator lanes this warp may read; its column groups
     pdl_wait();                    // the output buffer may still be read by the predecessor
     int i = 0;
     OutT *out = static_cast<OutT *>(a.out);
@@ -202,9 +205,10 @@ __global__ void __launch_bounds__(kThreads, 1)
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const int n_live = min(BN, a.n_rows - n0);
       float *part = reinterpret_cast<float *>(smem);  // [BN][128]: the operand stages are free by now
+      const bool silu = a.act == kActSilu && o < a.act_rows, relu2 = a.act == kActRelu2;
+      OutT *p = out + (int64_t)(n0 + 16 * half) * a.out_ld + o;
 #pragma unroll 1
-      for (int c = 0; c < BN; c += 16) {
-        if (c >= n_live) break;
+      for (int c = 16 * half; c < n_live; c += 32, p += 32 * a.out_ld) {
         float r[16];
         if (nk > 0) {
           tmem_ld16(tbase + slot * TSLOT + c + ((uint32_t)(quarter * 32) << 16), r);
@@ -215,14 +219,28 @@ __global__ void __launch_bounds__(kThreads, 1)
         if (a.split > 1) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) part[(c + j) * kBM + quarter * 32 + lane] = r[j];
-        } else if (o < a.m_rows) {
+          continue;
+        }
+        if (silu) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j)
-            if (c + j < n_live) {
-              const float v = lin_activate(r[j], a.act, o < a.act_rows);
-              if constexpr (sizeof(OutT) == 2) out[(int64_t)(n0 + c + j) * a.out_ld + o] = __float2bfloat16_rn(v);
-              else out[(int64_t)(n0 + c + j) * a.out_ld + o] = v;
-            }
+          for (int j = 0; j < 16; ++j) r[j] = r[j] * sigmoid_f(r[j]);
+        } else if (relu2) {
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            const float v = fmaxf(r[j], 0.0f);
+            r[j] = v * v;
+          }
+        }
+        if (o < a.m_rows) {
+          OutT *w = p;
+          if (c + 16 <= n_live) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j, w += a.out_ld) put(w, r[j]);
+          } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j, w += a.out_ld)
+              if (c + j < n_live) put(w, r[j]);
+          }
         }
       }
       asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -243,8 +261,7 @@ __global__ void __launch_bounds__(kThreads, 1)
         for (int p = 0; p < a.split; ++p) v += ld_peer(base + 4u * e, p);
         if (o < a.m_rows) {
           v = lin_activate(v, a.act, o < a.act_rows);
-          if constexpr (sizeof(OutT) == 2) out[(int64_t)(n0 + n) * a.out_ld + o] = __float2bfloat16_rn(v);
-          else out[(int64_t)(n0 + n) * a.out_ld + o] = v;
+          put(out + (int64_t)(n0 + n) * a.out_ld + o, v);
         }
       }
     }

@@ -6,7 +6,9 @@ namespace cmld {
 
 namespace {
 
-constexpr int kMixThreads = 256;
+// One CTA per row: wide CTAs while the rows are too few to fill the machine.
+constexpr int kMixThreads = 1024;
+int mix_threads(int rows) { return rows >= 512 ? 256 : rows >= 256 ? 512 : kMixThreads; }
 
 __global__ void __launch_bounds__(kMixThreads) stream_mix_kernel(const StreamMix m, ActBuf out) {
   extern __shared__ float u[];
@@ -33,8 +35,10 @@ __global__ void __launch_bounds__(kMixThreads) rms_rows_kernel(const float *x, i
   const int64_t r = blockIdx.x;
   const float *xr = x + r * x_ld;
   float s = 0.0f;
+#pragma unroll 4
   for (int i = threadIdx.x; i < cols; i += blockDim.x) s = fmaf(xr[i], xr[i], s);
   const float inv = 1.0f / sqrtf(cta_total(s, red) / (float)cols + eps);
+#pragma unroll 4
   for (int i = threadIdx.x; i < cols; i += blockDim.x) {
     float v = xr[i] * inv * w[i];
     if (gate.p) v *= sigmoid_f(act_load(gate.p, gate.half, r * gate.ld + i));
@@ -47,18 +51,18 @@ __global__ void __launch_bounds__(kMixThreads) rms_rows_kernel(const float *x, i
 int32_t launch_stream_mix(const StreamMix &m, int32_t rows, ActBuf out, bool pdl, cudaStream_t s) {
   const size_t smem = (size_t)m.width * 4;
   if (smem > 48 * 1024) CMLD_TRY(allow_smem(stream_mix_kernel, smem));
-  return launch_kernel(stream_mix_kernel, dim3(rows), dim3(kMixThreads), smem, pdl, s, m, out);
+  return launch_kernel(stream_mix_kernel, dim3(rows), dim3(mix_threads(rows)), smem, pdl, s, m, out);
 }
 
 int32_t launch_stream_tap(const StreamMix &m, int32_t rows, float *out, cudaStream_t s) {
   const size_t smem = (size_t)m.width * 4;
   if (smem > 48 * 1024) CMLD_TRY(allow_smem(stream_tap_kernel, smem));
-  return launch_kernel(stream_tap_kernel, dim3(rows), dim3(kMixThreads), smem, false, s, m, out);
+  return launch_kernel(stream_tap_kernel, dim3(rows), dim3(mix_threads(rows)), smem, false, s, m, out);
 }
 
 int32_t launch_rms_rows(const float *x, int64_t x_ld, const float *w, int32_t cols, float eps, ActBuf gate, ActBuf out, int32_t rows,
                         bool pdl, cudaStream_t s) {
-  return launch_kernel(rms_rows_kernel, dim3(rows), dim3(kMixThreads), 0, pdl, s, x, x_ld, w, cols, eps, gate, out);
+  return launch_kernel(rms_rows_kernel, dim3(rows), dim3(mix_threads(rows)), 0, pdl, s, x, x_ld, w, cols, eps, gate, out);
 }
 
 }  // namespace cmld
