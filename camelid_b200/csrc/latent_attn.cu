@@ -29,13 +29,34 @@ __device__ __forceinline__ float rotated(const float *x, int j, int dims, const 
   return (j & 1) ? v * c + u * s : u * c - v * s;
 }
 
-// grid: x = row groups (appending CTAs: rows), y = head * slices + slice of the latent; the last y appends.
+// One new cache row, by the whole CTA: the latent RMS-normed, the key part rotated.
+__device__ __forceinline__ void latent_append(const LatentArgs &a, int r, float *red) {
+  const LatentShape &m = a.m;
+  const float *low = a.low + (int64_t)r * a.low_ld;
+  const int64_t pos = a.positions[r];
+  const int64_t at = ((int64_t)a.slots[r] * a.max_pos + pos) * a.cache_ld;
+  float s = 0.0f;
+  for (int i = threadIdx.x; i < m.rank; i += blockDim.x) s = fmaf(low[i], low[i], s);
+  const float inv = 1.0f / sqrtf(cta_total(s, red) / (float)m.rank + m.eps);
+  for (int i = threadIdx.x; i < m.rank; i += blockDim.x) act_store(a.cache, a.cache_half, at + i, low[i] * inv * a.latent_norm[i]);
+  for (int i = threadIdx.x; i < m.rot_dim; i += blockDim.x)
+    act_store(a.cache, a.cache_half, at + m.rank + i, rotated(low + m.rank, i, m.rot_dims, a.cs + pos * m.rot_dims));
+}
+
+__global__ void __launch_bounds__(128) latent_append_kernel(const LatentArgs a) {
+  __shared__ float red[4];
+  pdl_launch();
+  pdl_wait();
+  latent_append(a, blockIdx.x, red);
+}
+
+// grid: x = row groups, y = head * slices + slice of the latent; the last ROWS y append the new cache rows.
 // ROWS: rows that share a CTA's pass over its weights.
 template <int ROWS>
-__global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentArgs a, int slices, int query_ys) {
+__global__ void __launch_bounds__(kPrepThreads, 2) latent_prep_kernel(const LatentArgs a, int slices, int query_ys) {
   __shared__ float red[kPrepThreads / 32];
   extern __shared__ float prep_sm[];
-  float *qn = prep_sm, *part = prep_sm + ROWS * ((a.m.dim + 3) & ~3);  // [ROWS][dim]; [16][kPrepRanks], one row at a time
+  float *qn = prep_sm, *part = prep_sm + ROWS * ((a.m.dim + 3) & ~3);  // [ROWS][dim]; [16][ROWS][kPrepRanks]
   pdl_launch();
   const LatentShape &m = a.m;
   const int tid = threadIdx.x, h = blockIdx.y / slices, sl = blockIdx.y % slices;
@@ -48,19 +69,8 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
 #pragma unroll
   for (int j = 0; j < 8; ++j) pre[j] = in && dg + 16 * j < m.dim ? ld_stream16(w + (int64_t)(dg + 16 * j) * a.uk.ld) : make_uint4(0, 0, 0, 0);
   pdl_wait();
-  if ((int)blockIdx.y == query_ys) {
-    // new cache rows
-    for (int r = blockIdx.x; r < a.rows; r += gridDim.x) {
-      const float *low = a.low + (int64_t)r * a.low_ld;
-      const int64_t pos = a.positions[r];
-      const int64_t at = ((int64_t)a.slots[r] * a.max_pos + pos) * a.cache_ld;
-      float s = 0.0f;
-      for (int i = tid; i < m.rank; i += kPrepThreads) s = fmaf(low[i], low[i], s);
-      const float inv = 1.0f / sqrtf(cta_total(s, red) / (float)m.rank + m.eps);
-      for (int i = tid; i < m.rank; i += kPrepThreads) act_store(a.cache, a.cache_half, at + i, low[i] * inv * a.latent_norm[i]);
-      for (int i = tid; i < m.rot_dim; i += kPrepThreads)
-        act_store(a.cache, a.cache_half, at + m.rank + i, rotated(low + m.rank, i, m.rot_dims, a.cs + pos * m.rot_dims));
-    }
+  if ((int)blockIdx.y >= query_ys) {
+    for (int row = blockIdx.x + gridDim.x * (blockIdx.y - query_ys); row < a.rows; row += gridDim.x * ROWS) latent_append(a, row, red);
     return;
   }
   const int qd = m.dim + m.rot_dim, D = m.rank + m.rot_dim;
@@ -88,23 +98,21 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentA
       if (dg + 16 * j < m.dim) take(pre[j], dg + 16 * j);
     if (in)
       for (int d = dg + 128; d < m.dim; d += 16) take(ld_stream16(w + (int64_t)d * a.uk.ld), d);
-    for (int i = 0; i < nr; ++i) {
-      __syncthreads();
-      float4 *o = reinterpret_cast<float4 *>(part + dg * kPrepRanks + (tid & 15) * 8);
-      float f[8];
 #pragma unroll
-      for (int k = 0; k < ROWS; ++k)
-        if (k == i)
+    for (int i = 0; i < ROWS; ++i) {
+      float4 *o = reinterpret_cast<float4 *>(part + (dg * ROWS + i) * kPrepRanks + (tid & 15) * 8);
+      o[0] = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+      o[1] = make_float4(acc[i][4], acc[i][5], acc[i][6], acc[i][7]);
+    }
+    __syncthreads();
 #pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = acc[k][e];
-      o[0] = make_float4(f[0], f[1], f[2], f[3]);
-      o[1] = make_float4(f[4], f[5], f[6], f[7]);
-      __syncthreads();
-      if (tid < kPrepRanks && sl * kPrepRanks + tid < m.rank) {
+    for (int o = tid; o < ROWS * kPrepRanks; o += kPrepThreads) {
+      const int i = o / kPrepRanks, c = o % kPrepRanks;
+      if (i < nr && sl * kPrepRanks + c < m.rank) {
         float t = 0.0f;
 #pragma unroll
-        for (int k = 0; k < 16; ++k) t += part[k * kPrepRanks + tid];
-        a.qa[((int64_t)(r0 + i) * m.heads + h) * D + sl * kPrepRanks + tid] = m.scale * t;
+        for (int k = 0; k < 16; ++k) t += part[(k * ROWS + i) * kPrepRanks + c];
+        a.qa[((int64_t)(r0 + i) * m.heads + h) * D + sl * kPrepRanks + c] = m.scale * t;
       }
     }
     if (sl == 0)
@@ -268,24 +276,25 @@ __global__ void __launch_bounds__(kAttThreads) latent_attn_kernel(const LatentAr
 
 constexpr int kMmaHeads = 16, kMmaKeys = 32, kMmaThreads = 256;
 
-__host__ __device__ inline int mma_dp(int D) { return (D + 31) & ~31; }
+__host__ __device__ inline int mma_dp(int D) { return (D + 15) & ~15; }
 __host__ __device__ inline int mma_smem(int D) {
-  const int ds = mma_dp(D) + 8;
-  return (2 * kMmaHeads + 2 * kMmaKeys) * ds * 2 + 2 * kMmaHeads * (kMmaKeys + 1) * 4 + 2 * kMmaHeads * (kMmaKeys + 8) * 2 + kMmaHeads * 4;
+  return 2 * kMmaKeys * (mma_dp(D) + 8) * 2 + 8 * kMmaHeads * (kMmaKeys + 1) * 4 + 2 * kMmaHeads * (kMmaKeys + 8) * 2 + kMmaHeads * 4;
 }
 
-// NT: 8-wide tiles of the latent per warp (rank <= 64 * NT)
-template <int NT>
+// NT: 8-wide tiles of the latent per warp in the second product (rank <= 64 * NT).  KS: 16-wide steps of the dimensions
+// per warp in the first (D <= 128 * KS); a warp keeps its share of the queries in registers.
+template <int NT, int KS>
 __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const LatentArgs a) {
   extern __shared__ __align__(16) uint8_t mraw[];
   const LatentShape &m = a.m;
   const int D = m.rank + m.rot_dim, DP = mma_dp(D), DS = DP + 8, PS = kMmaKeys + 8;
-  bf16 *qh = reinterpret_cast<bf16 *>(mraw), *ql = qh + kMmaHeads * DS, *ks = ql + kMmaHeads * DS;
-  float *sc = reinterpret_cast<float *>(ks + 2 * kMmaKeys * DS);          // [2 halves of D][16][33]
-  bf16 *ph = reinterpret_cast<bf16 *>(sc + 2 * kMmaHeads * (kMmaKeys + 1)), *pl = ph + kMmaHeads * PS;
+  bf16 *ks = reinterpret_cast<bf16 *>(mraw);                                // two stages of [32][DS]
+  float *sc = reinterpret_cast<float *>(ks + 2 * kMmaKeys * DS);            // [8 shares of D][16][33]
+  bf16 *ph = reinterpret_cast<bf16 *>(sc + 8 * kMmaHeads * (kMmaKeys + 1)), *pl = ph + kMmaHeads * PS;
   float *corr = reinterpret_cast<float *>(pl + kMmaHeads * PS);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int split = blockIdx.x, h0 = blockIdx.y * kMmaHeads, row = blockIdx.z, nh = min(kMmaHeads, m.heads - h0);
+  const int tr = lane >> 2, tc = (lane & 3) * 2;
   pdl_launch();
   pdl_wait();
   const int n = a.positions[row] + 1;
@@ -307,15 +316,16 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (t_lo < t_hi) load(t_lo, ks);
-  for (int h = warp; h < kMmaHeads; h += kMmaThreads / 32) {
-    const float *q = a.qa + ((int64_t)row * m.heads + h0 + h) * D;
-#pragma unroll 4
-    for (int d = lane; d < DP; d += 32) {
-      const float v = h < nh && d < D ? q[d] : 0.0f;
-      const bf16 hi = __float2bfloat16_rn(v);
-      qh[h * DS + d] = hi;
-      ql[h * DS + d] = __float2bfloat16_rn(v - __bfloat162float(hi));
-    }
+  uint32_t QH[KS][4], QL[KS][4];
+  if (t_lo < t_hi) {
+    const float *q = a.qa + ((int64_t)row * m.heads + h0) * D;
+#pragma unroll
+    for (int i = 0; i < KS; ++i)
+#pragma unroll
+      for (int f = 0; f < 4; ++f) {
+        const int h = tr + (f & 1) * 8, d = (warp * KS + i) * 16 + (f >> 1) * 8 + tc;
+        split_pair(h < nh && d < D ? q[(int64_t)h * D + d] : 0.0f, h < nh && d + 1 < D ? q[(int64_t)h * D + d + 1] : 0.0f, QH[i][f], QL[i][f]);
+      }
   }
   float O[NT][4];
 #pragma unroll
@@ -323,33 +333,37 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
 #pragma unroll
     for (int e = 0; e < 4; ++e) O[i][e] = 0.0f;
   float mx[2] = {-INFINITY, -INFINITY}, sum[2] = {0.0f, 0.0f};  // of heads 2 * warp, 2 * warp + 1
-  const int tr = lane >> 2, tc = (lane & 3) * 2;
-  const int dh = warp >> 2, kt = (warp & 3) * 8;                // this warp's half of D and its eight keys
   for (int t = t_lo; t < t_hi; ++t) {
     bf16 *k_s = ks + ((t - t_lo) & 1) * kMmaKeys * DS;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     if (t + 1 < t_hi) load(t + 1, ks + ((t + 1 - t_lo) & 1) * kMmaKeys * DS);
-    float P[4] = {};
-    const int d0 = dh * (DP / 2);
-    for (int k = d0; k < d0 + DP / 2; k += 16) {
-      uint32_t A[4], L[4], b0, b1;
-      ldsm4(A, qh + (lane & 15) * DS + k + (lane >> 4) * 8);
-      ldsm4(L, ql + (lane & 15) * DS + k + (lane >> 4) * 8);
-      asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];"
-                   : "=r"(b0), "=r"(b1)
-                   : "r"((uint32_t)__cvta_generic_to_shared(k_s + (kt + (lane & 7)) * DS + k + ((lane >> 3) & 1) * 8))
-                   : "memory");
-      mma16816(P, A, b0, b1);
-      mma16816(P, L, b0, b1);
+    float P[4][4] = {};
+#pragma unroll
+    for (int i = 0; i < KS; ++i) {
+      const int k = (warp * KS + i) * 16;
+      if (k >= DP) break;
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {  // 16 keys at a time
+        uint32_t B[4];
+        ldsm4(B, k_s + (j * 16 + (lane & 7) + ((lane >> 4) << 3)) * DS + k + ((lane >> 3) & 1) * 8);
+        mma16816(P[2 * j], QH[i], B[0], B[1]);
+        mma16816(P[2 * j + 1], QH[i], B[2], B[3]);
+        mma16816(P[2 * j], QL[i], B[0], B[1]);
+        mma16816(P[2 * j + 1], QL[i], B[2], B[3]);
+      }
     }
 #pragma unroll
-    for (int e = 0; e < 4; ++e) sc[(dh * kMmaHeads + tr + (e >> 1) * 8) * (kMmaKeys + 1) + kt + tc + (e & 1)] = P[e];
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sc[(warp * kMmaHeads + tr + (e >> 1) * 8) * (kMmaKeys + 1) + j * 8 + tc + (e & 1)] = P[j][e];
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < 2; ++i) {
       const int h = 2 * warp + i;
-      float v = sc[h * (kMmaKeys + 1) + lane] + sc[(kMmaHeads + h) * (kMmaKeys + 1) + lane];
+      float v = 0.0f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) v += sc[(w * kMmaHeads + h) * (kMmaKeys + 1) + lane];
       if (t * kMmaKeys + lane >= n) v = -INFINITY;
       const float nm = fmaxf(mx[i], warp_max(v)), c = expf(mx[i] - nm), p = expf(v - nm);
       sum[i] = fmaf(sum[i], c, warp_sum(p));
@@ -405,12 +419,13 @@ __global__ void __launch_bounds__(kMmaThreads) latent_attn_mma_kernel(const Late
 
 // ---------------------------------------------------------------- merge, W_uv, gate
 
-constexpr int kOutThreads = 512, kOutCols = 32, kOutRows = 4;
+constexpr int kOutThreads = 512, kOutCols = 32;
 
-// grid: x = slices of a head's value dimensions, y = head, z = groups of rows (they share the weights in registers)
-__global__ void __launch_bounds__(kOutThreads) latent_output_kernel(const LatentArgs a, int keys_per_tile) {
-  extern __shared__ __align__(16) float ctx[];  // [ld of W_uv]
-  __shared__ float wgt[64];
+// grid: x = slices of a head's value dimensions, y = head, z = groups of ROWS rows (they share the weights in registers)
+template <int ROWS>
+__global__ void __launch_bounds__(kOutThreads, 2) latent_output_kernel(const LatentArgs a, int keys_per_tile) {
+  extern __shared__ __align__(16) float ctx[];  // [ROWS][ld of W_uv]
+  __shared__ float wgt[ROWS][64];
   pdl_launch();
   const LatentShape &m = a.m;
   const int h = blockIdx.y, v0 = blockIdx.x * kOutCols, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -425,43 +440,64 @@ __global__ void __launch_bounds__(kOutThreads) latent_output_kernel(const Latent
     }
   pdl_wait();
   const int64_t ps = m.rank + 2;
-  for (int row = blockIdx.z * kOutRows; row < min(((int)blockIdx.z + 1) * kOutRows, a.rows); ++row) {
-    const float *part = a.part + ((int64_t)row * m.heads + h) * a.splits * ps;
-    // the ranges that hold keys (the others are empty)
-    const int tiles = a.positions[row] / keys_per_tile + 1, per = (tiles + a.splits - 1) / a.splits, live = (tiles + per - 1) / per;
-    __syncthreads();
-    if (warp == 0) {
-      const float m0 = lane < live ? part[lane * ps] : -INFINITY, m1 = lane + 32 < live ? part[(lane + 32) * ps] : -INFINITY;
-      const float mx = warp_max(fmaxf(m0, m1));
-      const float e0 = lane < live ? expf(m0 - mx) : 0.0f, e1 = lane + 32 < live ? expf(m1 - mx) : 0.0f;
-      const float l = warp_sum((lane < live ? e0 * part[lane * ps + 1] : 0.0f) + (lane + 32 < live ? e1 * part[(lane + 32) * ps + 1] : 0.0f));
-      wgt[lane] = e0 / l;
-      wgt[lane + 32] = e1 / l;
-    }
-    __syncthreads();
-    for (int i = tid; i < (int)a.uv.ld; i += kOutThreads) {
-      float c = 0.0f;
-      if (i < m.rank)
-#pragma unroll 16
-        for (int s = 0; s < live; ++s) c = fmaf(wgt[s], part[s * ps + 2 + i], c);
-      ctx[i] = c;
-    }
-    __syncthreads();
+  const int row0 = blockIdx.z * ROWS, nr = min(ROWS, a.rows - row0), ld = (int)a.uv.ld;
+  // the ranges of a row that hold keys (the others are empty)
+  auto live_of = [&](int r) {
+    const int tiles = a.positions[row0 + r] / keys_per_tile + 1, per = (tiles + a.splits - 1) / a.splits;
+    return (tiles + per - 1) / per;
+  };
+  if (warp < nr) {
+    const int live = live_of(warp);
+    const float *part = a.part + ((int64_t)(row0 + warp) * m.heads + h) * a.splits * ps;
+    const float m0 = lane < live ? part[lane * ps] : -INFINITY, m1 = lane + 32 < live ? part[(lane + 32) * ps] : -INFINITY;
+    const float l0 = lane < live ? part[lane * ps + 1] : 0.0f, l1 = lane + 32 < live ? part[(lane + 32) * ps + 1] : 0.0f;
+    const float mx = warp_max(fmaxf(m0, m1));
+    const float e0 = lane < live ? expf(m0 - mx) : 0.0f, e1 = lane + 32 < live ? expf(m1 - mx) : 0.0f;
+    const float l = warp_sum(e0 * l0 + e1 * l1);
+    wgt[warp][lane] = e0 / l;
+    wgt[warp][lane + 32] = e1 / l;
+  }
+  __syncthreads();
+  constexpr int kFlight = ROWS == 1 ? 16 : 4;  // partials of a row in flight
+  for (int i = tid; i < ld; i += kOutThreads)
 #pragma unroll
-    for (int j = 0; j < kPer; ++j) {
-      const int v = v0 + warp + j * (kOutThreads / 32);
-      if (v >= m.vdim) break;
-      float s = 0.0f;
-      for (int k = lane * 8, q = 0; k < (int)a.uv.ld; k += 256, ++q) {
-        const uint4 x = q == 0 ? w[j][0] : q == 1 ? w[j][1] : ld_stream16(a.uv.w + ((int64_t)h * m.vdim + v) * a.uv.ld + k);
-        const float4 c0 = *reinterpret_cast<const float4 *>(ctx + k), c1 = *reinterpret_cast<const float4 *>(ctx + k + 4);
-        s = fmaf(bf16_lo(x.x), c0.x, fmaf(bf16_hi(x.x), c0.y, s));
-        s = fmaf(bf16_lo(x.y), c0.z, fmaf(bf16_hi(x.y), c0.w, s));
-        s = fmaf(bf16_lo(x.z), c1.x, fmaf(bf16_hi(x.z), c1.y, s));
-        s = fmaf(bf16_lo(x.w), c1.z, fmaf(bf16_hi(x.w), c1.w, s));
+    for (int r = 0; r < ROWS; ++r) {
+      if (r >= nr) break;
+      const int live = live_of(r);
+      const float *part = a.part + ((int64_t)(row0 + r) * m.heads + h) * a.splits * ps + 2;
+      float c = 0.0f;
+      for (int s0 = 0; s0 < live; s0 += kFlight) {
+        float p[kFlight];
+#pragma unroll
+        for (int j = 0; j < kFlight; ++j) p[j] = s0 + j < live && i < m.rank ? part[(s0 + j) * ps + i] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < kFlight; ++j) c = fmaf(wgt[r][s0 + j], p[j], c);
       }
-      s = warp_sum(s);
-      if (lane == 0) act_store(a.out.p, a.out.half, row * a.out.ld + h * m.vdim + v, s * sigmoid_f(a.gate[row * a.gate_ld + h * m.vdim + v]));
+      ctx[r * ld + i] = c;
+    }
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < kPer; ++j) {
+    const int v = v0 + warp + j * (kOutThreads / 32);
+    if (v >= m.vdim) break;
+    float s[ROWS] = {};
+    for (int k = lane * 8, q = 0; k < ld; k += 256, ++q) {
+      const uint4 x = q == 0 ? w[j][0] : q == 1 ? w[j][1] : ld_stream16(a.uv.w + ((int64_t)h * m.vdim + v) * ld + k);
+#pragma unroll
+      for (int r = 0; r < ROWS; ++r)
+        if (r < nr) {
+          const float4 c0 = *reinterpret_cast<const float4 *>(ctx + r * ld + k), c1 = *reinterpret_cast<const float4 *>(ctx + r * ld + k + 4);
+          s[r] = fmaf(bf16_lo(x.x), c0.x, fmaf(bf16_hi(x.x), c0.y, s[r]));
+          s[r] = fmaf(bf16_lo(x.y), c0.z, fmaf(bf16_hi(x.y), c0.w, s[r]));
+          s[r] = fmaf(bf16_lo(x.z), c1.x, fmaf(bf16_hi(x.z), c1.y, s[r]));
+          s[r] = fmaf(bf16_lo(x.w), c1.z, fmaf(bf16_hi(x.w), c1.w, s[r]));
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+      const float t = warp_sum(s[r]);
+      const int64_t row = row0 + r;
+      if (lane == 0 && r < nr) act_store(a.out.p, a.out.half, row * a.out.ld + h * m.vdim + v, t * sigmoid_f(a.gate[row * a.gate_ld + h * m.vdim + v]));
     }
   }
 }
@@ -660,22 +696,24 @@ bool latent_shape_ok(const LatentShape &m) {
          m.rot_dims <= m.rot_dim && att_smem(m.rank + m.rot_dim) <= 227 * 1024 && m.dim <= 4096;
 }
 
-int32_t launch_latent_prep(const LatentArgs &a, bool queries, bool pdl, cudaStream_t s) {
-  const int slices = (a.m.rank + kPrepRanks - 1) / kPrepRanks, ys = queries ? a.m.heads * slices : 0;
-  const int rows = queries && a.rows > 2 ? 8 : queries ? 2 : 1;
-  const int gx = std::min<int>((a.rows + rows - 1) / rows, 16384);
-  const size_t smem = (size_t)(rows * ((a.m.dim + 3) & ~3) + 16 * kPrepRanks) * 4;
+template <int ROWS>
+int32_t prep(const LatentArgs &a, bool pdl, cudaStream_t s) {
   static bool ready = false;
   if (!ready) {
-    CMLD_TRY(allow_smem(latent_prep_kernel<8>, 160 * 1024));
-    CMLD_TRY(allow_smem(latent_prep_kernel<2>, 160 * 1024));
+    CMLD_TRY(allow_smem(latent_prep_kernel<ROWS>, 160 * 1024));
     ready = true;
   }
-  if (rows == 8) return launch_kernel(latent_prep_kernel<8>, dim3(gx, ys + 1), dim3(kPrepThreads), smem, pdl, s, a, slices, ys);
-  return launch_kernel(latent_prep_kernel<2>, dim3(gx, ys + 1), dim3(kPrepThreads), (size_t)(2 * ((a.m.dim + 3) & ~3) + 16 * kPrepRanks) * 4, pdl, s, a, slices, ys);
+  const int slices = (a.m.rank + kPrepRanks - 1) / kPrepRanks, ys = a.m.heads * slices;
+  const size_t smem = (size_t)(ROWS * ((a.m.dim + 3) & ~3) + 16 * ROWS * kPrepRanks) * 4;
+  return launch_kernel(latent_prep_kernel<ROWS>, dim3((a.rows + ROWS - 1) / ROWS, ys + ROWS), dim3(kPrepThreads), smem, pdl, s, a, slices, ys);
 }
 
-bool latent_attention_mma(const LatentArgs &a) { return a.cache_half && mma_smem(a.m.rank + a.m.rot_dim) <= 227 * 1024; }
+int32_t launch_latent_prep(const LatentArgs &a, bool queries, bool pdl, cudaStream_t s) {
+  if (!queries) return launch_kernel(latent_append_kernel, dim3(a.rows), dim3(128), 0, pdl, s, a);
+  return a.rows > 2 ? prep<4>(a, pdl, s) : prep<2>(a, pdl, s);
+}
+
+bool latent_attention_mma(const LatentArgs &a) { return a.cache_half && a.m.rank + a.m.rot_dim <= 1152 && mma_smem(a.m.rank + a.m.rot_dim) <= 227 * 1024; }
 
 int latent_attention_groups(const LatentArgs &a) {
   const int g = latent_attention_mma(a) ? kMmaHeads : kAttHeads;
@@ -687,20 +725,20 @@ int32_t launch_latent_attention(const LatentArgs &a, bool pdl, cudaStream_t s) {
   if (!ready) {
     CMLD_TRY(allow_smem(latent_attn_kernel<1>, 227 * 1024));
     CMLD_TRY(allow_smem(latent_attn_kernel<2>, 227 * 1024));
-    CMLD_TRY(allow_smem(latent_attn_mma_kernel<2>, 227 * 1024));
-    CMLD_TRY(allow_smem(latent_attn_mma_kernel<4>, 227 * 1024));
-    CMLD_TRY(allow_smem(latent_attn_mma_kernel<8>, 227 * 1024));
-    CMLD_TRY(allow_smem(latent_attn_mma_kernel<16>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<2, 2>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<4, 3>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<8, 5>, 227 * 1024));
+    CMLD_TRY(allow_smem(latent_attn_mma_kernel<16, 9>, 227 * 1024));
     ready = true;
   }
   const dim3 grid(a.splits, latent_attention_groups(a), a.rows);
   const int D = a.m.rank + a.m.rot_dim;
   if (latent_attention_mma(a)) {
     const dim3 block(kMmaThreads);
-    if (a.m.rank <= 128) return launch_kernel(latent_attn_mma_kernel<2>, grid, block, mma_smem(D), pdl, s, a);
-    if (a.m.rank <= 256) return launch_kernel(latent_attn_mma_kernel<4>, grid, block, mma_smem(D), pdl, s, a);
-    if (a.m.rank <= 512) return launch_kernel(latent_attn_mma_kernel<8>, grid, block, mma_smem(D), pdl, s, a);
-    return launch_kernel(latent_attn_mma_kernel<16>, grid, block, mma_smem(D), pdl, s, a);
+    if (a.m.rank <= 128 && D <= 256) return launch_kernel(latent_attn_mma_kernel<2, 2>, grid, block, mma_smem(D), pdl, s, a);
+    if (a.m.rank <= 256 && D <= 384) return launch_kernel(latent_attn_mma_kernel<4, 3>, grid, block, mma_smem(D), pdl, s, a);
+    if (a.m.rank <= 512 && D <= 640) return launch_kernel(latent_attn_mma_kernel<8, 5>, grid, block, mma_smem(D), pdl, s, a);
+    return launch_kernel(latent_attn_mma_kernel<16, 9>, grid, block, mma_smem(D), pdl, s, a);
   }
   if (a.m.rank <= 512) return launch_kernel(latent_attn_kernel<1>, grid, dim3(kAttThreads), att_smem(D), pdl, s, a);
   return launch_kernel(latent_attn_kernel<2>, grid, dim3(kAttThreads), att_smem(D), pdl, s, a);
@@ -709,8 +747,9 @@ int32_t launch_latent_attention(const LatentArgs &a, bool pdl, cudaStream_t s) {
 int32_t launch_latent_output(const LatentArgs &a, bool pdl, cudaStream_t s) {
   if (a.splits > 64) return fail(CMLD_ERR_INVALID, "latent attention: %d ranges, at most 64", a.splits);
   static_assert(kMmaKeys == kAttKeys, "both attention kernels cut a range at the same keys");
-  return launch_kernel(latent_output_kernel, dim3((a.m.vdim + kOutCols - 1) / kOutCols, a.m.heads, (a.rows + kOutRows - 1) / kOutRows), dim3(kOutThreads),
-                       (size_t)a.uv.ld * 4, pdl, s, a, kMmaKeys);
+  const dim3 grid((a.m.vdim + kOutCols - 1) / kOutCols, a.m.heads, a.rows <= 2 ? a.rows : (a.rows + 3) / 4);
+  if (a.rows <= 2) return launch_kernel(latent_output_kernel<1>, grid, dim3(kOutThreads), (size_t)a.uv.ld * 4, pdl, s, a, kMmaKeys);
+  return launch_kernel(latent_output_kernel<4>, grid, dim3(kOutThreads), (size_t)4 * a.uv.ld * 4, pdl, s, a, kMmaKeys);
 }
 
 bool latent_prefill_fits(const LatentShape &m, int64_t cache_ld, int64_t kv_ld) {
