@@ -426,6 +426,7 @@ template <int ROWS>
 __global__ void __launch_bounds__(kOutThreads, 2) latent_output_kernel(const LatentArgs a, int keys_per_tile) {
   extern __shared__ __align__(16) float ctx[];  // [ROWS][ld of W_uv]
   __shared__ float wgt[ROWS][64];
+  __shared__ int ranges[ROWS];
   pdl_launch();
   const LatentShape &m = a.m;
   const int h = blockIdx.y, v0 = blockIdx.x * kOutCols, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -441,13 +442,10 @@ __global__ void __launch_bounds__(kOutThreads, 2) latent_output_kernel(const Lat
   pdl_wait();
   const int64_t ps = m.rank + 2;
   const int row0 = blockIdx.z * ROWS, nr = min(ROWS, a.rows - row0), ld = (int)a.uv.ld;
-  // the ranges of a row that hold keys (the others are empty)
-  auto live_of = [&](int r) {
-    const int tiles = a.positions[row0 + r] / keys_per_tile + 1, per = (tiles + a.splits - 1) / a.splits;
-    return (tiles + per - 1) / per;
-  };
   if (warp < nr) {
-    const int live = live_of(warp);
+    // the ranges of the row that hold keys (the others are empty)
+    const int tiles = a.positions[row0 + warp] / keys_per_tile + 1, per = (tiles + a.splits - 1) / a.splits, live = (tiles + per - 1) / per;
+    if (lane == 0) ranges[warp] = live;
     const float *part = a.part + ((int64_t)(row0 + warp) * m.heads + h) * a.splits * ps;
     const float m0 = lane < live ? part[lane * ps] : -INFINITY, m1 = lane + 32 < live ? part[(lane + 32) * ps] : -INFINITY;
     const float l0 = lane < live ? part[lane * ps + 1] : 0.0f, l1 = lane + 32 < live ? part[(lane + 32) * ps + 1] : 0.0f;
@@ -463,13 +461,13 @@ __global__ void __launch_bounds__(kOutThreads, 2) latent_output_kernel(const Lat
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
       if (r >= nr) break;
-      const int live = live_of(r);
-      const float *part = a.part + ((int64_t)(row0 + r) * m.heads + h) * a.splits * ps + 2;
+      const int live = i < m.rank ? ranges[r] : 0;
+      const float *part = a.part + ((int64_t)(row0 + r) * m.heads + h) * a.splits * ps + 2 + i;
       float c = 0.0f;
-      for (int s0 = 0; s0 < live; s0 += kFlight) {
+      for (int s0 = 0; s0 < live; s0 += kFlight, part += kFlight * (int)ps) {
         float p[kFlight];
 #pragma unroll
-        for (int j = 0; j < kFlight; ++j) p[j] = s0 + j < live && i < m.rank ? part[(s0 + j) * ps + i] : 0.0f;
+        for (int j = 0; j < kFlight; ++j) p[j] = s0 + j < live ? part[j * (int)ps] : 0.0f;
 #pragma unroll
         for (int j = 0; j < kFlight; ++j) c = fmaf(wgt[r][s0 + j], p[j], c);
       }
