@@ -29,15 +29,24 @@ class Tensor(C.Structure):
     _fields_ = [("data", C.c_void_p), ("nbytes", C.c_uint64), ("qtype", C.c_int32), ("reserved", C.c_int32)]
 
 
+class WindowDesc(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("heads", "kv_heads", "dim", "vdim", "rot_dims", "window")] + [("scale", C.c_float)] + [
+        (n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")]
+
+
+class GatedDesc(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("heads", "dim", "vdim", "rank")] + [("tau", C.c_double)]
+
+
 class LayerDesc(C.Structure):
-    _fields_ = [(n, C.c_int32) for n in ("type", "heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "ff")] + [
-        ("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.POINTER(C.c_float))]
+    _fields_ = [(n, C.c_int32) for n in ("type", "heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "ff", "mlp")] + [
+        ("scale", C.c_float), ("rot_base", C.c_double), ("decay", C.POINTER(C.c_float)), ("window", WindowDesc), ("gated", GatedDesc)]
 
 
 class LayeredConfig(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_layers", "loop_start", "loop_stop", "loop_times", "streams", "width", "vocab", "max_pos",
-                                         "max_seqs", "dtype", "device", "flags")] + [
-        ("eps", C.c_float), ("layers", C.POINTER(LayerDesc))]
+                                         "max_seqs", "dtype", "device", "flags", "residual", "portion")] + [
+        ("eps", C.c_float), ("embed_scale", C.c_float), ("logit_scale", C.c_float), ("layers", C.POINTER(LayerDesc))]
 
 
 def lib_path() -> Path:
@@ -158,7 +167,7 @@ def lib():
         "cmld_attention_decode": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, f32, vp]),
         "cmld_attention_decode_noalloc": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, f32, vp]),
         "cmld_attention_decode_ordered": (i32, [vp, vp, vp, i32, i32, i32, i64, i64, f32, vp]),
-        "cmld_linear": (i32, [i32, vp, i64, i64, vp, i32, vp, i32, i32, i32, i32, i32, P(f32)]),
+        "cmld_linear": (i32, [i32, vp, i64, i64, vp, i32, vp, i32, i32, i32, vp, f32, i32, i32, P(f32)]),
         "cmld_gemv_time": (i32, [P(vp), i32, vp, i32, vp, i32, i32, P(f32)]),
     }
     for name, (res, args) in sig.items():

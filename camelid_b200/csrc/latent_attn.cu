@@ -504,10 +504,6 @@ __global__ void __launch_bounds__(kOutThreads, 2) latent_output_kernel(const Lat
 
 constexpr int kPfThreads = 128, kPfQ = 64, kPfK = 64;
 
-__device__ __forceinline__ void cp16(void *dst, const void *src, bool live) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
-}
-
 __host__ __device__ inline int pf_qd(const LatentShape &m) { return (m.dim + m.rot_dim + 15) & ~15; }
 __host__ __device__ inline int pf_smem(int qd, int dv) { return (kPfQ * (qd + 8) + 2 * kPfK * (qd + 8) + 2 * kPfK * (dv + 8)) * 2; }
 

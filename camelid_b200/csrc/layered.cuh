@@ -26,25 +26,32 @@ struct ActBuf {
   int64_t ld = 0;  // elements
 };
 
-// What a linear layer does to its sums: SiLU on output rows below act_rows, the square of ReLU on all, or nothing.
-enum LinAct { kActNone = 0, kActSilu = 1, kActRelu2 = 2 };
+// What a linear layer does to its sums: SiLU on output rows below act_rows, the square of ReLU on all, SiLU of an even row's
+// sum times the sum of the next row (half as many outputs as rows), or nothing.
+enum LinAct { kActNone = 0, kActSilu = 1, kActRelu2 = 2, kActSwiGlu = 3 };
+inline int64_t lin_outputs(int64_t rows, int act) { return act == kActSwiGlu ? rows / 2 : rows; }
 
-// One boundary between two sublayers of a residual held as `streams` parallel copies (hyper-connections): the update of
-// the sublayer that has just produced y, then the read-out and layer norm that feed the next one.
-//   x'_t = sum_s mix[s][t] x_s + out[t] y;   u = sum_t in[t] x'_t (in == null: the plain sum);   result = LN(u)
-// embed != null: the first boundary instead: x' = LN_embed(embed[token]) in every stream.
+// One boundary between two sublayers: the update of the residual with what the sublayer has just produced, then the read-out
+// and norm that feed the next one.
+//   y' = y, or 0.5 (rms(y) y_norm + rms(y2) y2_norm) where two branches ran side by side; with out_norm: y' <- rms(y') out_norm
+//   several copies of the residual (hyper-connections):
+//     x'_t = sum_s mix[s][t] x_s + out[t] y';   u = sum_t in[t] x'_t (in == null: the plain sum)
+//   mix == null: one stream, u = x' = x + y'
+//   result = LN(u) (norm_w and norm_b), rms(u) norm_w (norm_w alone), or u
+// embed != null: the first boundary instead: x' = embed_scale * embed[token], layer-normed with enorm_w, in every stream.
 // All of it in 32-bit.
 struct StreamMix {
   const float *x_in = nullptr;  // [row][streams][width]
   float *x_out = nullptr;       // same layout, another buffer; null: the updated streams are not kept
   const float *y = nullptr;     // [row][width]
+  const float *y2 = nullptr, *y_norm = nullptr, *y2_norm = nullptr, *out_norm = nullptr;  // mix == null only
   const float *mix = nullptr, *out = nullptr, *in = nullptr;
-  const float *norm_w = nullptr, *norm_b = nullptr;  // null: no norm
-  float eps = 0.0f;
+  const float *norm_w = nullptr, *norm_b = nullptr;
+  float eps = 0.0f, embed_scale = 1.0f;
   const bf16 *embed = nullptr;
   int64_t embed_ld = 0;
   const int32_t *tokens = nullptr;
-  const float *enorm_w = nullptr, *enorm_b = nullptr;
+  const float *enorm_w = nullptr, *enorm_b = nullptr;  // null: no norm
   int32_t streams = 1, width = 0;
   const int32_t *row_map = nullptr;  // result row r comes from row row_map[r]; null: r
 };
@@ -56,10 +63,13 @@ int32_t launch_stream_tap(const StreamMix &m, int32_t rows, float *out, cudaStre
 // out[r] = x[r] / rms(x[r]) * w (* sigmoid(gate[r])), x f32 [rows][x_ld]; gate f32 or bf16
 int32_t launch_rms_rows(const float *x, int64_t x_ld, const float *w, int32_t cols, float eps, ActBuf gate, ActBuf out, int32_t rows,
                         bool pdl, cudaStream_t s);
+// The same over groups of `group` columns that share the weights w[group], times silu(gate[r]) (f32).
+int32_t launch_rms_groups(const float *x, int64_t x_ld, const float *w, int32_t cols, int32_t group, float eps, const float *gate, int64_t gate_ld,
+                          ActBuf out, int32_t rows, bool pdl, cudaStream_t s);
 
 // lin_mv.cu: up to two activation rows, one pass over the weights at HBM speed, with the operand's preparation fused
 // into the prologue of every CTA.
-enum LinPrologue { kProPlain = 0, kProRms = 1, kProRmsGate = 2, kProStreams = 3 };
+enum LinPrologue { kProPlain = 0, kProRms = 1, kProRmsGate = 2, kProStreams = 3, kProRmsGroups = 4 };
 struct LinMvArgs {
   LinW w;
   int32_t batch = 1;
@@ -69,16 +79,21 @@ struct LinMvArgs {
   int64_t x_ld = 0;
   const float *norm_w = nullptr;
   float eps = 0.0f;
-  const float *gate = nullptr;  // kProRmsGate: f32 rows, multiplied by their sigmoid
+  const float *gate = nullptr;  // kProRmsGate: f32 rows, multiplied by their sigmoid; kProRmsGroups: by their SiLU
   int64_t gate_ld = 0;
+  int32_t group = 0;            // kProRmsGroups: columns of a group
   float *y = nullptr;
   int64_t y_ld = 0;
   int32_t act = kActNone, act_rows = 0;
+  const float *bias = nullptr;  // [rows], added before the activation
+  float scale = 1.0f;           // of the sums
 };
 bool lin_mv_fits(int32_t cols, int32_t batch);
 int32_t launch_lin_mv(const LinMvArgs &a, bool pdl, cudaStream_t s);
+// Two products that do not depend on each other in one launch, the CTAs split between them by their weights.
+int32_t launch_lin_mv_pair(const LinMvArgs &a, const LinMvArgs &b, bool pdl, cudaStream_t s);
 
-// lin_tc5.cu / lin_f32.cu: any number of rows.  out[r][o] = act(sum_k w[o][k] x[r][k])
+// lin_tc5.cu / lin_f32.cu: any number of rows.  out[r][o] = act(scale * sum_k w[o][k] x[r][k] + bias[o])
 struct LinArgs {
   LinW w;
   const void *x = nullptr;  // bf16 rows (tcgen05) or f32 rows (f32 kernel), x_ld elements apart
@@ -88,6 +103,8 @@ struct LinArgs {
   int32_t out_half = 0;
   int64_t out_ld = 0;
   int32_t act = kActNone, act_rows = 0;
+  const float *bias = nullptr;
+  float scale = 1.0f;
 };
 int32_t launch_lin_tc5(const LinArgs &a, int32_t sm_count, int32_t *status, bool pdl, cudaStream_t s);
 int32_t launch_lin_f32(const LinArgs &a, cudaStream_t s);
@@ -142,10 +159,55 @@ struct LatentPrefillArgs {
 bool latent_prefill_fits(const LatentShape &m, int64_t cache_ld, int64_t kv_ld);
 int32_t launch_latent_prefill(const LatentPrefillArgs &a, bool pdl, cudaStream_t s);
 
-// lightning.cu: linear attention with a fixed decay per head, state [slot][heads][dim][vdim] in f32.
+// window_attn.cu: attention of grouped heads over a sliding window.  A slot's keys (normed and rotated) and values lie in a
+// ring of `cap` positions, position p in row p % cap, head by head: [slot][kv_head][cap][kp | vp], kp and vp the sizes
+// rounded up to 16, the padding zero.
+struct WindowShape {
+  int32_t heads, kv_heads, dim, vdim, rot_dims;
+  int32_t window;  // 0: every earlier position
+  float scale, eps;
+};
+inline __host__ __device__ int window_pad(int n) { return (n + 15) & ~15; }
+struct WindowArgs {
+  WindowShape m;
+  int32_t rows = 0;
+  const int32_t *positions = nullptr, *slots = nullptr;  // per row
+  const float *cs = nullptr;    // [position][rot_dims / 2][cos, sin]
+  const float *q_norm = nullptr, *k_norm = nullptr;      // [dim]
+  const float *qkv = nullptr;   // [row][ld]: q (heads x dim) | k (kv_heads x dim) | v (kv_heads x vdim)
+  int64_t ld = 0;
+  void *cache = nullptr;
+  int32_t cache_half = 0, cap = 0;
+  void *q = nullptr;            // prepared queries: [row][heads][dim] f32, or [row][heads][kp] bf16
+  int32_t q_half = 0;
+  int32_t append = 0;           // decode: the row's own key and value come from qkv and go into the cache
+  int32_t splits = 1;           // decode: CTAs (one cluster) that share a row's positions
+  ActBuf out;                   // [row][heads * vdim]
+};
+bool window_shape_ok(const WindowShape &m);
+// Norms and rotations: keys and values of the rows into the cache; with `queries` also the queries into q.
+int32_t launch_window_prep(const WindowArgs &a, bool queries, bool pdl, cudaStream_t s);
+int32_t launch_window_attention(const WindowArgs &a, bool pdl, cudaStream_t s);      // FP32 units, any cache; reads q
+bool window_decode_fits(const WindowArgs &a);
+int window_decode_groups(const WindowArgs &a);                                       // CTAs of a row before splitting
+int32_t launch_window_decode(const WindowArgs &a, bool pdl, cudaStream_t s);         // bf16 cache, tensor cores; prepares its queries
+bool window_prefill_fits(const WindowArgs &a);
+int32_t launch_window_prefill(const WindowArgs &a, bool pdl, cudaStream_t s);        // consecutive rows of one sequence, bf16; reads q
+
+// A decay per key channel and token: sigmoid(w x + b)^(1 / tau), x the low-rank projection of the layer's input.
+struct ChannelDecay {
+  LinW w;                          // [heads * dim][rank]
+  const float *b = nullptr;        // [heads * dim]
+  const float *x = nullptr;        // [row][ld of qkv]
+  float inv_tau = 1.0f;
+};
+
+// lightning.cu: linear attention, state [slot][heads][dim][vdim] in f32, with a fixed decay per head or one per channel.
 struct LightningArgs {
   int32_t heads, dim, vdim;
-  const float *powers = nullptr;   // [heads][kLightningChunk + 1]: decay^0, decay^1, ...
+  const float *powers = nullptr;   // [heads][kLightningChunk + 1]: decay^0, decay^1, ...; null: `channel` applies
+  ChannelDecay channel;
+  float q_scale = 1.0f;
   float *state = nullptr;
   const void *qkv = nullptr;       // [row][ld]: q (heads x dim) | k (heads x dim) | v (heads x vdim), f32 or bf16
   int32_t half = 0;
@@ -154,12 +216,20 @@ struct LightningArgs {
   const int32_t *positions = nullptr, *slots = nullptr;
   int32_t rows = 0;
   int32_t one_sequence = 0;        // 1: the rows are consecutive tokens of one sequence; 0: one token of each row's own
+  // 1: the inputs were complete before the predecessor let this kernel start; it waits for the predecessor only at its end
+  int32_t late_wait = 0;
 };
 constexpr int kLightningChunk = 64;
 bool lightning_shape_ok(int32_t heads, int32_t dim, int32_t vdim);
 int32_t launch_lightning_steps(const LightningArgs &a, bool pdl, cudaStream_t s);   // token after token
 bool lightning_chunk_fits(const LightningArgs &a);
 int32_t launch_lightning_chunks(const LightningArgs &a, bool pdl, cudaStream_t s);  // 64 tokens at a time on the tensor cores
+
+// gated_linear.cu: the recurrence with a decay per channel, 64 tokens at a time on the tensor cores (f32 rows of one sequence)
+bool gated_shape_ok(int32_t heads, int32_t dim, int32_t vdim, int32_t rank);
+bool gated_chunk_fits(int32_t dim, int32_t rank);
+int64_t gated_scratch_bytes(int32_t heads, int32_t dim, int32_t vdim, int64_t rows);
+int32_t launch_gated_chunks(const LightningArgs &a, void *scratch, bool pdl, cudaStream_t s);
 
 #ifdef __CUDACC__
 
@@ -188,7 +258,24 @@ inline int32_t allow_smem(K k, size_t bytes) {
 __device__ __forceinline__ void pdl_launch() { asm volatile("griddepcontrol.launch_dependents;"); }
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 
+__device__ __forceinline__ void cluster_sync() {
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+__device__ __forceinline__ float ld_peer(uint32_t local_addr, uint32_t rank) {
+  uint32_t a;
+  float v;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(local_addr), "r"(rank));
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
+  return v;
+}
+__device__ __forceinline__ void cp16(void *dst, const void *src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
+// log(sigmoid(z)) / tau
+__device__ __forceinline__ float log_decay(float z, float inv_tau) { return (fminf(z, 0.0f) - log1pf(expf(-fabsf(z)))) * inv_tau; }
 __device__ __forceinline__ float lin_activate(float v, int act, bool in_range) {
   if (act == kActSilu && in_range) return v * sigmoid_f(v);
   if (act == kActRelu2) {
@@ -281,13 +368,50 @@ __device__ __forceinline__ void layer_norm_cta(float *u, int n, const float *w, 
   for (int i = threadIdx.x; i < n; i += blockDim.x) u[i] = (u[i] - mean) * r * w[i] + b[i];
 }
 
+// x + y' of a single stream (see StreamMix).
+__device__ __forceinline__ void post_norm_update(const StreamMix &m, int64_t row, float *u, float *red, bool store) {
+  const float *x = m.x_in + row * m.width, *y = m.y + row * m.width;
+  float *xo = store && m.x_out ? m.x_out + row * m.width : nullptr;
+  if (m.y2) {
+    const float *z = m.y2 + row * m.width;
+    float sy = 0.0f, sz = 0.0f;
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) {
+      sy = fmaf(y[i], y[i], sy);
+      sz = fmaf(z[i], z[i], sz);
+    }
+    const float ry = 1.0f / sqrtf(cta_total(sy, red) / (float)m.width + m.eps), rz = 1.0f / sqrtf(cta_total(sz, red) / (float)m.width + m.eps);
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = 0.5f * (y[i] * ry * m.y_norm[i] + z[i] * rz * m.y2_norm[i]);
+  } else {
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = y[i];
+  }
+  float r = 1.0f;
+  if (m.out_norm) {
+    float s = 0.0f;
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) s = fmaf(u[i], u[i], s);
+    r = 1.0f / sqrtf(cta_total(s, red) / (float)m.width + m.eps);
+  }
+  for (int i = threadIdx.x; i < m.width; i += blockDim.x) {
+    const float v = x[i] + u[i] * r * (m.out_norm ? m.out_norm[i] : 1.0f);
+    if (xo) xo[i] = v;
+    u[i] = v;
+  }
+}
+
+// u / rms(u) * w in place over the CTA.
+__device__ __forceinline__ void rms_norm_cta(float *u, int n, const float *w, float eps, float *red) {
+  float s = 0.0f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) s = fmaf(u[i], u[i], s);
+  const float r = 1.0f / sqrtf(cta_total(s, red) / (float)n + eps);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) u[i] = u[i] * r * w[i];
+}
+
 // The whole boundary for one row; the result is left in u[width] (shared memory; each thread holds its own stride).
 __device__ __forceinline__ void stream_mix_row(const StreamMix &m, int r, float *u, float *red, bool store) {
   const int64_t row = m.row_map ? m.row_map[r] : r;
   if (m.embed) {
     const bf16 *e = m.embed + (int64_t)m.tokens[row] * m.embed_ld;
-    for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = __bfloat162float(e[i]);
-    layer_norm_cta(u, m.width, m.enorm_w, m.enorm_b, m.eps, red);
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = m.embed_scale * __bfloat162float(e[i]);
+    if (m.enorm_w) layer_norm_cta(u, m.width, m.enorm_w, m.enorm_b, m.eps, red);
     float in = 0.0f;
     for (int s = 0; s < m.streams; ++s) in += m.in ? m.in[s] : 1.0f;
     for (int i = threadIdx.x; i < m.width; i += blockDim.x) {
@@ -296,6 +420,8 @@ __device__ __forceinline__ void stream_mix_row(const StreamMix &m, int r, float 
         for (int s = 0; s < m.streams; ++s) m.x_out[(row * m.streams + s) * m.width + i] = x;
       u[i] = in * x;
     }
+  } else if (!m.mix) {
+    post_norm_update(m, row, u, red, store);
   } else {
     switch (m.streams) {
       case 1: stream_update<1>(m, row, u, store); break;
@@ -305,7 +431,8 @@ __device__ __forceinline__ void stream_mix_row(const StreamMix &m, int r, float 
       default: stream_update_many(m, row, u, store); break;
     }
   }
-  if (m.norm_w) layer_norm_cta(u, m.width, m.norm_w, m.norm_b, m.eps, red);
+  if (m.norm_b) layer_norm_cta(u, m.width, m.norm_w, m.norm_b, m.eps, red);
+  else if (m.norm_w) rms_norm_cta(u, m.width, m.norm_w, m.eps, red);
 }
 
 #endif  // __CUDACC__

@@ -1,10 +1,11 @@
-// Linear attention with a fixed decay per head (lightning attention): per head
-//   S_t = decay S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t
-// with the state S [dim][vdim] in 32-bit, one per sequence slot.  A sequence starts from zero: the kernels ignore what
+// Linear attention, per head
+//   S_t = diag(decay_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t
+// with the state S [dim][vdim] in 32-bit, one per sequence slot, and the decay either fixed per head (lightning attention)
+// or computed per token and key channel (gated linear attention).  A sequence starts from zero: the kernels ignore what
 // the slot holds when a row's position is 0, so a slot can be handed to the next sequence as it is.
 //
-// lightning_steps_kernel: token after token, the state in registers (32 value columns per CTA).
-// lightning_chunk_kernel: 64 tokens at a time.  With the tokens of a chunk numbered i, j = 0..63,
+// linear_steps_kernel: token after token, the state in registers (32 value columns per CTA), either decay.
+// lightning_chunk_kernel: the fixed decay, 64 tokens at a time.  With the tokens of a chunk numbered i, j = 0..63,
 //   O = (Q K^T * [decay^(i-j), j <= i]) V + diag(decay^(i+1)) Q S,   S' = decay^64 S + K^T diag(decay^(63-j)) V.
 // Q, K, V are bfloat16; the scores, the scaled values and the state enter the tensor cores as two bfloat16 terms each.
 #include "layered.cuh"
@@ -16,38 +17,65 @@ namespace {
 
 constexpr int kStepThreads = 256, kStepCols = 32, kStepGroups = kStepThreads / kStepCols;
 
-template <int DPT>
-__global__ void __launch_bounds__(kStepThreads) lightning_steps_kernel(const LightningArgs a) {
-  extern __shared__ float sm[];
-  float *qs = sm, *ks = sm + a.dim;                   // this row's q and k of the head
+// shared memory: q, k and, with a decay per channel, the decays of this row and the head's decay weights [dim][pad]
+__host__ __device__ inline int decay_ld(int rank) { return ((rank + 7) & ~7) + 8; }
+inline size_t steps_smem(const LightningArgs &a) {
+  return a.powers ? (size_t)2 * a.dim * 4 : (size_t)((3 * a.dim + 3) & ~3) * 4 + (size_t)a.dim * decay_ld(a.channel.w.cols) * 2;
+}
+
+// Activations may have been written just before this kernel started (late_wait): they are read past the L1 cache.
+__device__ __forceinline__ float act_load_cg(const void *p, int half, int64_t i) {
+  if (half) return bf16_lo(__ldcg(reinterpret_cast<const unsigned short *>(p) + i));
+  return __ldcg(static_cast<const float *>(p) + i);
+}
+
+template <int DPT, bool CHANNEL>
+__global__ void __launch_bounds__(kStepThreads) linear_steps_kernel(const LightningArgs a) {
+  extern __shared__ __align__(16) float sm[];
+  float *qs = sm, *ks = sm + a.dim, *al = ks + a.dim;  // this row's q, k and decays of the head
   __shared__ float red[kStepGroups][kStepCols];
-  pdl_launch();
-  pdl_wait();
   const int h = blockIdx.x, c = threadIdx.x % kStepCols, g = threadIdx.x / kStepCols;
+  const int rank = CHANNEL ? a.channel.w.cols : 0, wl = decay_ld(rank);
+  bf16 *w = reinterpret_cast<bf16 *>(sm + ((3 * a.dim + 3) & ~3));
+  pdl_launch();
+  if (CHANNEL) {  // weights depend on no earlier kernel
+    const int units = (int)a.channel.w.ld / 8;
+    for (int i = threadIdx.x; i < a.dim * units; i += kStepThreads)
+      *reinterpret_cast<uint4 *>(w + (i / units) * wl + (i % units) * 8) =
+          *reinterpret_cast<const uint4 *>(a.channel.w.w + (int64_t)(h * a.dim + i / units) * a.channel.w.ld + (i % units) * 8);
+  }
+  if (!a.late_wait) pdl_wait();
   const int col = blockIdx.y * kStepCols + c;
   const bool live = col < a.vdim;
   const int r0 = a.one_sequence ? 0 : blockIdx.z, n = a.one_sequence ? a.rows : 1;
   float *st = a.state + (((int64_t)a.slots[r0] * a.heads + h) * a.dim) * a.vdim + col;
-  const float decay = a.powers[(int64_t)h * (kLightningChunk + 1) + 1];
+  const float decay = CHANNEL ? 0.0f : a.powers[(int64_t)h * (kLightningChunk + 1) + 1];
   const bool fresh = a.positions[r0] == 0;
   const int d0 = g * DPT;  // this thread's rows of the state
   float s[DPT];
 #pragma unroll
-  for (int j = 0; j < DPT; ++j) s[j] = live && !fresh && d0 + j < a.dim ? st[(int64_t)(d0 + j) * a.vdim] : 0.0f;
+  for (int j = 0; j < DPT; ++j) s[j] = live && !fresh && d0 + j < a.dim ? __ldcg(st + (int64_t)(d0 + j) * a.vdim) : 0.0f;
   const int64_t hd = (int64_t)a.heads * a.dim;
+  if (CHANNEL) __syncthreads();
   for (int r = r0; r < r0 + n; ++r) {
     const int64_t row = (int64_t)r * a.ld;
     for (int i = threadIdx.x; i < a.dim; i += kStepThreads) {
-      qs[i] = act_load(a.qkv, a.half, row + h * a.dim + i);
-      ks[i] = act_load(a.qkv, a.half, row + hd + h * a.dim + i);
+      qs[i] = a.q_scale * act_load_cg(a.qkv, a.half, row + h * a.dim + i);
+      ks[i] = act_load_cg(a.qkv, a.half, row + hd + h * a.dim + i);
+      if (CHANNEL) {
+        float z = 0.0f;
+#pragma unroll 8
+        for (int j = 0; j < rank; ++j) z = fmaf(__bfloat162float(w[i * wl + j]), __ldcg(a.channel.x + row + j), z);
+        al[i] = expf(log_decay(z + a.channel.b[h * a.dim + i], a.channel.inv_tau));
+      }
     }
-    const float v = live ? act_load(a.qkv, a.half, row + 2 * hd + h * a.vdim + col) : 0.0f;
+    const float v = live ? act_load_cg(a.qkv, a.half, row + 2 * hd + h * a.vdim + col) : 0.0f;
     __syncthreads();
     float o = 0.0f;
 #pragma unroll
     for (int j = 0; j < DPT; ++j)
       if (d0 + j < a.dim) {
-        s[j] = fmaf(decay, s[j], ks[d0 + j] * v);
+        s[j] = fmaf(CHANNEL ? al[d0 + j] : decay, s[j], ks[d0 + j] * v);
         o = fmaf(s[j], qs[d0 + j], o);
       }
     red[g][c] = o;
@@ -62,6 +90,7 @@ __global__ void __launch_bounds__(kStepThreads) lightning_steps_kernel(const Lig
 #pragma unroll
   for (int j = 0; j < DPT; ++j)
     if (live && d0 + j < a.dim) st[(int64_t)(d0 + j) * a.vdim] = s[j];
+  if (a.late_wait) pdl_wait();
 }
 
 constexpr int kC = kLightningChunk, kChunkCols = 32, kChunkThreads = 128;
@@ -72,9 +101,6 @@ __host__ __device__ inline int chunk_smem(int dp) {
   return 2 * (2 * kC * (dp + 8) + kC * (kChunkCols + 8)) * 2 + 2 * kC * (kChunkCols + 8) * 2 + 2 * dp * (kChunkCols + 8) * 2 + (kC + 1) * 4 + 16;
 }
 
-__device__ __forceinline__ void cp16(void *dst, const void *src, bool live) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
-}
 
 // MT: 16-row tiles of the state per warp (dim <= 64 * MT)
 template <int MT>
@@ -271,8 +297,14 @@ __global__ void __launch_bounds__(kChunkThreads) lightning_chunk_kernel(const Li
 
 template <int DPT>
 int32_t steps(const LightningArgs &a, bool pdl, cudaStream_t s) {
-  return launch_kernel(lightning_steps_kernel<DPT>, dim3(a.heads, (a.vdim + kStepCols - 1) / kStepCols, a.one_sequence ? 1 : a.rows), dim3(kStepThreads),
-                       (size_t)2 * a.dim * 4, pdl, s, a);
+  const dim3 grid(a.heads, (a.vdim + kStepCols - 1) / kStepCols, a.one_sequence ? 1 : a.rows);
+  if (a.powers) return launch_kernel(linear_steps_kernel<DPT, false>, grid, dim3(kStepThreads), steps_smem(a), pdl, s, a);
+  static bool ready = false;
+  if (!ready) {
+    CMLD_TRY(allow_smem(linear_steps_kernel<DPT, true>, 160 * 1024));
+    ready = true;
+  }
+  return launch_kernel(linear_steps_kernel<DPT, true>, grid, dim3(kStepThreads), steps_smem(a), pdl, s, a);
 }
 
 template <int MT>
@@ -298,7 +330,11 @@ int32_t launch_lightning_steps(const LightningArgs &a, bool pdl, cudaStream_t s)
   return fail(CMLD_ERR_SHAPE, "lightning attention: %d key dimensions, at most 512", a.dim);
 }
 
-bool lightning_chunk_fits(const LightningArgs &a) { return a.half && a.one_sequence && a.dim <= 256; }
+bool gated_shape_ok(int32_t heads, int32_t dim, int32_t vdim, int32_t rank) {
+  return lightning_shape_ok(heads, dim, vdim) && rank >= 1 && (size_t)dim * (12 + decay_ld(rank) * 2) + 16 <= 160 * 1024;
+}
+
+bool lightning_chunk_fits(const LightningArgs &a) { return a.powers && a.half && a.one_sequence && a.dim <= 256; }
 
 int32_t launch_lightning_chunks(const LightningArgs &a, bool pdl, cudaStream_t s) {
   if (a.dim <= 64) return chunks<1>(a, pdl, s);

@@ -40,13 +40,17 @@ __global__ void __launch_bounds__(256) lin_f32_kernel(const LinArgs a) {
 #pragma unroll
     for (int m = 0; m < 4; ++m) {
       const int row = n0 + tn + n, o = m0 + tm + m;
-      if (row < a.rows && o < a.w.rows) act_store(a.out, a.out_half, (int64_t)row * a.out_ld + o, lin_activate(acc[n][m], a.act, o < a.act_rows));
+      if (row >= a.rows || o >= a.w.rows) continue;
+      acc[n][m] = fmaf(acc[n][m], a.scale, a.bias ? a.bias[o] : 0.0f);
+      if (a.act != kActSwiGlu) act_store(a.out, a.out_half, (int64_t)row * a.out_ld + o, lin_activate(acc[n][m], a.act, o < a.act_rows));
+      else if (m & 1) act_store(a.out, a.out_half, (int64_t)row * a.out_ld + (o >> 1), silu_f(acc[n][m - 1]) * acc[n][m]);
     }
 }
 
 }  // namespace
 
 int32_t launch_lin_f32(const LinArgs &a, cudaStream_t s) {
+  if (a.act == kActSwiGlu && a.w.rows % 2) return fail(CMLD_ERR_SHAPE, "linear: gated pairs need an even number of rows");
   return launch_kernel(lin_f32_kernel, dim3((a.w.rows + kT - 1) / kT, (a.rows + kT - 1) / kT), dim3(256), 0, false, s, a);
 }
 

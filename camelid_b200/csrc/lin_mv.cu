@@ -3,7 +3,8 @@
 // Persistent grid, one CTA of 16 warps per SM.  A warp owns one or two output rows at a time; a lane reads 16 bytes
 // (eight weights) of each, four steps of 256 columns in flight.  The first weights are asked for before the kernel
 // waits for its predecessor (weights never depend on earlier kernels), then every CTA prepares the operand itself:
-// the hyper-connection boundary with its layer norm, an RMS norm, an RMS norm times a sigmoid gate, or a plain copy.
+// the boundary between sublayers, an RMS norm (with a sigmoid gate, or over groups of columns with a SiLU gate), or a plain
+// copy.  Two products that do not depend on each other can share a launch: the first `n_first` CTAs work on one.
 // The prepared rows sit in shared memory as f32 in two planes (values 8j..8j+3 and 8j+4..8j+7), so that the lanes of
 // a warp read consecutive 16-byte words.
 #include "layered.cuh"
@@ -18,15 +19,15 @@ constexpr size_t kMvMaxSmem = 220 * 1024;
 __host__ __device__ constexpr int mv_kpad(int cols) { return (cols + 255) & ~255; }
 
 template <int R, int ROWS>
-__global__ void __launch_bounds__(kMvThreads, 1) lin_mv_kernel(const LinMvArgs a) {
+__device__ __forceinline__ void lin_mv_cta(const LinMvArgs &a, int cta, int ctas) {
   extern __shared__ float smem[];
   __shared__ float red[kMvThreads / 32];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int K = a.w.cols, kp = mv_kpad(K), half = kp / 2, nit = kp / 256;
   float *xs = smem;              // [R][2][kp / 2]
   float *u = smem + R * kp;      // one row in plain order
-  const int groups = (a.w.rows + ROWS - 1) / ROWS, stride = gridDim.x * (kMvThreads / 32);
-  int g = blockIdx.x + gridDim.x * warp;
+  const int groups = (a.w.rows + ROWS - 1) / ROWS, stride = ctas * (kMvThreads / 32);
+  int g = cta + ctas * warp;
 
   uint4 w[ROWS][kMvUnroll];
   auto fetch = [&](int grp, int it0) {
@@ -49,8 +50,18 @@ __global__ void __launch_bounds__(kMvThreads, 1) lin_mv_kernel(const LinMvArgs a
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     if (a.prologue == kProStreams) {
-      stream_mix_row(a.mix, r, u, red, blockIdx.x == 0);
+      stream_mix_row(a.mix, r, u, red, cta == 0);
       for (int i = tid; i < kp; i += kMvThreads) put(r, i, i < K ? u[i] : 0.0f);
+    } else if (a.prologue == kProRmsGroups) {
+      // a warp per group of columns
+      const float *x = a.x + r * a.x_ld, *gate = a.gate + r * a.gate_ld;
+      for (int c0 = warp * a.group; c0 < K; c0 += (kMvThreads / 32) * a.group) {
+        float s = 0.0f;
+        for (int i = lane; i < a.group; i += 32) s = fmaf(x[c0 + i], x[c0 + i], s);
+        const float inv = 1.0f / sqrtf(warp_sum(s) / (float)a.group + a.eps);
+        for (int i = lane; i < a.group; i += 32) put(r, c0 + i, x[c0 + i] * inv * a.norm_w[i] * silu_f(gate[c0 + i]));
+      }
+      for (int i = K + tid; i < kp; i += kMvThreads) put(r, i, 0.0f);
     } else {
       const float *x = a.x + r * a.x_ld;
       float inv = 1.0f;
@@ -106,17 +117,38 @@ __global__ void __launch_bounds__(kMvThreads, 1) lin_mv_kernel(const LinMvArgs a
       }
     }
 #pragma unroll
-    for (int i = 0; i < ROWS; ++i)
+    for (int r = 0; r < R; ++r) {
+      float v[ROWS];
 #pragma unroll
-      for (int r = 0; r < R; ++r) {
-        const float v = warp_sum(acc[i][r]);
+      for (int i = 0; i < ROWS; ++i) {
         const int row = g * ROWS + i;
-        if (lane == 0 && row < a.w.rows) a.y[r * a.y_ld + row] = lin_activate(v, a.act, row < a.act_rows);
+        v[i] = fmaf(warp_sum(acc[i][r]), a.scale, a.bias && row < a.w.rows ? a.bias[row] : 0.0f);
+        if (lane == 0 && row < a.w.rows && a.act != kActSwiGlu) a.y[r * a.y_ld + row] = lin_activate(v[i], a.act, row < a.act_rows);
       }
+      if (ROWS == 2 && lane == 0 && a.act == kActSwiGlu) a.y[r * a.y_ld + g] = silu_f(v[0]) * v[ROWS - 1];
+    }
   }
 }
 
+template <int R, int ROWS>
+__global__ void __launch_bounds__(kMvThreads, 1) lin_mv_kernel(const __grid_constant__ LinMvArgs a) {
+  lin_mv_cta<R, ROWS>(a, blockIdx.x, gridDim.x);
+}
+
+template <int R, int ROWS>
+__global__ void __launch_bounds__(kMvThreads, 1) lin_mv_pair_kernel(const __grid_constant__ LinMvArgs a, const __grid_constant__ LinMvArgs b, int n_first) {
+  if ((int)blockIdx.x < n_first) lin_mv_cta<R, ROWS>(a, blockIdx.x, n_first);
+  else lin_mv_cta<R, ROWS>(b, blockIdx.x - n_first, gridDim.x - n_first);
+}
+
 size_t mv_smem(int cols, int batch) { return (size_t)(batch + 1) * mv_kpad(cols) * 4; }
+
+int mv_sms() {
+  int dev = 0, sms = 148;
+  cudaGetDevice(&dev);
+  cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+  return sms;
+}
 
 template <int R, int ROWS>
 int32_t mv_launch(const LinMvArgs &a, bool pdl, cudaStream_t s) {
@@ -126,11 +158,22 @@ int32_t mv_launch(const LinMvArgs &a, bool pdl, cudaStream_t s) {
     prefer_max_smem_carveout(lin_mv_kernel<R, ROWS>);
     ready = true;
   }
-  int dev = 0, sms = 148;
-  cudaGetDevice(&dev);
-  cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   const int groups = (a.w.rows + ROWS - 1) / ROWS;
-  return launch_kernel(lin_mv_kernel<R, ROWS>, dim3(std::min(groups, sms)), dim3(kMvThreads), mv_smem(a.w.cols, R), pdl, s, a);
+  return launch_kernel(lin_mv_kernel<R, ROWS>, dim3(std::min(groups, mv_sms())), dim3(kMvThreads), mv_smem(a.w.cols, R), pdl, s, a);
+}
+
+template <int R, int ROWS>
+int32_t mv_launch_pair(const LinMvArgs &a, const LinMvArgs &b, bool pdl, cudaStream_t s) {
+  static bool ready = false;
+  if (!ready) {
+    CMLD_TRY(allow_smem(lin_mv_pair_kernel<R, ROWS>, kMvMaxSmem));
+    prefer_max_smem_carveout(lin_mv_pair_kernel<R, ROWS>);
+    ready = true;
+  }
+  const int sms = mv_sms();
+  const double wa = (double)a.w.rows * a.w.ld, wb = (double)b.w.rows * b.w.ld;
+  const int first = std::min(sms - 1, std::max(1, (int)(sms * wa / (wa + wb) + 0.5)));
+  return launch_kernel(lin_mv_pair_kernel<R, ROWS>, dim3(sms), dim3(kMvThreads), mv_smem(std::max(a.w.cols, b.w.cols), R), pdl, s, a, b, first);
 }
 
 }  // namespace
@@ -139,10 +182,20 @@ bool lin_mv_fits(int32_t cols, int32_t batch) { return batch >= 1 && batch <= 2 
 
 int32_t launch_lin_mv(const LinMvArgs &a, bool pdl, cudaStream_t s) {
   if (!lin_mv_fits(a.w.cols, a.batch)) return fail(CMLD_ERR_SHAPE, "matrix-vector product of %d columns and %d rows does not fit", a.w.cols, a.batch);
+  if (a.act == kActSwiGlu) {
+    if (a.w.rows % 2) return fail(CMLD_ERR_SHAPE, "linear: gated pairs need an even number of rows");
+    return a.batch == 1 ? mv_launch<1, 2>(a, pdl, s) : mv_launch<2, 2>(a, pdl, s);
+  }
   // one output row per warp while that is needed to give every warp of the machine something to do
   const bool single = a.w.rows <= 148 * (kMvThreads / 32) * 3 / 2;
   if (a.batch == 1) return single ? mv_launch<1, 1>(a, pdl, s) : mv_launch<1, 2>(a, pdl, s);
   return single ? mv_launch<2, 1>(a, pdl, s) : mv_launch<2, 2>(a, pdl, s);
+}
+
+int32_t launch_lin_mv_pair(const LinMvArgs &a, const LinMvArgs &b, bool pdl, cudaStream_t s) {
+  if (a.batch != b.batch || a.act == kActSwiGlu || b.act == kActSwiGlu || !lin_mv_fits(a.w.cols, a.batch) || !lin_mv_fits(b.w.cols, b.batch))
+    return fail(CMLD_ERR_SHAPE, "a pair of matrix-vector products does not fit one launch");
+  return a.batch == 1 ? mv_launch_pair<1, 1>(a, b, pdl, s) : mv_launch_pair<2, 1>(a, b, pdl, s);
 }
 
 }  // namespace cmld

@@ -1,5 +1,5 @@
-// Linear layers on the 5th-generation tensor cores: out[r][o] = act(sum_k w[o][k] x[r][k]), bfloat16 operands, f32
-// accumulators in tensor memory.
+// Linear layers on the 5th-generation tensor cores: out[r][o] = act(scale * sum_k w[o][k] x[r][k] + bias[o]), bfloat16
+// operands, f32 accumulators in tensor memory.
 //
 // The weights are operand A (tiles of 128 output rows), the activation rows operand B (tiles of BN rows), both K-major
 // and brought by TMA in 128-byte-swizzled boxes of 64 columns.  Persistent CTAs, one per SM; warp roles:
@@ -34,6 +34,8 @@ struct TcLinArgs {
   void *out;
   int64_t out_ld;
   int32_t act, act_rows;
+  const float *bias;
+  float scale;
   int32_t *status;
 };
 
@@ -89,17 +91,6 @@ __device__ __forceinline__ void tmem_ld16(uint32_t t, float (&r)[16]) {
       : "r"(t)
       : "memory");
 }
-__device__ __forceinline__ void cluster_sync() {
-  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-__device__ __forceinline__ float ld_peer(uint32_t local_addr, uint32_t rank) {
-  uint32_t a;
-  float v;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(local_addr), "r"(rank));
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(a) : "memory");
-  return v;
-}
-
 __device__ __forceinline__ void put(float *p, float v) { *p = v; }
 __device__ __forceinline__ void put(bf16 *p, float v) { *p = __float2bfloat16_rn(v); }
 
@@ -205,8 +196,10 @@ __global__ void __launch_bounds__(kThreads, 1)
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const int n_live = min(BN, a.n_rows - n0);
       float *part = reinterpret_cast<float *>(smem);  // [BN][128]: the operand stages are free by now
-      const bool silu = a.act == kActSilu && o < a.act_rows, relu2 = a.act == kActRelu2;
-      OutT *p = out + (int64_t)(n0 + 16 * half) * a.out_ld + o;
+      const bool silu = a.act == kActSilu && o < a.act_rows, relu2 = a.act == kActRelu2, swiglu = a.act == kActSwiGlu;
+      const float bias = a.bias && o < a.m_rows ? a.bias[o] : 0.0f;
+      const bool odd = lane & 1;
+      OutT *p = out + (int64_t)(n0 + 16 * half) * a.out_ld + (swiglu ? o >> 1 : o);
 #pragma unroll 1
       for (int c = 16 * half; c < n_live; c += 32, p += 32 * a.out_ld) {
         float r[16];
@@ -221,9 +214,23 @@ __global__ void __launch_bounds__(kThreads, 1)
           for (int j = 0; j < 16; ++j) part[(c + j) * kBM + quarter * 32 + lane] = r[j];
           continue;
         }
+#pragma unroll
+        for (int j = 0; j < 16; ++j) r[j] = fmaf(r[j], a.scale, bias);
+        if (swiglu) {
+          // a lane holds the gate (even rows) or the other factor (odd rows); of two columns the even lane finishes one,
+          // the odd lane the other
+          OutT *w = p + (odd ? a.out_ld : 0);
+#pragma unroll
+          for (int j = 0; j < 16; j += 2, w += 2 * a.out_ld) {
+            const float t = __shfl_xor_sync(0xffffffffu, odd ? r[j] : r[j + 1], 1);
+            const float v = odd ? silu_f(t) * r[j + 1] : silu_f(r[j]) * t;
+            if (o < a.m_rows && c + j + (odd ? 1 : 0) < n_live) put(w, v);
+          }
+          continue;
+        }
         if (silu) {
 #pragma unroll
-          for (int j = 0; j < 16; ++j) r[j] = r[j] * sigmoid_f(r[j]);
+          for (int j = 0; j < 16; ++j) r[j] = silu_f(r[j]);
         } else if (relu2) {
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -255,13 +262,22 @@ __global__ void __launch_bounds__(kThreads, 1)
     if (first < a.tiles && !*abort_flag) {
       OutT *out = static_cast<OutT *>(a.out);
       const int m0 = (first % a.tiles_m) * kBM, n0 = (first / a.tiles_m) * BN, n_live = min(BN, a.n_rows - n0);
-      for (int e = rank * kThreads + tid; e < n_live * kBM; e += a.split * kThreads) {
-        const int o = m0 + e % kBM, n = e / kBM;
+      auto total = [&](int e, int o) {
         float v = 0.0f;
         for (int p = 0; p < a.split; ++p) v += ld_peer(base + 4u * e, p);
-        if (o < a.m_rows) {
-          v = lin_activate(v, a.act, o < a.act_rows);
-          put(out + (int64_t)(n0 + n) * a.out_ld + o, v);
+        return fmaf(v, a.scale, a.bias && o < a.m_rows ? a.bias[o] : 0.0f);
+      };
+      if (a.act == kActSwiGlu) {
+        for (int e = 2 * (rank * kThreads + tid); e < n_live * kBM; e += 2 * a.split * kThreads) {
+          const int o = m0 + e % kBM, n = e / kBM;
+          const float v = silu_f(total(e, o)) * total(e + 1, o + 1);
+          if (o < a.m_rows) put(out + (int64_t)(n0 + n) * a.out_ld + (o >> 1), v);
+        }
+      } else {
+        for (int e = rank * kThreads + tid; e < n_live * kBM; e += a.split * kThreads) {
+          const int o = m0 + e % kBM, n = e / kBM;
+          const float v = total(e, o);
+          if (o < a.m_rows) put(out + (int64_t)(n0 + n) * a.out_ld + o, lin_activate(v, a.act, o < a.act_rows));
         }
       }
     }
@@ -318,6 +334,8 @@ int32_t launch_bn(const LinArgs &L, int32_t sms, int32_t *status, bool pdl, cuda
   a.out_ld = L.out_ld;
   a.act = L.act;
   a.act_rows = L.act_rows;
+  a.bias = L.bias;
+  a.scale = L.scale;
   a.status = status;
   cudaLaunchConfig_t cfg{};
   cfg.gridDim = dim3((unsigned)(a.split > 1 ? a.tiles * a.split : std::min(a.tiles, sms)));
@@ -356,6 +374,7 @@ int32_t launch_out(const LinArgs &a, int32_t sms, int32_t *status, bool pdl, cud
 
 int32_t launch_lin_tc5(const LinArgs &a, int32_t sms, int32_t *status, bool pdl, cudaStream_t s) {
   if (a.rows < 1) return CMLD_OK;
+  if (a.act == kActSwiGlu && a.w.rows % 2) return fail(CMLD_ERR_SHAPE, "linear: gated pairs need an even number of rows");
   return a.out_half ? launch_out<bf16>(a, sms, status, pdl, s) : launch_out<float>(a, sms, status, pdl, s);
 }
 

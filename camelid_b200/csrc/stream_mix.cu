@@ -1,5 +1,5 @@
-// Row operations of layered models: the hyper-connection boundary (stream update, read-out, layer norm), the embedding
-// with its norm, RMS norm with an optional gate.
+// Row operations of layered models: the boundary between sublayers (residual update, read-out, norm), the embedding, RMS
+// norm with an optional gate, over whole rows or over groups of columns.
 #include "layered.cuh"
 
 namespace cmld {
@@ -46,6 +46,24 @@ __global__ void __launch_bounds__(kMixThreads) rms_rows_kernel(const float *x, i
   }
 }
 
+// A warp per group of columns.
+__global__ void __launch_bounds__(256) rms_groups_kernel(const float *x, int64_t x_ld, const float *w, int groups, int group, float eps, const float *gate,
+                                                         int64_t gate_ld, ActBuf out, int rows) {
+  pdl_launch();
+  pdl_wait();
+  const int64_t unit = blockIdx.x * 8ll + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (unit >= (int64_t)rows * groups) return;
+  const int64_t r = unit / groups, c0 = unit % groups * group;
+  const float *xr = x + r * x_ld + c0, *gr = gate + r * gate_ld + c0;
+  float s = 0.0f;
+#pragma unroll 4
+  for (int i = lane; i < group; i += 32) s = fmaf(xr[i], xr[i], s);
+  const float inv = 1.0f / sqrtf(warp_sum(s) / (float)group + eps);
+#pragma unroll 4
+  for (int i = lane; i < group; i += 32) act_store(out.p, out.half, r * out.ld + c0 + i, xr[i] * inv * w[i] * silu_f(gr[i]));
+}
+
 }  // namespace
 
 int32_t launch_stream_mix(const StreamMix &m, int32_t rows, ActBuf out, bool pdl, cudaStream_t s) {
@@ -63,6 +81,13 @@ int32_t launch_stream_tap(const StreamMix &m, int32_t rows, float *out, cudaStre
 int32_t launch_rms_rows(const float *x, int64_t x_ld, const float *w, int32_t cols, float eps, ActBuf gate, ActBuf out, int32_t rows,
                         bool pdl, cudaStream_t s) {
   return launch_kernel(rms_rows_kernel, dim3(rows), dim3(mix_threads(rows)), 0, pdl, s, x, x_ld, w, cols, eps, gate, out);
+}
+
+int32_t launch_rms_groups(const float *x, int64_t x_ld, const float *w, int32_t cols, int32_t group, float eps, const float *gate, int64_t gate_ld,
+                          ActBuf out, int32_t rows, bool pdl, cudaStream_t s) {
+  const int groups = cols / group;
+  return launch_kernel(rms_groups_kernel, dim3((unsigned)(((int64_t)rows * groups + 7) / 8)), dim3(256), 0, pdl, s, x, x_ld, w, groups, group, eps, gate,
+                       gate_ld, out, rows);
 }
 
 }  // namespace cmld

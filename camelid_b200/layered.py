@@ -6,21 +6,55 @@ from dataclasses import dataclass, field
 
 import numpy as np
 
-from ._lib import LayerDesc, LayeredConfig, check, lib
+from ._lib import GatedDesc, LayerDesc, LayeredConfig, WindowDesc, check, lib
 from .engine import BF16, F32, TokenEngine, _np_ptr
 
-LATENT, LIGHTNING = 1, 2
+LATENT, LIGHTNING, PARALLEL = 1, 2, 3
+RELU2, SWIGLU = 0, 1
+STREAMS, POST_NORM = 0, 1
 DTYPES = {"bfloat16": BF16, "float32": F32}
 
 
 @dataclass
-class LayerSpec:
-    """One layer: a mixer and, unless ``ff`` is 0, a squared-ReLU feed-forward of that width."""
-    type: int
+class WindowSpec:
+    """Attention with grouped heads: a query sees ``window`` tokens, itself included (0: every earlier one); the first
+    ``rot_dims`` dimensions turn, with YaRN-scaled frequencies if ``rot_factor`` is given."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    window: int
+    scale: float
+    rot_dims: int = 0
+    rot_base: float = 0.0
+    rot_factor: float = 0.0
+    rot_original: float = 0.0
+    rot_fast: float = 0.0
+    rot_slow: float = 0.0
+
+
+@dataclass
+class GatedSpec:
+    """Linear attention with a decay per key channel, from a projection of rank ``rank``."""
     heads: int
     dim: int
     vdim: int
+    rank: int
+    tau: float
+
+
+@dataclass
+class LayerSpec:
+    """One layer: a mixer and, unless ``ff`` is 0, a feed-forward of that width (``mlp``: its kind).  A parallel layer's
+    sizes are in ``window`` and ``gated``."""
+    type: int
+    heads: int = 0
+    dim: int = 0
+    vdim: int = 0
     ff: int = 0
+    mlp: int = RELU2
+    window: WindowSpec | None = None
+    gated: GatedSpec | None = None
     # latent attention
     q_rank: int = 0
     kv_rank: int = 0
@@ -40,6 +74,9 @@ class LayeredSpec:
     layers: list
     streams: int = 1
     loop: tuple = (0, 0, 1)  # layers start .. stop-1 run `times` times in a row
+    residual: int = STREAMS
+    embed_scale: float = 1.0
+    logit_scale: float = 1.0
 
     @property
     def runs(self) -> list:
@@ -60,7 +97,9 @@ class LayeredEngine(TokenEngine):
     """A layered design on the device.  Sequences live in slots 0..max_seqs-1; a slot's caches and states belong together,
     so a call starts a sequence at position 0 or continues it where it ends (``filled``)."""
 
-    def __init__(self, spec: LayeredSpec, max_pos: int, max_seqs: int = 1, dtype: str = "bfloat16", device: int = -1, flags: int = 0):
+    def __init__(self, spec: LayeredSpec, max_pos: int, max_seqs: int = 1, dtype: str = "bfloat16", device: int = -1, flags: int = 0,
+                 portion: int = 0):
+        """portion: most rows of one step of a prompt (0: the library's own number); windowed caches are sized by it."""
         if dtype not in DTYPES:
             raise ValueError(f"dtype {dtype!r} is not one of {sorted(DTYPES)}")
         self.spec = spec
@@ -68,8 +107,10 @@ class LayeredEngine(TokenEngine):
         arr = (LayerDesc * len(spec.layers))()
         keep = []
         for d, s in zip(arr, spec.layers):
-            for name in ("type", "heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "ff", "scale", "rot_base"):
+            for name in ("type", "heads", "dim", "vdim", "q_rank", "kv_rank", "rot_dim", "rot_dims", "ff", "mlp", "scale", "rot_base"):
                 setattr(d, name, getattr(s, name))
+            if s.type == PARALLEL:
+                d.window, d.gated = WindowDesc(**vars(s.window)), GatedDesc(**vars(s.gated))
             if s.type == LIGHTNING:
                 if len(s.decay) != s.heads:
                     raise ValueError(f"{len(s.decay)} decays for {s.heads} heads")
@@ -78,7 +119,8 @@ class LayeredEngine(TokenEngine):
                 d.decay = dec.ctypes.data_as(C.POINTER(C.c_float))
         c = LayeredConfig(n_layers=len(spec.layers), loop_start=spec.loop[0], loop_stop=spec.loop[1], loop_times=spec.loop[2], streams=spec.streams,
                           width=spec.width, vocab=spec.vocab, max_pos=max_pos, max_seqs=self.cfg.max_seqs, dtype=DTYPES[dtype], device=device,
-                          flags=flags, eps=spec.eps, layers=arr)
+                          flags=flags, residual=spec.residual, portion=portion, eps=spec.eps, embed_scale=spec.embed_scale,
+                          logit_scale=spec.logit_scale, layers=arr)
         h = C.c_void_p()
         check(lib().cmld_engine_create_layered(C.byref(c), C.byref(h)))
         self._h = h.value

@@ -7,7 +7,7 @@ from __future__ import annotations
 import json
 from pathlib import Path
 
-from . import gguf, losarax
+from . import gguf, losarax, tokovik
 
 
 def _load_gguf(path, max_pos, max_seqs, dtype, **kw):
@@ -16,15 +16,18 @@ def _load_gguf(path, max_pos, max_seqs, dtype, **kw):
     return gguf.load_engine(path, max_pos=max_pos, max_seqs=max_seqs, **kw)
 
 
-def _load_losarax(path, max_pos, max_seqs, dtype, **kw):
-    if not max_pos:
-        raise ValueError("this design sets no context length of its own: give max_pos")
-    return losarax.load_engine(path, max_pos, max_seqs, dtype or "bfloat16", **kw)
+def _load_layered(design):
+    def load(path, max_pos, max_seqs, dtype, **kw):
+        if not max_pos:
+            raise ValueError("this design sets no context length of its own: give max_pos")
+        return design.load_engine(path, max_pos, max_seqs, dtype or "bfloat16", **kw)
+
+    return load
 
 
 ARCHITECTURES = {
     "llama": _load_gguf,  # dense llama shapes and Mixtral shapes
-    losarax.ARCHITECTURE: _load_losarax,
+    **{design.ARCHITECTURE: _load_layered(design) for design in (losarax, tokovik)},
 }
 
 

@@ -240,30 +240,60 @@ CMLD_API int32_t cmld_engine_read_kv_layer(cmld_engine *e, int32_t layer, int64_
  * decode_greedy, step_batch without hidden_out, sample_row, last_timing) and weights_ready / max_pos / n_layers;
  * the calls that speak of llama-shaped layers return CMLD_ERR_UNSUPPORTED.
  *
- * The residual is held as `streams` parallel copies x_s.  For each sublayer, with its vectors in, out and matrix mix:
- *   u = sum_s in[s] x_s;  y = sublayer(layernorm(u));  x_t <- sum_s mix[s][t] x_s + out[t] y.
+ * The residual comes in two kinds.  CMLD_RESIDUAL_STREAMS: `streams` parallel copies x_s; for each sublayer, with its vectors
+ * in, out and matrix mix:
+ *   u = sum_s in[s] x_s;  y = sublayer(layernorm(u));  x_t <- sum_s mix[s][t] x_s + out[t] y,
+ * and layer norms (with bias) on the embedding and before the output matrix.  CMLD_RESIDUAL_POST_NORM: one stream,
+ *   x <- x + rmsnorm(sublayer(x)), starting from embed_scale * embedding row, an RMS norm before the output matrix; the
+ * weights of these norms are stored around zero (1 + w is applied).
  * Layers loop_start .. loop_stop-1 run loop_times times in a row with the same weights, each pass with its own cache
  * or state.  A sequence slot holds rows and states that belong together: a call either starts a sequence (position 0) or
  * continues it where it ends (cmld_engine_slot_filled). */
 typedef enum {
   CMLD_LAYER_LATENT = 1,    /* attention over a cached latent and a rotated key part shared by the heads */
-  CMLD_LAYER_LIGHTNING = 2  /* linear attention with a fixed decay per head, RMS-normed and gated */
+  CMLD_LAYER_LIGHTNING = 2, /* linear attention with a fixed decay per head, RMS-normed and gated */
+  CMLD_LAYER_PARALLEL = 3   /* two branches on one input: sliding-window attention with grouped heads, and linear attention with
+                               a decay per key channel; half the sum of their outputs, each RMS-normed over the width */
 } cmld_layer_type;
+typedef enum {
+  CMLD_MLP_RELU2 = 0, /* W_down (max(W_up h, 0)^2) */
+  CMLD_MLP_SWIGLU = 1 /* W_down (silu(W_gate h) * (W_up h)) */
+} cmld_mlp_type;
+typedef enum { CMLD_RESIDUAL_STREAMS = 0, CMLD_RESIDUAL_POST_NORM = 1 } cmld_residual_type;
+/* Attention with grouped heads over a sliding window: projections with bias, RMS norms on queries and keys, rotation of the first
+ * rot_dims dimensions in pairs (i, i + rot_dims / 2).  rot_factor > 0: YaRN-scaled frequencies. */
+typedef struct {
+  int32_t heads, kv_heads, dim, vdim, rot_dims;
+  int32_t window; /* tokens a query sees, itself included; 0 = every earlier one */
+  float scale;    /* factor of the scores */
+  double rot_base, rot_factor, rot_original, rot_fast, rot_slow;
+} cmld_window_desc;
+/* Linear attention with the decay sigmoid(a2 (a1 h) + b)^(1 / tau) per key channel; `rank` rows of a1. */
+typedef struct {
+  int32_t heads, dim, vdim, rank;
+  double tau;
+} cmld_gated_desc;
 typedef struct {
   int32_t type;
-  int32_t heads, dim, vdim;
+  int32_t heads, dim, vdim;                   /* latent, lightning */
   int32_t q_rank, kv_rank, rot_dim, rot_dims; /* latent: rot_dims of the rot_dim values turn, in pairs (2i, 2i + 1) */
-  int32_t ff;                                 /* width of the squared-ReLU feed-forward; 0 = none */
+  int32_t ff;                                 /* width of the feed-forward; 0 = none */
+  int32_t mlp;                                /* cmld_mlp_type */
   float scale;                                /* latent: factor of the scores */
   double rot_base;                            /* latent: pair i turns by position * rot_base^(-2i / rot_dims) */
   const float *decay;                         /* lightning: [heads]; borrowed for the duration of the call */
+  cmld_window_desc window;                    /* parallel */
+  cmld_gated_desc gated;                      /* parallel */
 } cmld_layer_desc;
 typedef struct {
   int32_t n_layers, loop_start, loop_stop, loop_times; /* loop_times 0 or 1: every layer once */
   int32_t streams, width, vocab, max_pos, max_seqs;
   int32_t dtype;  /* CMLD_BF16: bfloat16 products with 32-bit sums, residual, norms, scores and states; CMLD_F32: all 32-bit */
   int32_t device, flags;
+  int32_t residual;  /* cmld_residual_type; POST_NORM has one stream */
+  int32_t portion;   /* rows of one step of a prompt (0 = 2048); a windowed cache holds window + portion - 1 positions */
   float eps;
+  float embed_scale, logit_scale; /* factors of the embedding row and of the logits; 0 = 1 */
   const cmld_layer_desc *layers;
 } cmld_layered_config;
 CMLD_API int32_t cmld_engine_create_layered(const cmld_layered_config *cfg, cmld_engine **out);
@@ -425,11 +455,14 @@ CMLD_API int32_t cmld_attention_decode_noalloc(const float *q_dev, const void *k
 /* The linear layer of layered designs as an operator: out[r][o] = act(sum_k w[o][k] x[r][k]) for n rows of x.
  * kernel 0: matrix-vector form (n <= 2, x f32, out f32); 1: tcgen05 (x bfloat16); 2: FP32 units (x f32).
  * w_dev: bfloat16 [rows][ld], ld = cols rounded up to 8 with zero padding; x_dev rows of the same ld; out_dev [n][rows]
- * bfloat16 if out_bf16 else f32.  act 0 none, 1 SiLU on the first act_rows outputs, 2 square of ReLU.
+ * bfloat16 if out_bf16 else f32.  act 0 none, 1 SiLU on the first act_rows outputs, 2 square of ReLU, 3 SiLU of an even row's
+ * sum times the next row's (out_dev is then [n][rows / 2]).  bias_dev: f32 [rows] added to the sums, or NULL; scale: factor
+ * of the sums.
  * iters > 0: afterwards iters launches are timed (one CUDA-graph replay, CUDA events), the weights visited round-robin
  * through n_copies matrices w_dev + i * rows * ld; *ms_out = mean milliseconds per launch. */
 CMLD_API int32_t cmld_linear(int32_t kernel, const void *w_dev, int64_t rows, int64_t cols, const void *x_dev, int32_t n, void *out_dev,
-                             int32_t out_bf16, int32_t act, int32_t act_rows, int32_t n_copies, int32_t iters, float *ms_out);
+                             int32_t out_bf16, int32_t act, int32_t act_rows, const float *bias_dev, float scale, int32_t n_copies,
+                             int32_t iters, float *ms_out);
 /* Time `iters` back-to-back launches of cmld_gemv with CUDA events around one CUDA-graph replay of
  * them (so the host's enqueue rate is not measured); the weights are `n_copies` distinct matrices
  * visited round-robin so that the stream comes from HBM when their total exceeds the L2.

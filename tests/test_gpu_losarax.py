@@ -72,7 +72,7 @@ def linear(cm, kernel, w, x, out_bf16=False, act=0, act_rows=0):
     wd, xd = device_rows(w, True), device_rows(x, kernel == 1)
     out = DeviceBuffer(x.shape[0] * w.shape[0] * (2 if out_bf16 else 4))
     ms = C.c_float(0)
-    ok(cm.lib().cmld_linear(kernel, wd.ptr, w.shape[0], w.shape[1], xd.ptr, x.shape[0], out.ptr, int(out_bf16), act, act_rows, 1, 0, C.byref(ms)))
+    ok(cm.lib().cmld_linear(kernel, wd.ptr, w.shape[0], w.shape[1], xd.ptr, x.shape[0], out.ptr, int(out_bf16), act, act_rows, None, 1.0, 1, 0, C.byref(ms)))
     y = out.to_numpy(np.uint16 if out_bf16 else np.float32)
     return (from_bf16(y) if out_bf16 else y).reshape(x.shape[0], w.shape[0])
 
