@@ -1,13 +1,12 @@
 """Small random Losarax models for the tests: configurations, weights rounded to bfloat16, checkpoint folders."""
 from __future__ import annotations
 
-import json
-
 import numpy as np
 
-from camelid_b200.safetensors import from_bf16, to_bf16, write_safetensors
+from camelid_b200.safetensors import from_bf16, to_bf16
 
 import plain_losarax as pl
+from layered_helpers import LIMIT, rel_rms, tokens, write_folder  # noqa: F401
 
 
 def latent(heads=3, dim=24, vdim=16, q_rank=40, kv_rank=56, rot_dim=8, dims=None, base=10000.0, scale=None):
@@ -109,25 +108,5 @@ def engine(cfg, params, max_pos, max_seqs=1, dtype="float32", **kw):
         eng.set_tensor(name, to_bf16(params[name]))
     return eng
 
-
-def write_folder(path, cfg, params):
-    path.mkdir(parents=True, exist_ok=True)
-    (path / "config.json").write_text(json.dumps(cfg))
-    write_safetensors(path / "model.safetensors", {k: to_bf16(v).reshape(v.shape) for k, v in params.items()})
-    return path
-
-
-def tokens(cfg, n, seed):
-    return np.random.default_rng(seed).integers(0, cfg["vocab"], n).tolist()
-
-
-def rel_rms(got, ref):
-    """Per row: rms of the difference over the rms of the whole reference."""
-    got, ref = np.asarray(got, np.float64), np.asarray(ref, np.float64)
-    return np.sqrt(((got - ref) ** 2).mean(-1)) / np.sqrt((ref ** 2).mean())
-
-
-# largest row error allowed, relative to the reference's rms
-LIMIT = {"float32": 2e-5, "bfloat16": 4e-2}
 
 plain = pl.forward

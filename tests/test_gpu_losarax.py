@@ -10,38 +10,12 @@ import pytest
 
 import losarax_cases as lc
 import plain_losarax as pl
+import layered_helpers as lh
 from helpers import has_gpu
+from layered_helpers import DTYPES, check, cut, feed
 
 pytestmark = [pytest.mark.gpu, pytest.mark.skipif(not has_gpu(), reason="needs a GPU")]
-DTYPES = ["float32", "bfloat16"]
 ROOT = Path(__file__).resolve().parent.parent
-
-
-def feed(eng, seq, tokens, parts, taps=0):
-    """The tokens in portions of the given sizes; logits of every token (and the residual after every layer run)."""
-    at, logits, stream = 0, [], []
-    for k in parts:
-        r = eng.extend(seq, tokens[at:at + k], at, list(range(k)), taps=taps)
-        logits.append(r[1])
-        if taps:
-            stream.append(r[2])
-        at += k
-    assert at == len(tokens)
-    return (np.concatenate(logits), np.concatenate(stream, 1)) if taps else np.concatenate(logits)
-
-
-def cut(n, sizes):
-    """n cut into portions of the sizes, over and over."""
-    out, i = [], 0
-    while sum(out) < n:
-        out.append(min(sizes[i % len(sizes)], n - sum(out)))
-        i += 1
-    return out
-
-
-def check(got, ref, dtype, what, factor=1.0):
-    e = lc.rel_rms(got, ref)
-    assert np.isfinite(got).all() and e.max() <= factor * lc.LIMIT[dtype], (what, float(e.max()), int(np.unravel_index(e.argmax(), e.shape)[-1]))
 
 
 # ---------------------------------------------------------------- the linear layers alone
@@ -62,7 +36,7 @@ def device_rows(a, bf16):
     return DeviceBuffer.from_numpy(to_bf16(p) if bf16 else p)
 
 
-def linear(cm, kernel, w, x, out_bf16=False, act=0, act_rows=0):
+def linear(cm, kernel, w, x, out_bf16=False, act=0, act_rows=0, bias=None, scale=1.0):
     import ctypes as C
 
     from camelid_b200._lib import check as ok
@@ -70,11 +44,14 @@ def linear(cm, kernel, w, x, out_bf16=False, act=0, act_rows=0):
     from camelid_b200.safetensors import from_bf16
 
     wd, xd = device_rows(w, True), device_rows(x, kernel == 1)
-    out = DeviceBuffer(x.shape[0] * w.shape[0] * (2 if out_bf16 else 4))
+    outs = w.shape[0] // 2 if act == 3 else w.shape[0]
+    out = DeviceBuffer(x.shape[0] * outs * (2 if out_bf16 else 4))
+    bd = None if bias is None else DeviceBuffer.from_numpy(np.asarray(bias, np.float32))
     ms = C.c_float(0)
-    ok(cm.lib().cmld_linear(kernel, wd.ptr, w.shape[0], w.shape[1], xd.ptr, x.shape[0], out.ptr, int(out_bf16), act, act_rows, None, 1.0, 1, 0, C.byref(ms)))
+    ok(cm.lib().cmld_linear(kernel, wd.ptr, w.shape[0], w.shape[1], xd.ptr, x.shape[0], out.ptr, int(out_bf16), act, act_rows,
+                            bd.ptr if bd else None, scale, 1, 0, C.byref(ms)))
     y = out.to_numpy(np.uint16 if out_bf16 else np.float32)
-    return (from_bf16(y) if out_bf16 else y).reshape(x.shape[0], w.shape[0])
+    return (from_bf16(y) if out_bf16 else y).reshape(x.shape[0], outs)
 
 
 def lin_case(shape, seed=0):
@@ -105,6 +82,19 @@ def test_linear_activations(cm):
     for kernel, rows in ((0, 2), (1, 40), (2, 40)):
         assert np.abs(linear(cm, kernel, w, x[:rows], act=1, act_rows=70) - silu[:rows]).max() < 5e-5
         assert np.abs(linear(cm, kernel, w, x[:rows], act=2) - np.maximum(ref[:rows], 0) ** 2).max() < 1e-4
+
+
+@pytest.mark.parametrize("shape", [(200, 96, 40), (130, 1024, 5), (2, 8, 3), (258, 72, 64), (514, 320, 129), (1026, 256, 300)])
+def test_linear_gated_pairs_bias_and_scale(cm, shape):
+    """Tiles, clusters that share a tile, odd row counts; bias and factor before the activation."""
+    w, x = lin_case(shape, 5)
+    b = np.random.default_rng(6).standard_normal(shape[0]).astype(np.float32)
+    ref = 0.7 * (x.astype(np.float64) @ w.astype(np.float64).T) + b
+    pair = pl.silu(ref[:, 0::2]) * ref[:, 1::2]
+    for kernel, rows in ((0, 1), (0, 2), (1, shape[2]), (2, shape[2])):
+        assert np.abs(linear(cm, kernel, w, x[:rows], bias=b, scale=0.7) - ref[:rows]).max() < 5e-5, kernel
+        assert np.abs(linear(cm, kernel, w, x[:rows], act=3, bias=b, scale=0.7) - pair[:rows]).max() < 2e-4, kernel
+    assert np.abs(linear(cm, 1, w, x, out_bf16=True, act=3, bias=b, scale=0.7) - pair).max() < 2e-2 * max(1.0, np.abs(pair).max())
 
 
 # ---------------------------------------------------------------- whole models
@@ -344,11 +334,7 @@ def test_extend_and_sample_on_a_llama_shaped_engine(cm, orc):
 # ---------------------------------------------------------------- generation through the framework's own entry points
 
 def greedy_follows(params, cfg, prompt, out, dtype):
-    toks = list(prompt)
-    for t in out:
-        ref = lc.plain(params, cfg, toks)[0][-1]
-        assert ref[t] >= ref.max() - 4 * lc.LIMIT[dtype] * np.sqrt((ref ** 2).mean()), (len(toks), t)
-        toks.append(t)
+    lh.greedy_follows(lc.plain, params, cfg, prompt, out, dtype)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
