@@ -582,8 +582,8 @@ def design_case(eng, vocab, batch, n_prompt, steps, warmup, local_rank):
 
 
 def run_design(args):
-    """--design losarax: the layered design at several sizes beside the llama shape of equal width, depth, feed-forward width
-    and vocabulary (Q4_K_M, this library's closest model).  Weights are random; one JSON line."""
+    """--design NAME: a layered design at several sizes beside this library's closest models of equal width, depth, feed-forward
+    width and vocabulary (the other layered design in bfloat16, the llama shape in Q4_K_M).  Weights are random; one JSON line."""
     import camelid_b200 as cm
     from camelid_b200 import synth
 
@@ -595,33 +595,39 @@ def run_design(args):
     rows = []
     n_prompt = args.prompt or 1024
     steps, warmup = args.steps, max(3, args.warmup)
-    shapes = [s for s in (args.design_shapes or "losarax-2k,losarax-4k").split(",") if s]
+    ctx = n_prompt + steps + warmup + 8
+
+    def layered(shape, batch):
+        spec = synth.layered_spec(shape, args.design_layers or None)
+        eng = synth.build_layered(spec, SEED, ctx, batch)
+        r = design_case(eng, spec.vocab, batch, n_prompt, steps, warmup, 0)
+        wb = synth.layered_bytes(eng)
+        by = wb + synth.layered_context_bytes(eng, r["context"], batch)
+        flops = wb * n_prompt  # two per bfloat16 weight; the head runs for one row
+        flops -= 2 * (n_prompt - 1) * spec.vocab * spec.width
+        return eng, len(spec.layers), "bf16", wb, by, flops, r
+
+    def llama(shape, batch):
+        cfg = synth.engine_config(shape, max_pos=ctx, max_seqs=batch, n_layers=depth)
+        eng = synth.build_engine(cfg, "q4_k_m", SEED)
+        r = design_case(eng, cfg.vocab, batch, n_prompt, steps, warmup, 0)
+        wb = synth.weight_bytes_per_token(cfg, "q4_k_m")
+        by = wb + batch * synth.kv_bytes_per_position(cfg) * r["context"]
+        flops = 2 * n_prompt * cfg.n_layers * sum(a * b for a, b in synth.proj_shapes(cfg).values())
+        return eng, cfg.n_layers, "q4_k_m", wb, by, flops, r
+
+    shapes = [s for s in (args.design_shapes or f"{args.design}-2k,{args.design}-4k").split(",") if s]
     for shape in shapes:
-        peer = synth.LOSARAX_PEER[shape]
+        depth = args.design_layers or len(synth.layered_spec(shape).layers)
+        peers = (synth.LOSARAX_PEER[shape],) if args.design == "losarax" else synth.TOKOVIK_PEER[shape]
         for batch in [int(b) for b in args.design_batches.split(",")]:
-            spec = synth.losarax_spec(shape, args.design_layers or None)
-            ctx = n_prompt + steps + warmup + 8
-            eng = synth.build_layered(spec, SEED, ctx, batch)
-            r = design_case(eng, spec.vocab, batch, n_prompt, steps, warmup, 0)
-            wb = synth.layered_bytes(eng)
-            by = wb + synth.layered_context_bytes(eng, r["context"], batch)
-            flops = wb * n_prompt  # two per bfloat16 weight; the head runs for one row
-            flops -= 2 * (n_prompt - 1) * spec.vocab * spec.width
-            r.update(model=shape, layers=len(spec.layers), dtype="bf16", weight_bytes=wb, decode_frac_of_hbm=by / (r["ms_per_step"] * 1e-3) / 1e9 / hbm,
-                     prefill_linear_tflops=flops / (r["prefill_ms"] * 1e-3) / 1e12, prefill_frac_of_bf16=flops / (r["prefill_ms"] * 1e-3) / 1e12 / tflops)
-            rows.append(r)
-            eng.close()
-            cfg = synth.engine_config(peer, max_pos=ctx, max_seqs=batch, n_layers=len(spec.layers))
-            eng = synth.build_engine(cfg, "q4_k_m", SEED)
-            r = design_case(eng, cfg.vocab, batch, n_prompt, steps, warmup, 0)
-            wb = synth.weight_bytes_per_token(cfg, "q4_k_m")
-            by = wb + batch * synth.kv_bytes_per_position(cfg) * r["context"]
-            sh = synth.proj_shapes(cfg)
-            flops = 2 * n_prompt * cfg.n_layers * sum(a * b for a, b in sh.values())
-            r.update(model=peer, layers=cfg.n_layers, dtype="q4_k_m", weight_bytes=wb, decode_frac_of_hbm=by / (r["ms_per_step"] * 1e-3) / 1e9 / hbm,
-                     prefill_linear_tflops=flops / (r["prefill_ms"] * 1e-3) / 1e12, prefill_frac_of_bf16=flops / (r["prefill_ms"] * 1e-3) / 1e12 / tflops)
-            rows.append(r)
-            eng.close()
+            for model in (shape, *(peers if not args.design_alone else ())):
+                run = llama if model in synth.SHAPES else layered
+                eng, layers, dtype, wb, by, flops, r = run(model, batch)
+                eng.close()
+                r.update(model=model, layers=layers, dtype=dtype, weight_bytes=wb, decode_frac_of_hbm=by / (r["ms_per_step"] * 1e-3) / 1e9 / hbm,
+                         prefill_linear_tflops=flops / (r["prefill_ms"] * 1e-3) / 1e12, prefill_frac_of_bf16=flops / (r["prefill_ms"] * 1e-3) / 1e12 / tflops)
+                rows.append(r)
     print(json.dumps({"design": args.design, "steps": steps, "warmup": warmup, "data": "synthetic (random weights)", "hbm_gbs": hbm, "bf16_tflops": tflops,
                       "peak_kind": kind, "l2": "inputs larger than L2: every step streams the model's weights from HBM", "results": rows}), flush=True)
 
@@ -668,9 +674,10 @@ def main():
                     help="profiling runs only: start decoding at the prompt length over an all-zero KV cache instead of ingesting a prompt")
     ap.add_argument("--prompt", type=int, default=0, help="override the workload's prompt length (profiling runs)")
     ap.add_argument("--engine-flags", type=int, default=0, help="CMLD_FLAG_* bits: 1 no CUDA graph, 2 direct-load matvec, 4 no PDL, 8 separate prep kernels, 16 plain reference-order kernels, 32 NCCL-only sums, 64 tensor-core matvec from 5 rows, 128 lane-parallel f32 sums")
-    ap.add_argument("--design", default="", choices=["", "losarax"],
-                    help="measure a layered design at --design-shapes beside the llama shapes of equal size, instead of the workload")
-    ap.add_argument("--design-shapes", default="", help="comma-separated names from synth.LOSARAX_SHAPES")
+    ap.add_argument("--design", default="", choices=["", "losarax", "tokovik"],
+                    help="measure a layered design at --design-shapes beside the closest models of equal size, instead of the workload")
+    ap.add_argument("--design-alone", action="store_true", help="the design only, without the models beside it")
+    ap.add_argument("--design-shapes", default="", help="comma-separated names from synth.LOSARAX_SHAPES or synth.TOKOVIK_SHAPES")
     ap.add_argument("--design-layers", type=int, default=0, help="layers instead of the shape's own number (profiling runs)")
     ap.add_argument("--design-batches", default="1,32")
     ap.add_argument("--watchdog", type=int, default=-1,

@@ -3,9 +3,9 @@
 //   o_t = (q_t exp(B_t))^T S + sum over s <= t of A_ts v_s,   A_ts = sum over channels of q_t k_s exp(B_t - B_s)
 //   S'  = diag(exp(B_end)) S + sum over s of (k_s exp(B_end - B_s)) v_s^T
 // Every exponent is <= 0.  exp(-B_s) alone would overflow under strong decays, so A is cut into blocks of 16 x 16 tokens
-// (secondary chunks, as in "Gated Linear Attention Transformers with Hardware-Efficient Training", Yang et al.): a block off
-// the diagonal factors at the borders between the blocks and runs on the tensor cores, a block on the diagonal takes the
-// exponential of each pair's difference.
+// (secondary chunks, as in "Gated Linear Attention Transformers with Hardware-Efficient Training", Yang et al.), those on the
+// diagonal once more into 8 x 8: a block off the diagonal factors at the borders between the blocks and runs on the tensor
+// cores, one on the diagonal takes the exponential of each pair's difference.
 //
 // gated_prep_kernel: everything that does not need the state, all chunks and heads at once: decays, A, the scaled queries
 //   and keys, as two bfloat16 terms each.
@@ -41,19 +41,29 @@ __host__ __device__ inline ChunkLayout chunk_layout(int dim, int vdim) {
 }
 
 __host__ __device__ inline int prep_w_ld(int rank) { return ((rank + 7) & ~7) + 8; }
+__host__ __device__ inline int prep_u_ld(int rank) { return (rank + 3) & ~3; }
 __host__ __device__ inline int prep_smem(int dim, int rank) {
-  const int dp = pad16(dim), rows = kC * (dp + 1) * 4, qk = 2 * rows, w = dim * prep_w_ld(rank) * 2 + kC * rank * 4;
-  return 4 * dp * 4 + rows + (qk > w ? qk : w);
+  const int dp = pad16(dim), rows = kC * (dp + 8) * 4, w = dim * prep_w_ld(rank) * 2 + kC * prep_u_ld(rank) * 4;
+  return 12 * dp * 4 + 2 * rows + (rows > w ? rows : w);
 }
 
-__global__ void __launch_bounds__(kPrepThreads) gated_prep_kernel(const LightningArgs a, uint8_t *scratch) {
+// 2^x, x <= 0 here
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// Logarithms of decays are to base 2 in this kernel.
+__global__ void __launch_bounds__(kPrepThreads, 2) gated_prep_kernel(const LightningArgs a, uint8_t *scratch) {
   extern __shared__ __align__(16) uint8_t raw[];
   const ChunkLayout L = chunk_layout(a.dim, a.vdim);
-  const int dp = L.dp, ld = dp + 1, rank = a.channel.w.cols, wl = prep_w_ld(rank);
-  float *T = reinterpret_cast<float *>(raw);  // [4][dp]: sums of log decays over 16 tokens
-  float *lb = T + 4 * dp;                     // [64][ld]: sums of log decays since the 16 tokens began
+  const int dp = L.dp, ld = dp + 8, rank = a.channel.w.cols, wl = prep_w_ld(rank), ul = prep_u_ld(rank);
+  float *T = reinterpret_cast<float *>(raw);         // [4][dp]: log decays summed over 16 tokens,
+  float *before = T + 4 * dp, *rest = before + 4 * dp;  //   over the 16s before, over this one and those after it
+  float *lb = T + 12 * dp;                    // [64][ld]: log decays summed since the 16 tokens began
   float *q = lb + kC * ld, *k = q + kC * ld;  // [64][ld]
-  bf16 *w = reinterpret_cast<bf16 *>(q);      // first the decay weights [dim][wl] and the low-rank rows [64][rank]
+  bf16 *w = reinterpret_cast<bf16 *>(k);      // first the decay weights [dim][wl] and the low-rank rows [64][ul]
   float *u = reinterpret_cast<float *>(w + a.dim * wl);
   const int h = blockIdx.x, c0 = blockIdx.y * kC, len = min(kC, a.rows - c0), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   uint8_t *out = scratch + ((int64_t)blockIdx.y * a.heads + h) * L.bytes;
@@ -64,114 +74,173 @@ __global__ void __launch_bounds__(kPrepThreads) gated_prep_kernel(const Lightnin
     *reinterpret_cast<uint4 *>(w + (i / units) * wl + (i % units) * 8) =
         *reinterpret_cast<const uint4 *>(a.channel.w.w + (int64_t)(h * a.dim + i / units) * a.channel.w.ld + (i % units) * 8);
   if (!a.late_wait) pdl_wait();
-  for (int i = tid; i < kC * rank; i += kPrepThreads) u[i] = i / rank < len ? __ldcg(a.channel.x + (c0 + i / rank) * a.ld + i % rank) : 0.0f;
+  const int64_t hd = (int64_t)a.heads * a.dim;
+  const float *x = static_cast<const float *>(a.qkv) + (int64_t)c0 * a.ld + h * a.dim, *xv = x + 2 * hd + h * (a.vdim - a.dim);
+  const bool vec = ((a.ld | a.dim) & 3) == 0 && (reinterpret_cast<uintptr_t>(a.qkv) & 15) == 0;
+  const bool vec_v = vec && (a.vdim & 3) == 0;
+  // a head's rows of one chunk; what lies past the portion or the sizes is zero
+  auto bring = [&](float *dst, const float *src) {
+    if (vec) {
+#pragma unroll 4
+      for (int t = warp; t < kC; t += kPrepThreads / 32)
+        for (int d = lane * 4; d < dp; d += 128) {
+          const bool live = t < len && d < a.dim;
+          cp16(dst + t * ld + d, live ? src + t * a.ld + d : src, live);
+        }
+    } else {
+      for (int t = warp; t < kC; t += kPrepThreads / 32)
+        for (int d = lane; d < dp; d += 32) dst[t * ld + d] = t < len && d < a.dim ? __ldcg(src + t * a.ld + d) : 0.0f;
+    }
+  };
+  bring(q, x);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+#pragma unroll 4
+  for (int i = tid; i < kC * ul; i += kPrepThreads) u[i] = i / ul < len && i % ul < rank ? __ldcg(a.channel.x + (c0 + i / ul) * a.ld + i % ul) : 0.0f;
   __syncthreads();
+  // a thread sums a channel's log decays over 16 tokens
   for (int i = tid; i < 4 * dp; i += kPrepThreads) {
-    const int d = i % dp, sub = i / dp;
-    const float b = d < a.dim ? a.channel.b[h * a.dim + d] : 0.0f;
-    float run = 0.0f;
-    for (int t = sub * kSub; t < (sub + 1) * kSub; ++t) {
-      if (d < a.dim && t < len) {
-        float z = 0.0f;
-#pragma unroll 8
-        for (int j = 0; j < rank; ++j) z = fmaf(__bfloat162float(w[d * wl + j]), u[t * rank + j], z);
-        run += log_decay(z + b, a.channel.inv_tau);
+    const int d = i % dp, t0 = i / dp * kSub;
+    const bool live = d < a.dim;
+    const float b = live ? a.channel.b[h * a.dim + d] : 0.0f;
+    float z[kSub];
+#pragma unroll
+    for (int t = 0; t < kSub; ++t) z[t] = b;
+    if (live)
+      for (int j = 0; j < rank; j += 4) {
+        const uint2 v = *reinterpret_cast<const uint2 *>(w + d * wl + j);  // past the rank: zero
+        const float w0 = bf16_lo(v.x), w1 = bf16_hi(v.x), w2 = bf16_lo(v.y), w3 = bf16_hi(v.y);
+#pragma unroll
+        for (int t = 0; t < kSub; ++t) {
+          const float4 f = *reinterpret_cast<const float4 *>(u + (t0 + t) * ul + j);
+          z[t] = fmaf(w0, f.x, fmaf(w1, f.y, fmaf(w2, f.z, fmaf(w3, f.w, z[t]))));
+        }
       }
-      lb[t * ld + d] = run;
+    float run = 0.0f;
+#pragma unroll
+    for (int t = 0; t < kSub; ++t) {
+      if (live && t0 + t < len) run += log_decay(z[t], a.channel.inv_tau * 1.44269504f);
+      lb[(t0 + t) * ld + d] = run;
     }
     T[i] = run;
   }
   __syncthreads();
-  const int64_t hd = (int64_t)a.heads * a.dim;
-  const float *x = static_cast<const float *>(a.qkv) + (int64_t)c0 * a.ld;
-#pragma unroll 4
-  for (int i = tid; i < kC * dp; i += kPrepThreads) {
-    const int t = i / dp, d = i % dp;
-    const bool live = t < len && d < a.dim;
-    const float *p = x + t * a.ld + h * a.dim + d;
-    q[t * ld + d] = live ? a.q_scale * __ldcg(p) : 0.0f;
-    k[t * ld + d] = live ? __ldcg(p + hd) : 0.0f;
+  bring(k, x + hd);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  if (vec_v) {
+#pragma unroll 8
+    for (int t = warp; t < kC; t += kPrepThreads / 32)
+      for (int c = lane * 4; c < L.vp; c += 128) {
+        const float4 v = t < len && c < a.vdim ? __ldcg(reinterpret_cast<const float4 *>(xv + t * a.ld + c)) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        *reinterpret_cast<uint2 *>(o16 + L.v + t * L.vp + c) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+      }
+  } else {
+    for (int t = warp; t < kC; t += kPrepThreads / 32)
+      for (int c = lane; c < L.vp; c += 32) o16[L.v + t * L.vp + c] = __float2bfloat16_rn(t < len && c < a.vdim ? __ldcg(xv + t * a.ld + c) : 0.0f);
   }
-#pragma unroll 4
-  for (int i = tid; i < kC * L.vp; i += kPrepThreads) {
-    const int t = i / L.vp, c = i % L.vp;
-    o16[L.v + i] = __float2bfloat16_rn(t < len && c < a.vdim ? __ldcg(x + t * a.ld + 2 * hd + h * a.vdim + c) : 0.0f);
+  for (int d = tid; d < dp; d += kPrepThreads) {
+    const float s0 = T[d], s1 = T[dp + d], s2 = T[2 * dp + d], s3 = T[3 * dp + d];
+    before[d] = 0.0f;
+    before[dp + d] = s0;
+    before[2 * dp + d] = s0 + s1;
+    before[3 * dp + d] = s0 + s1 + s2;
+    rest[3 * dp + d] = s3;
+    rest[2 * dp + d] = s2 + s3;
+    rest[dp + d] = s1 + (s2 + s3);
+    rest[d] = s0 + (s1 + (s2 + s3));
+    reinterpret_cast<float *>(o16 + L.d)[d] = ex2(rest[d]);
   }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
   // queries from the chunk's start, keys to its end
-  for (int i = tid; i < kC * dp / 2; i += kPrepThreads) {
-    const int t = i / (dp / 2), d = i % (dp / 2) * 2, sub = t / kSub;
-    float qv[2], kv[2];
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const float l = lb[t * ld + d + e];
-      float from = l, to = T[sub * dp + d + e] - l;
-      for (int s = 0; s < 4; ++s) {
-        if (s < sub) from += T[s * dp + d + e];
-        if (s > sub) to += T[s * dp + d + e];
-      }
-      qv[e] = q[t * ld + d + e] * expf(from);
-      kv[e] = k[t * ld + d + e] * expf(to);
+#pragma unroll 2
+  for (int t = warp; t < kC; t += kPrepThreads / 32) {
+    const float *bt = before + t / kSub * dp, *rt = rest + t / kSub * dp;
+    for (int d = lane * 2; d < dp; d += 64) {
+      const float2 l = *reinterpret_cast<const float2 *>(lb + t * ld + d), qv = *reinterpret_cast<const float2 *>(q + t * ld + d);
+      const float2 kv = *reinterpret_cast<const float2 *>(k + t * ld + d), f = *reinterpret_cast<const float2 *>(bt + d);
+      const float2 r = *reinterpret_cast<const float2 *>(rt + d);
+      uint32_t hi, lo;
+      uint32_t *o = reinterpret_cast<uint32_t *>(o16 + t * dp + d);
+      split_pair(a.q_scale * qv.x * ex2(f.x + l.x), a.q_scale * qv.y * ex2(f.y + l.y), hi, lo);
+      o[0] = hi;
+      o[kC * dp / 2] = lo;
+      split_pair(kv.x * ex2(r.x - l.x), kv.y * ex2(r.y - l.y), hi, lo);
+      o[2 * kC * dp / 2] = hi;
+      o[3 * kC * dp / 2] = lo;
     }
-    uint32_t hi, lo;
-    uint32_t *o = reinterpret_cast<uint32_t *>(o16 + t * dp + d);
-    split_pair(qv[0], qv[1], hi, lo);
-    o[0] = hi;
-    o[kC * dp / 2] = lo;
-    split_pair(kv[0], kv[1], hi, lo);
-    o[2 * kC * dp / 2] = hi;
-    o[3 * kC * dp / 2] = lo;
   }
-  for (int d = tid; d < dp; d += kPrepThreads) reinterpret_cast<float *>(o16 + L.d)[d] = expf(T[d] + T[dp + d] + T[2 * dp + d] + T[3 * dp + d]);
   bf16 *A = o16 + L.a;
   auto put = [&](int t, int s, float v) {
     const bf16 hi = __float2bfloat16_rn(v);
     A[t * kC + s] = hi;
     A[kC * kC + t * kC + s] = __float2bfloat16_rn(v - __bfloat162float(hi));
   };
-  // blocks on the diagonal, pair by pair
-  constexpr int kPairs = kSub * (kSub + 1) / 2;
-  for (int i = tid; i < 4 * kPairs; i += kPrepThreads) {
-    const int sub = i / kPairs, r = i % kPairs;
-    int t = (int)((sqrtf(8.0f * r + 1.0f) - 1.0f) * 0.5f);
-    while (t * (t + 1) / 2 > r) --t;
-    while ((t + 1) * (t + 2) / 2 <= r) ++t;
-    const int s = sub * kSub + r - t * (t + 1) / 2;
-    t += sub * kSub;
-    float v = 0.0f;
-#pragma unroll 4
-    for (int d = 0; d < a.dim; ++d) v = fmaf(q[t * ld + d] * k[s * ld + d], expf(lb[t * ld + d] - lb[s * ld + d]), v);
-    put(t, s, v);
+  // pairs of the same eight tokens: a warp takes eight tokens, its lanes the channels
+#pragma unroll 1
+  for (int e = 0; e < 8; ++e) {
+    const int t0 = warp * 8, t = t0 + e;
+    float v[8] = {};
+    for (int d = lane; d < dp; d += 32) {
+      const float qd = q[t * ld + d], l = lb[t * ld + d];
+#pragma unroll
+      for (int s = 0; s < 8; ++s)
+        if (s <= e) v[s] = fmaf(qd * k[(t0 + s) * ld + d], ex2(l - lb[(t0 + s) * ld + d]), v[s]);
+    }
+    float mine = 0.0f;
+#pragma unroll
+    for (int s = 0; s < 8; ++s) {
+      if (s > e) break;
+      const float f = warp_sum(v[s]);
+      if (lane == s) mine = f;
+    }
+    if (lane < 8) put(t, t0 + lane, a.q_scale * mine);  // zero above the diagonal
+    if (lane < 8 && (warp & 1) == 0) put(t, t0 + 8 + lane, 0.0f);
   }
-  for (int i = tid; i < 4 * kSub * kSub; i += kPrepThreads) {
-    const int sub = i / (kSub * kSub), t = i / kSub % kSub, s = i % kSub;
-    if (s > t) put(sub * kSub + t, sub * kSub + s, 0.0f);
-  }
-  // blocks below it: warp 0 (1,0), 1 (2,0), 2 (2,1), 3 (3,0), 4 (3,1), 5 (3,2)
-  if (warp < 6) {
-    const int bi = warp == 0 ? 1 : warp < 3 ? 2 : 3, bj = warp == 0 ? 0 : warp < 3 ? warp - 1 : warp - 3;
-    const int tr = lane >> 2, tc = (lane & 3) * 2;
+  // blocks below the diagonal on the tensor cores, factored at a place between their queries and their keys: 16 x 16, task
+  // 0..5 = (1,0), (2,0), (2,1), (3,0), (3,1), (3,2); 8 x 8, task 6..9 = the two halves of 16 tokens
+  const int tr = lane >> 2, tc = (lane & 3) * 2;
+#pragma unroll 1
+  for (int task = warp; task < 10; task += kPrepThreads / 32) {
+    const bool half = task >= 6;
+    const int bi = half ? task - 6 : task == 0 ? 1 : task < 3 ? 2 : 3, bj = half ? bi : task == 0 ? 0 : task < 3 ? task - 1 : task - 3;
+    const int tq = bi * kSub + (half ? 8 : 0), tk = bj * kSub;
+    const float *edge = half ? lb + (tk + 7) * ld : T + bj * dp;  // sum up to the last of the keys
     float acc[2][4] = {};
     auto qe = [&](int t, int d) {
-      float e = lb[t * ld + d];
-      for (int s = bj + 1; s < bi; ++s) e += T[s * dp + d];
-      return q[t * ld + d] * expf(e);
+      const float2 l = *reinterpret_cast<const float2 *>(lb + t * ld + d), v = *reinterpret_cast<const float2 *>(q + t * ld + d);
+      float2 e = l;
+      if (half) {
+        e.x -= edge[d];
+        e.y -= edge[d + 1];
+      }
+      for (int s = bj + 1; s < bi; ++s) {
+        e.x += T[s * dp + d];
+        e.y += T[s * dp + d + 1];
+      }
+      return make_float2(v.x * ex2(e.x), v.y * ex2(e.y));
     };
-    auto ke = [&](int s, int d) { return k[s * ld + d] * expf(T[bj * dp + d] - lb[s * ld + d]); };
+    auto ke = [&](int s, int d) {
+      const float2 l = *reinterpret_cast<const float2 *>(lb + s * ld + d), v = *reinterpret_cast<const float2 *>(k + s * ld + d);
+      return make_float2(v.x * ex2(edge[d] - l.x), v.y * ex2(edge[d + 1] - l.y));
+    };
+#pragma unroll 1
     for (int d0 = 0; d0 < dp; d0 += 16) {
       uint32_t AH[4], AL[4];
 #pragma unroll
       for (int f = 0; f < 4; ++f) {
-        const int t = bi * kSub + tr + (f & 1) * 8, d = d0 + (f >> 1) * 8 + tc;
-        split_pair(qe(t, d), qe(t, d + 1), AH[f], AL[f]);
+        AH[f] = AL[f] = 0;
+        if (half && (f & 1)) continue;  // eight queries only
+        const float2 v = qe(tq + tr + (f & 1) * 8, d0 + (f >> 1) * 8 + tc);
+        split_pair(v.x, v.y, AH[f], AL[f]);
       }
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
+        if (half && n) continue;
         uint32_t BH[2], BL[2];
 #pragma unroll
         for (int f = 0; f < 2; ++f) {
-          const int s = bj * kSub + n * 8 + tr, d = d0 + f * 8 + tc;
-          split_pair(ke(s, d), ke(s, d + 1), BH[f], BL[f]);
+          const float2 v = ke(tk + n * 8 + tr, d0 + f * 8 + tc);
+          split_pair(v.x, v.y, BH[f], BL[f]);
         }
         mma16816(acc[n], AH, BH[0], BH[1]);
         mma16816(acc[n], AH, BL[0], BL[1]);
@@ -181,7 +250,8 @@ __global__ void __launch_bounds__(kPrepThreads) gated_prep_kernel(const Lightnin
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) put(bi * kSub + tr + (e >> 1) * 8, bj * kSub + n * 8 + tc + (e & 1), acc[n][e]);
+      for (int e = 0; e < 4; ++e)
+        if (!half || (n == 0 && e < 2)) put(tq + tr + (e >> 1) * 8, tk + n * 8 + tc + (e & 1), a.q_scale * acc[n][e]);
   }
   if (a.late_wait) pdl_wait();
 }

@@ -379,7 +379,7 @@ int32_t build(cmld_engine *e, LayeredModel *m) {
     ff = std::max(ff, lin_ld(std::max(d.ff, 1)));
     if (d.type == CMLD_LAYER_PARALLEL) {
       const cmld_gated_desc &g = d.gated;
-      proj = std::max<int64_t>(proj, L.in.rows);
+      proj = std::max(proj, lin_ld(L.in.rows));
       q = std::max(q, (int64_t)L.win.heads * window_pad(L.win.dim));
       mixed = std::max(mixed, lin_ld((int64_t)L.win.heads * L.win.vdim));
       wide = std::max(wide, lin_ld((int64_t)g.heads * g.vdim));
@@ -773,7 +773,7 @@ struct Step {
 
   int32_t parallel(const LayerDef &L, void *store, void *state, const StreamMix &s) {
     const cmld_gated_desc &g = L.d.gated;
-    const int64_t pl = L.in.rows, wv = (int64_t)L.win.heads * L.win.vdim, gv = (int64_t)g.heads * g.vdim, gk = (int64_t)g.heads * g.dim;
+    const int64_t pl = lin_ld(L.in.rows), wv = (int64_t)L.win.heads * L.win.vdim, gv = (int64_t)g.heads * g.vdim, gk = (int64_t)g.heads * g.dim;
     const int64_t at = (int64_t)(L.win.heads + L.win.kv_heads) * L.win.dim + (int64_t)L.win.kv_heads * L.win.vdim;
     const float *gate = m->proj + at + 2 * gk + gv;
     CMLD_TRY(read_in(s, L.in, m->proj, false, pl, kActNone, 0, L.in_bias));

@@ -368,19 +368,109 @@ __device__ __forceinline__ void layer_norm_cta(float *u, int n, const float *w, 
   for (int i = threadIdx.x; i < n; i += blockDim.x) u[i] = (u[i] - mean) * r * w[i] + b[i];
 }
 
-// x + y' of a single stream (see StreamMix).
+// Two sums over the CTA at once.
+__device__ __forceinline__ float2 cta_total2(float2 v, float *red) {
+  v.x = warp_sum(v.x);
+  v.y = warp_sum(v.y);
+  const int warp = threadIdx.x >> 5, n = (blockDim.x + 31) >> 5;
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) *reinterpret_cast<float2 *>(red + 2 * warp) = v;
+  __syncthreads();
+  float2 t = make_float2(0.0f, 0.0f);
+  for (int i = 0; i < n; ++i) {
+    const float2 p = *reinterpret_cast<const float2 *>(red + 2 * i);
+    t.x += p.x;
+    t.y += p.y;
+  }
+  return t;
+}
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
+
+// x + y' of a single stream (see StreamMix); put(i, v) takes values 4i .. 4i + 3 of the result.  The row stays in registers,
+// V times four values per thread (width a multiple of four, at most 4 V blockDim.x).  `red` holds 2 * blockDim.x / 32 floats.
+template <int V, typename Put>
+__device__ __forceinline__ void post_norm_row(const StreamMix &m, int64_t row, float *red, Put put) {
+  const int n4 = m.width / 4;
+  const float4 *x = reinterpret_cast<const float4 *>(m.x_in + row * m.width), *y = reinterpret_cast<const float4 *>(m.y + row * m.width);
+  float4 xv[V], yv[V];
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    yv[j] = i < n4 ? y[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
+  if (m.y2) {
+    const float4 *z = reinterpret_cast<const float4 *>(m.y2 + row * m.width), *yw = reinterpret_cast<const float4 *>(m.y_norm);
+    const float4 *zw = reinterpret_cast<const float4 *>(m.y2_norm);
+    float4 zv[V];
+    float2 s = make_float2(0.0f, 0.0f);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      zv[j] = i < n4 ? z[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      s.x += dot4(yv[j], yv[j]);
+      s.y += dot4(zv[j], zv[j]);
+      const int i = threadIdx.x + j * blockDim.x;
+      if (i < n4) {  // the branches' weights do not wait for the sums
+        const float4 a = yw[i], b = zw[i];
+        yv[j] = make_float4(yv[j].x * a.x, yv[j].y * a.y, yv[j].z * a.z, yv[j].w * a.w);
+        zv[j] = make_float4(zv[j].x * b.x, zv[j].y * b.y, zv[j].z * b.z, zv[j].w * b.w);
+      }
+    }
+    s = cta_total2(s, red);
+    const float ry = 0.5f / sqrtf(s.x / (float)m.width + m.eps), rz = 0.5f / sqrtf(s.y / (float)m.width + m.eps);
+#pragma unroll
+    for (int j = 0; j < V; ++j)
+      yv[j] = make_float4(fmaf(yv[j].x, ry, zv[j].x * rz), fmaf(yv[j].y, ry, zv[j].y * rz), fmaf(yv[j].z, ry, zv[j].z * rz), fmaf(yv[j].w, ry, zv[j].w * rz));
+  }
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    xv[j] = i < n4 ? x[i] : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
+  float r = 1.0f;
+  if (m.out_norm) {
+    float s = 0.0f;
+#pragma unroll
+    for (int j = 0; j < V; ++j) s += dot4(yv[j], yv[j]);
+    r = 1.0f / sqrtf(cta_total2(make_float2(s, 0.0f), red).x / (float)m.width + m.eps);
+  }
+#pragma unroll
+  for (int j = 0; j < V; ++j) {
+    const int i = threadIdx.x + j * blockDim.x;
+    if (i >= n4) break;
+    const float4 w = m.out_norm ? reinterpret_cast<const float4 *>(m.out_norm)[i] : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+    put(i, make_float4(fmaf(yv[j].x * r, w.x, xv[j].x), fmaf(yv[j].y * r, w.y, xv[j].y), fmaf(yv[j].z * r, w.z, xv[j].z), fmaf(yv[j].w * r, w.w, xv[j].w)));
+  }
+}
+
+// The same for any width, through u.
 __device__ __forceinline__ void post_norm_update(const StreamMix &m, int64_t row, float *u, float *red, bool store) {
   const float *x = m.x_in + row * m.width, *y = m.y + row * m.width;
   float *xo = store && m.x_out ? m.x_out + row * m.width : nullptr;
+  if (m.width % 4 == 0 && m.width <= 8 * (int)blockDim.x) {
+    if (!m.y2 && !m.out_norm) __syncthreads();  // no sum keeps the readers of an earlier row in u apart
+    auto put = [&](int i, float4 v) {
+      reinterpret_cast<float4 *>(u)[i] = v;
+      if (xo) reinterpret_cast<float4 *>(xo)[i] = v;
+    };
+    if (m.width <= 4 * (int)blockDim.x) post_norm_row<1>(m, row, red, put);
+    else post_norm_row<2>(m, row, red, put);
+    __syncthreads();  // a thread's values in u are not those of its stride
+    return;
+  }
   if (m.y2) {
     const float *z = m.y2 + row * m.width;
-    float sy = 0.0f, sz = 0.0f;
+    float2 s = make_float2(0.0f, 0.0f);
     for (int i = threadIdx.x; i < m.width; i += blockDim.x) {
-      sy = fmaf(y[i], y[i], sy);
-      sz = fmaf(z[i], z[i], sz);
+      s.x = fmaf(y[i], y[i], s.x);
+      s.y = fmaf(z[i], z[i], s.y);
     }
-    const float ry = 1.0f / sqrtf(cta_total(sy, red) / (float)m.width + m.eps), rz = 1.0f / sqrtf(cta_total(sz, red) / (float)m.width + m.eps);
-    for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = 0.5f * (y[i] * ry * m.y_norm[i] + z[i] * rz * m.y2_norm[i]);
+    s = cta_total2(s, red);
+    const float ry = 0.5f / sqrtf(s.x / (float)m.width + m.eps), rz = 0.5f / sqrtf(s.y / (float)m.width + m.eps);
+    for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = y[i] * m.y_norm[i] * ry + z[i] * m.y2_norm[i] * rz;
   } else {
     for (int i = threadIdx.x; i < m.width; i += blockDim.x) u[i] = y[i];
   }
@@ -405,7 +495,8 @@ __device__ __forceinline__ void rms_norm_cta(float *u, int n, const float *w, fl
   for (int i = threadIdx.x; i < n; i += blockDim.x) u[i] = u[i] * r * w[i];
 }
 
-// The whole boundary for one row; the result is left in u[width] (shared memory; each thread holds its own stride).
+// The whole boundary for one row; the result is left in u[width] (shared memory, 16-byte aligned; each thread may read its
+// own stride).  `red` holds 2 * blockDim.x / 32 floats, 8-byte aligned.
 __device__ __forceinline__ void stream_mix_row(const StreamMix &m, int r, float *u, float *red, bool store) {
   const int64_t row = m.row_map ? m.row_map[r] : r;
   if (m.embed) {

@@ -17,11 +17,8 @@ namespace {
 
 constexpr int kStepThreads = 256, kStepCols = 32, kStepGroups = kStepThreads / kStepCols;
 
-// shared memory: q, k and, with a decay per channel, the decays of this row and the head's decay weights [dim][pad]
-__host__ __device__ inline int decay_ld(int rank) { return ((rank + 7) & ~7) + 8; }
-inline size_t steps_smem(const LightningArgs &a) {
-  return a.powers ? (size_t)2 * a.dim * 4 : (size_t)((3 * a.dim + 3) & ~3) * 4 + (size_t)a.dim * decay_ld(a.channel.w.cols) * 2;
-}
+// shared memory: q, k and, with a decay per channel, the decays of this row
+inline size_t steps_smem(const LightningArgs &a) { return (size_t)(a.powers ? 2 : 3) * a.dim * 4; }
 
 // Activations may have been written just before this kernel started (late_wait): they are read past the L1 cache.
 __device__ __forceinline__ float act_load_cg(const void *p, int half, int64_t i) {
@@ -35,14 +32,16 @@ __global__ void __launch_bounds__(kStepThreads) linear_steps_kernel(const Lightn
   float *qs = sm, *ks = sm + a.dim, *al = ks + a.dim;  // this row's q, k and decays of the head
   __shared__ float red[kStepGroups][kStepCols];
   const int h = blockIdx.x, c = threadIdx.x % kStepCols, g = threadIdx.x / kStepCols;
-  const int rank = CHANNEL ? a.channel.w.cols : 0, wl = decay_ld(rank);
-  bf16 *w = reinterpret_cast<bf16 *>(sm + ((3 * a.dim + 3) & ~3));
+  const int rank = CHANNEL ? a.channel.w.cols : 0, wl = CHANNEL ? (int)a.channel.w.ld : 0, lane = threadIdx.x & 31;
+  const bf16 *w = CHANNEL ? a.channel.w.w + (int64_t)h * a.dim * wl : nullptr;
   pdl_launch();
-  if (CHANNEL) {  // weights depend on no earlier kernel
-    const int units = (int)a.channel.w.ld / 8;
-    for (int i = threadIdx.x; i < a.dim * units; i += kStepThreads)
-      *reinterpret_cast<uint4 *>(w + (i / units) * wl + (i % units) * 8) =
-          *reinterpret_cast<const uint4 *>(a.channel.w.w + (int64_t)(h * a.dim + i / units) * a.channel.w.ld + (i % units) * 8);
+  // the first 16 decay weights of this thread's channel and its bias: they depend on no earlier kernel
+  uint4 pre[2] = {};
+  float bias = 0.0f;
+  if (CHANNEL && (int)threadIdx.x < a.dim) {
+    pre[0] = *reinterpret_cast<const uint4 *>(w + threadIdx.x * wl);
+    if (wl > 8) pre[1] = *reinterpret_cast<const uint4 *>(w + threadIdx.x * wl + 8);
+    bias = a.channel.b[h * a.dim + threadIdx.x];
   }
   if (!a.late_wait) pdl_wait();
   const int col = blockIdx.y * kStepCols + c;
@@ -56,20 +55,31 @@ __global__ void __launch_bounds__(kStepThreads) linear_steps_kernel(const Lightn
 #pragma unroll
   for (int j = 0; j < DPT; ++j) s[j] = live && !fresh && d0 + j < a.dim ? __ldcg(st + (int64_t)(d0 + j) * a.vdim) : 0.0f;
   const int64_t hd = (int64_t)a.heads * a.dim;
-  if (CHANNEL) __syncthreads();
   for (int r = r0; r < r0 + n; ++r) {
     const int64_t row = (int64_t)r * a.ld;
+    float u = CHANNEL && lane < rank ? __ldcg(a.channel.x + row + lane) : 0.0f;  // 32 of the low-rank values, one per lane
     for (int i = threadIdx.x; i < a.dim; i += kStepThreads) {
       qs[i] = a.q_scale * act_load_cg(a.qkv, a.half, row + h * a.dim + i);
       ks[i] = act_load_cg(a.qkv, a.half, row + hd + h * a.dim + i);
-      if (CHANNEL) {
-        float z = 0.0f;
-#pragma unroll 8
-        for (int j = 0; j < rank; ++j) z = fmaf(__bfloat162float(w[i * wl + j]), __ldcg(a.channel.x + row + j), z);
-        al[i] = expf(log_decay(z + a.channel.b[h * a.dim + i], a.channel.inv_tau));
-      }
     }
     const float v = live ? act_load_cg(a.qkv, a.half, row + 2 * hd + h * a.vdim + col) : 0.0f;
+    if (CHANNEL) {
+      // whole warps, so that every lane can hand out its low-rank value
+      for (int i = threadIdx.x; i - lane < a.dim; i += kStepThreads) {
+        const bool mine = i < a.dim;
+        float z = i == (int)threadIdx.x ? bias : mine ? a.channel.b[h * a.dim + i] : 0.0f;
+        for (int j0 = 0; j0 < wl; j0 += 8) {
+          if ((j0 & 31) == 0 && (j0 > 0 || i != (int)threadIdx.x)) u = j0 + lane < rank ? __ldcg(a.channel.x + row + j0 + lane) : 0.0f;
+          uint4 p = make_uint4(0, 0, 0, 0);
+          if (j0 < 16 && i == (int)threadIdx.x) p = j0 == 0 ? pre[0] : pre[1];
+          else if (mine) p = *reinterpret_cast<const uint4 *>(w + (int64_t)i * wl + j0);
+          const float f[8] = {bf16_lo(p.x), bf16_hi(p.x), bf16_lo(p.y), bf16_hi(p.y), bf16_lo(p.z), bf16_hi(p.z), bf16_lo(p.w), bf16_hi(p.w)};
+#pragma unroll
+          for (int j = 0; j < 8; ++j) z = fmaf(f[j], __shfl_sync(0xffffffffu, u, (j0 & 31) + j), z);
+        }
+        if (mine) al[i] = expf(log_decay(z, a.channel.inv_tau));
+      }
+    }
     __syncthreads();
     float o = 0.0f;
 #pragma unroll
@@ -299,11 +309,6 @@ template <int DPT>
 int32_t steps(const LightningArgs &a, bool pdl, cudaStream_t s) {
   const dim3 grid(a.heads, (a.vdim + kStepCols - 1) / kStepCols, a.one_sequence ? 1 : a.rows);
   if (a.powers) return launch_kernel(linear_steps_kernel<DPT, false>, grid, dim3(kStepThreads), steps_smem(a), pdl, s, a);
-  static bool ready = false;
-  if (!ready) {
-    CMLD_TRY(allow_smem(linear_steps_kernel<DPT, true>, 160 * 1024));
-    ready = true;
-  }
   return launch_kernel(linear_steps_kernel<DPT, true>, grid, dim3(kStepThreads), steps_smem(a), pdl, s, a);
 }
 
@@ -331,7 +336,7 @@ int32_t launch_lightning_steps(const LightningArgs &a, bool pdl, cudaStream_t s)
 }
 
 bool gated_shape_ok(int32_t heads, int32_t dim, int32_t vdim, int32_t rank) {
-  return lightning_shape_ok(heads, dim, vdim) && rank >= 1 && (size_t)dim * (12 + decay_ld(rank) * 2) + 16 <= 160 * 1024;
+  return lightning_shape_ok(heads, dim, vdim) && rank >= 1 && rank <= 16384;
 }
 
 bool lightning_chunk_fits(const LightningArgs &a) { return a.powers && a.half && a.one_sequence && a.dim <= 256; }

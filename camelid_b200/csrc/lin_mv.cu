@@ -20,8 +20,8 @@ __host__ __device__ constexpr int mv_kpad(int cols) { return (cols + 255) & ~255
 
 template <int R, int ROWS>
 __device__ __forceinline__ void lin_mv_cta(const LinMvArgs &a, int cta, int ctas) {
-  extern __shared__ float smem[];
-  __shared__ float red[kMvThreads / 32];
+  extern __shared__ __align__(16) float smem[];
+  __shared__ __align__(8) float red[2 * kMvThreads / 32];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int K = a.w.cols, kp = mv_kpad(K), half = kp / 2, nit = kp / 256;
   float *xs = smem;              // [R][2][kp / 2]

@@ -11,8 +11,8 @@ constexpr int kMixThreads = 1024;
 int mix_threads(int rows) { return rows >= 512 ? 256 : rows >= 256 ? 512 : kMixThreads; }
 
 __global__ void __launch_bounds__(kMixThreads) stream_mix_kernel(const StreamMix m, ActBuf out) {
-  extern __shared__ float u[];
-  __shared__ float red[kMixThreads / 32];
+  extern __shared__ __align__(16) float u[];
+  __shared__ __align__(8) float red[2 * kMixThreads / 32];
   pdl_launch();
   pdl_wait();
   const int r = blockIdx.x;
@@ -20,9 +20,28 @@ __global__ void __launch_bounds__(kMixThreads) stream_mix_kernel(const StreamMix
   for (int i = threadIdx.x; i < m.width; i += blockDim.x) act_store(out.p, out.half, r * out.ld + i, u[i]);
 }
 
+// One stream with norms on the sublayers' outputs and no norm in front of the next: the row stays in registers.
+template <int V>
+__global__ void __launch_bounds__(V == 4 ? 512 : kMixThreads) post_norm_kernel(const __grid_constant__ StreamMix m, ActBuf out) {
+  __shared__ __align__(8) float red[2 * kMixThreads / 32];
+  pdl_launch();
+  pdl_wait();
+  const int64_t row = blockIdx.x;
+  post_norm_row<V>(m, row, red, [&](int i, float4 v) {
+    if (m.x_out) reinterpret_cast<float4 *>(m.x_out + row * m.width)[i] = v;
+    const int64_t at = row * out.ld + 4 * i;
+    if (out.half) {
+      __nv_bfloat162 p[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+      *reinterpret_cast<uint2 *>(static_cast<bf16 *>(out.p) + at) = *reinterpret_cast<const uint2 *>(p);
+    } else {
+      *reinterpret_cast<float4 *>(static_cast<float *>(out.p) + at) = v;
+    }
+  });
+}
+
 __global__ void __launch_bounds__(kMixThreads) stream_tap_kernel(const StreamMix m, float *out) {
-  extern __shared__ float u[];
-  __shared__ float red[kMixThreads / 32];
+  extern __shared__ __align__(16) float u[];
+  __shared__ __align__(8) float red[2 * kMixThreads / 32];
   pdl_wait();
   stream_mix_row(m, blockIdx.x, u, red, false);
   for (int i = threadIdx.x; i < m.width; i += blockDim.x) out[(int64_t)blockIdx.x * m.width + i] = u[i];
@@ -67,6 +86,14 @@ __global__ void __launch_bounds__(256) rms_groups_kernel(const float *x, int64_t
 }  // namespace
 
 int32_t launch_stream_mix(const StreamMix &m, int32_t rows, ActBuf out, bool pdl, cudaStream_t s) {
+  if (!m.embed && !m.mix && !m.norm_w && !m.row_map && m.width % 4 == 0 && m.width <= 8192 && out.ld % 4 == 0) {
+    // many rows: small CTAs, several values per thread
+    const int n4 = m.width / 4, per = rows >= 256 ? 4 : 1, threads = std::min(per == 4 ? 512 : kMixThreads, ((n4 + per - 1) / per + 31) & ~31);
+    const int v = (n4 + threads - 1) / threads;
+    if (v == 1) return launch_kernel(post_norm_kernel<1>, dim3(rows), dim3(threads), 0, pdl, s, m, out);
+    if (v == 2) return launch_kernel(post_norm_kernel<2>, dim3(rows), dim3(threads), 0, pdl, s, m, out);
+    return launch_kernel(post_norm_kernel<4>, dim3(rows), dim3(threads), 0, pdl, s, m, out);
+  }
   const size_t smem = (size_t)m.width * 4;
   if (smem > 48 * 1024) CMLD_TRY(allow_smem(stream_mix_kernel, smem));
   return launch_kernel(stream_mix_kernel, dim3(rows), dim3(mix_threads(rows)), smem, pdl, s, m, out);

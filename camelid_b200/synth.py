@@ -151,9 +151,32 @@ def losarax_spec(shape: str, n_layers: int | None = None):
     return LayeredSpec(vocab=vocab, width=width, eps=1e-5, layers=out, streams=streams)
 
 
+TOKOVIK_SHAPES = {
+    # name: (width, layers, heads, kv_heads, dim, vdim, window, rot_dims, gated heads, dim, vdim, rank, ff, vocab)
+    "tokovik-tiny": (256, 2, 4, 2, 32, 32, 48, 16, 4, 32, 32, 16, 512, 512),
+    "tokovik-2k": (2048, 8, 16, 4, 128, 128, 1024, 64, 16, 128, 128, 16, 8192, 128256),
+    "tokovik-4k": (4096, 8, 32, 8, 128, 128, 1024, 64, 32, 128, 128, 16, 14336, 128256),
+}
+# the models of equal width, feed-forward width and vocabulary: the other layered design, the llama shape
+TOKOVIK_PEER = {"tokovik-tiny": ("losarax-tiny", "tiny"), "tokovik-2k": ("losarax-2k", "llama-1b"), "tokovik-4k": ("losarax-4k", "llama-8b")}
+
+
+def tokovik_spec(shape: str, n_layers: int | None = None):
+    from .layered import PARALLEL, POST_NORM, SWIGLU, GatedSpec, LayerSpec, LayeredSpec, WindowSpec
+
+    width, layers, heads, kv, dim, vdim, window, rot, gh, gd, gv, rank, ff, vocab = TOKOVIK_SHAPES[shape]
+    one = LayerSpec(PARALLEL, ff=ff, mlp=SWIGLU, gated=GatedSpec(gh, gd, gv, rank, 16.0),
+                    window=WindowSpec(heads, kv, dim, vdim, window, float(dim ** -0.5), rot, 500000.0, 8.0, 8192.0, 32.0, 1.0))
+    return LayeredSpec(vocab=vocab, width=width, eps=1e-6, layers=[one] * (n_layers or layers), residual=POST_NORM, embed_scale=float(width ** 0.5))
+
+
+def layered_spec(shape: str, n_layers: int | None = None):
+    return (losarax_spec if shape in LOSARAX_SHAPES else tokovik_spec)(shape, n_layers)
+
+
 def build_layered(spec, seed: int, max_pos: int, max_seqs: int = 1, dtype: str = "bfloat16", **kw):
     """A layered engine with seeded random weights: matrices N(0, 1/cols), norms around 1, streams that stay bounded."""
-    from .layered import LayeredEngine
+    from .layered import POST_NORM, LayeredEngine
 
     eng = LayeredEngine(spec, max_pos, max_seqs, dtype, **kw)
     for i, (name, shape) in enumerate(eng.tensors().items()):
@@ -166,6 +189,8 @@ def build_layered(spec, seed: int, max_pos: int, max_seqs: int = 1, dtype: str =
             eng.synth_tensor(name, seed, i, 0.0, 0.1)
         elif name.endswith(".in"):
             eng.synth_tensor(name, seed, i, 1.0 / spec.streams, 0.1)
+        elif spec.residual == POST_NORM and name.endswith(("norm1", "norm2", "final.norm")):  # stored around zero
+            eng.synth_tensor(name, seed, i, 0.0, 0.1)
         else:
             eng.synth_tensor(name, seed, i, 1.0, 0.1)
     return eng
@@ -186,11 +211,15 @@ def layered_bytes(eng) -> int:
 
 def layered_context_bytes(eng, context: int, batch: int = 1) -> int:
     """Cache rows read (bfloat16) and states read and written (f32) by one decode step at that context."""
-    from .layered import LATENT
+    from .layered import LATENT, PARALLEL
 
     total = 0
     for i in eng.spec.runs:
         s = eng.spec.layers[i]
+        if s.type == PARALLEL:
+            w, g = s.window, s.gated
+            total += 2 * min(context, w.window or context) * w.kv_heads * (w.dim + w.vdim) + 8 * g.heads * g.dim * g.vdim
+            continue
         total += 2 * context * (s.kv_rank + s.rot_dim) if s.type == LATENT else 8 * s.heads * s.dim * s.vdim
     return total * batch
 
