@@ -54,6 +54,13 @@ __device__ __forceinline__ float ex2(float x) {
   return y;
 }
 
+// log2(sigmoid(z)); log(1 + e) by its series where e is small
+__device__ __forceinline__ float log2_sigmoid(float z) {
+  const float kLog2e = 1.44269504f, e = ex2(-fabsf(z) * kLog2e);
+  const float l = e > 0.015625f ? __log2f(1.0f + e) : e * kLog2e * fmaf(-e, fmaf(-e, 0.33333334f, 0.5f), 1.0f);
+  return fmaf(fminf(z, 0.0f), kLog2e, -l);
+}
+
 // Logarithms of decays are to base 2 in this kernel.
 __global__ void __launch_bounds__(kPrepThreads, 2) gated_prep_kernel(const LightningArgs a, uint8_t *scratch) {
   extern __shared__ __align__(16) uint8_t raw[];
@@ -118,7 +125,7 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gated_prep_kernel(const Light
     float run = 0.0f;
 #pragma unroll
     for (int t = 0; t < kSub; ++t) {
-      if (live && t0 + t < len) run += log_decay(z[t], a.channel.inv_tau * 1.44269504f);
+      if (live && t0 + t < len) run = fmaf(log2_sigmoid(z[t]), a.channel.inv_tau, run);
       lb[(t0 + t) * ld + d] = run;
     }
     T[i] = run;
@@ -151,107 +158,146 @@ __global__ void __launch_bounds__(kPrepThreads, 2) gated_prep_kernel(const Light
   }
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
-  // queries from the chunk's start, keys to its end
-#pragma unroll 2
-  for (int t = warp; t < kC; t += kPrepThreads / 32) {
-    const float *bt = before + t / kSub * dp, *rt = rest + t / kSub * dp;
-    for (int d = lane * 2; d < dp; d += 64) {
-      const float2 l = *reinterpret_cast<const float2 *>(lb + t * ld + d), qv = *reinterpret_cast<const float2 *>(q + t * ld + d);
-      const float2 kv = *reinterpret_cast<const float2 *>(k + t * ld + d), f = *reinterpret_cast<const float2 *>(bt + d);
-      const float2 r = *reinterpret_cast<const float2 *>(rt + d);
-      uint32_t hi, lo;
-      uint32_t *o = reinterpret_cast<uint32_t *>(o16 + t * dp + d);
-      split_pair(a.q_scale * qv.x * ex2(f.x + l.x), a.q_scale * qv.y * ex2(f.y + l.y), hi, lo);
-      o[0] = hi;
-      o[kC * dp / 2] = lo;
-      split_pair(kv.x * ex2(r.x - l.x), kv.y * ex2(r.y - l.y), hi, lo);
-      o[2 * kC * dp / 2] = hi;
-      o[3 * kC * dp / 2] = lo;
-    }
-  }
   bf16 *A = o16 + L.a;
   auto put = [&](int t, int s, float v) {
     const bf16 hi = __float2bfloat16_rn(v);
     A[t * kC + s] = hi;
     A[kC * kC + t * kC + s] = __float2bfloat16_rn(v - __bfloat162float(hi));
   };
-  // pairs of the same eight tokens: a warp takes eight tokens, its lanes the channels
-#pragma unroll 1
-  for (int e = 0; e < 8; ++e) {
-    const int t0 = warp * 8, t = t0 + e;
-    float v[8] = {};
-    for (int d = lane; d < dp; d += 32) {
-      const float qd = q[t * ld + d], l = lb[t * ld + d];
-#pragma unroll
-      for (int s = 0; s < 8; ++s)
-        if (s <= e) v[s] = fmaf(qd * k[(t0 + s) * ld + d], ex2(l - lb[(t0 + s) * ld + d]), v[s]);
-    }
-    float mine = 0.0f;
-#pragma unroll
-    for (int s = 0; s < 8; ++s) {
-      if (s > e) break;
-      const float f = warp_sum(v[s]);
-      if (lane == s) mine = f;
-    }
-    if (lane < 8) put(t, t0 + lane, a.q_scale * mine);  // zero above the diagonal
-    if (lane < 8 && (warp & 1) == 0) put(t, t0 + 8 + lane, 0.0f);
-  }
-  // blocks below the diagonal on the tensor cores, factored at a place between their queries and their keys: 16 x 16, task
-  // 0..5 = (1,0), (2,0), (2,1), (3,0), (3,1), (3,2); 8 x 8, task 6..9 = the two halves of 16 tokens
   const int tr = lane >> 2, tc = (lane & 3) * 2;
-#pragma unroll 1
-  for (int task = warp; task < 10; task += kPrepThreads / 32) {
-    const bool half = task >= 6;
-    const int bi = half ? task - 6 : task == 0 ? 1 : task < 3 ? 2 : 3, bj = half ? bi : task == 0 ? 0 : task < 3 ? task - 1 : task - 3;
-    const int tq = bi * kSub + (half ? 8 : 0), tk = bj * kSub;
-    const float *edge = half ? lb + (tk + 7) * ld : T + bj * dp;  // sum up to the last of the keys
-    float acc[2][4] = {};
-    auto qe = [&](int t, int d) {
-      const float2 l = *reinterpret_cast<const float2 *>(lb + t * ld + d), v = *reinterpret_cast<const float2 *>(q + t * ld + d);
-      float2 e = l;
-      if (half) {
-        e.x -= edge[d];
-        e.y -= edge[d + 1];
-      }
-      for (int s = bj + 1; s < bi; ++s) {
-        e.x += T[s * dp + d];
-        e.y += T[s * dp + d + 1];
-      }
-      return make_float2(v.x * ex2(e.x), v.y * ex2(e.y));
-    };
-    auto ke = [&](int s, int d) {
-      const float2 l = *reinterpret_cast<const float2 *>(lb + s * ld + d), v = *reinterpret_cast<const float2 *>(k + s * ld + d);
-      return make_float2(v.x * ex2(edge[d] - l.x), v.y * ex2(edge[d + 1] - l.y));
-    };
-#pragma unroll 1
-    for (int d0 = 0; d0 < dp; d0 += 16) {
-      uint32_t AH[4], AL[4];
+  {
+    // pairs within eight tokens: a warp takes eight, its lanes the channels
+    const int t0 = warp * 8;
+    float v[36] = {};
+    for (int d = lane; d < dp; d += 32) {
+      float kd[8], l[8];
 #pragma unroll
-      for (int f = 0; f < 4; ++f) {
-        AH[f] = AL[f] = 0;
-        if (half && (f & 1)) continue;  // eight queries only
-        const float2 v = qe(tq + tr + (f & 1) * 8, d0 + (f >> 1) * 8 + tc);
-        split_pair(v.x, v.y, AH[f], AL[f]);
+      for (int s = 0; s < 8; ++s) {
+        kd[s] = k[(t0 + s) * ld + d];
+        l[s] = lb[(t0 + s) * ld + d];
+      }
+#pragma unroll
+      for (int t = 0; t < 8; ++t) {
+        const float qd = q[(t0 + t) * ld + d];
+#pragma unroll
+        for (int s = 0; s <= t; ++s) v[t * (t + 1) / 2 + s] = fmaf(qd * kd[s], s < t ? ex2(l[t] - l[s]) : 1.0f, v[t * (t + 1) / 2 + s]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < 8; ++t) {
+      float mine = 0.0f;
+#pragma unroll
+      for (int s = 0; s <= t; ++s) {
+        const float f = warp_sum(v[t * (t + 1) / 2 + s]);
+        if (lane == s) mine = f;
+      }
+      if (lane < 8) put(t0 + t, t0 + lane, a.q_scale * mine);  // zero above the diagonal
+      if (lane >= 8 && lane < 16 && (warp & 1) == 0) put(t0 + t, t0 + lane, 0.0f);
+    }
+  }
+  if (warp < 4) {
+    // the second eight of 16 tokens against the first, factored at the last of those
+    const int tk = warp * kSub, tq = tk + 8;
+    const float *edge = lb + (tk + 7) * ld;
+    float acc[4] = {};
+#pragma unroll 2
+    for (int d0 = 0; d0 < dp; d0 += 16) {
+      uint32_t AH[4] = {}, AL[4] = {}, BH[2], BL[2];
+#pragma unroll
+      for (int f = 0; f < 2; ++f) {
+        const int d = d0 + f * 8 + tc;
+        const float2 e = *reinterpret_cast<const float2 *>(edge + d);
+        const float2 lq = *reinterpret_cast<const float2 *>(lb + (tq + tr) * ld + d), qv = *reinterpret_cast<const float2 *>(q + (tq + tr) * ld + d);
+        const float2 lk = *reinterpret_cast<const float2 *>(lb + (tk + tr) * ld + d), kv = *reinterpret_cast<const float2 *>(k + (tk + tr) * ld + d);
+        split_pair(qv.x * ex2(lq.x - e.x), qv.y * ex2(lq.y - e.y), AH[2 * f], AL[2 * f]);
+        split_pair(kv.x * ex2(e.x - lk.x), kv.y * ex2(e.y - lk.y), BH[f], BL[f]);
+      }
+      mma16816(acc, AH, BH[0], BH[1]);
+      mma16816(acc, AH, BL[0], BL[1]);
+      mma16816(acc, AL, BH[0], BH[1]);
+    }
+    put(tq + tr, tk + tc, a.q_scale * acc[0]);
+    put(tq + tr, tk + tc + 1, a.q_scale * acc[1]);
+  }
+  __syncthreads();
+  // queries from the start of their 16 tokens, keys to the end of theirs: as two bf16 terms in place of the 32-bit rows
+  // ([hi | lo] of dp each), and to the chunk's edges for the scan
+#pragma unroll 2
+  for (int t = warp; t < kC; t += kPrepThreads / 32) {
+    const int sub = t / kSub;
+    const float *Ts = T + sub * dp, *bt = before + sub * dp, *rt = rest + (sub + 1) * dp;
+    bf16 *qt = reinterpret_cast<bf16 *>(q + t * ld), *kt = reinterpret_cast<bf16 *>(k + t * ld);
+    for (int d0 = 0; d0 < dp; d0 += 256) {  // up to 256 channels in registers between the reads and the writes of a row
+      uint32_t w[4][4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int d = d0 + j * 64 + lane * 2;
+        if (d >= dp) break;
+        const float2 l = *reinterpret_cast<const float2 *>(lb + t * ld + d), qv = *reinterpret_cast<const float2 *>(q + t * ld + d);
+        const float2 kv = *reinterpret_cast<const float2 *>(k + t * ld + d), e = *reinterpret_cast<const float2 *>(Ts + d);
+        const float2 f = *reinterpret_cast<const float2 *>(bt + d), r = sub < 3 ? *reinterpret_cast<const float2 *>(rt + d) : make_float2(0.0f, 0.0f);
+        const float2 qe = make_float2(a.q_scale * qv.x * ex2(l.x), a.q_scale * qv.y * ex2(l.y)), ke = make_float2(kv.x * ex2(e.x - l.x), kv.y * ex2(e.y - l.y));
+        split_pair(qe.x, qe.y, w[j][0], w[j][1]);
+        split_pair(ke.x, ke.y, w[j][2], w[j][3]);
+        uint32_t hi, lo;
+        uint32_t *o = reinterpret_cast<uint32_t *>(o16 + t * dp + d);
+        split_pair(qe.x * ex2(f.x), qe.y * ex2(f.y), hi, lo);
+        o[0] = hi;
+        o[kC * dp / 2] = lo;
+        split_pair(ke.x * ex2(r.x), ke.y * ex2(r.y), hi, lo);
+        o[2 * kC * dp / 2] = hi;
+        o[3 * kC * dp / 2] = lo;
+      }
+      __syncwarp();
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int d = d0 + j * 64 + lane * 2;
+        if (d >= dp) break;
+        *reinterpret_cast<uint32_t *>(qt + d) = w[j][0];
+        *reinterpret_cast<uint32_t *>(qt + dp + d) = w[j][1];
+        *reinterpret_cast<uint32_t *>(kt + d) = w[j][2];
+        *reinterpret_cast<uint32_t *>(kt + dp + d) = w[j][3];
+      }
+    }
+  }
+  __syncthreads();
+  // blocks of 16 x 16 below the diagonal: warp 0..5 = (1,0), (2,0), (2,1), (3,0), (3,1), (3,2)
+  if (warp < 6) {
+    const int bi = warp == 0 ? 1 : warp < 3 ? 2 : 3, bj = warp == 0 ? 0 : warp < 3 ? warp - 1 : warp - 3;
+    const bf16 *q16 = reinterpret_cast<const bf16 *>(q + bi * kSub * ld), *k16 = reinterpret_cast<const bf16 *>(k + bj * kSub * ld);
+    float acc[2][4] = {};
+#pragma unroll 2
+    for (int d0 = 0; d0 < dp; d0 += 16) {
+      uint32_t AH[4], AL[4], BH[4], BL[4];
+      const bf16 *qa = q16 + (lane & 15) * 2 * ld + d0 + (lane >> 4) * 8;
+      const bf16 *kb = k16 + ((lane & 7) + ((lane >> 4) << 3)) * 2 * ld + d0 + ((lane >> 3) & 1) * 8;
+      ldsm4(AH, qa);
+      ldsm4(AL, qa + dp);
+      ldsm4(BH, kb);
+      ldsm4(BL, kb + dp);
+      if (bi - bj > 1) {  // the 16s in between
+#pragma unroll
+        for (int f = 0; f < 4; ++f) {
+          float2 g = make_float2(0.0f, 0.0f);
+          for (int s = bj + 1; s < bi; ++s) {
+            const float2 e = *reinterpret_cast<const float2 *>(T + s * dp + d0 + (f >> 1) * 8 + tc);
+            g.x += e.x;
+            g.y += e.y;
+          }
+          split_pair((bf16_lo(AH[f]) + bf16_lo(AL[f])) * ex2(g.x), (bf16_hi(AH[f]) + bf16_hi(AL[f])) * ex2(g.y), AH[f], AL[f]);
+        }
       }
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
-        if (half && n) continue;
-        uint32_t BH[2], BL[2];
-#pragma unroll
-        for (int f = 0; f < 2; ++f) {
-          const float2 v = ke(tk + n * 8 + tr, d0 + f * 8 + tc);
-          split_pair(v.x, v.y, BH[f], BL[f]);
-        }
-        mma16816(acc[n], AH, BH[0], BH[1]);
-        mma16816(acc[n], AH, BL[0], BL[1]);
-        mma16816(acc[n], AL, BH[0], BH[1]);
+        mma16816(acc[n], AH, BH[2 * n], BH[2 * n + 1]);
+        mma16816(acc[n], AH, BL[2 * n], BL[2 * n + 1]);
+        mma16816(acc[n], AL, BH[2 * n], BH[2 * n + 1]);
       }
     }
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (!half || (n == 0 && e < 2)) put(tq + tr + (e >> 1) * 8, tk + n * 8 + tc + (e & 1), a.q_scale * acc[n][e]);
+      for (int e = 0; e < 4; ++e) put(bi * kSub + tr + (e >> 1) * 8, bj * kSub + n * 8 + tc + (e & 1), acc[n][e]);
   }
   if (a.late_wait) pdl_wait();
 }

@@ -374,8 +374,8 @@ __global__ void __launch_bounds__(kPfThreads) window_prefill_kernel(const Window
   const WindowShape &m = a.m;
   const int kp = window_pad(m.dim), vp = window_pad(m.vdim), QS = kp + 8, VS = DV + 8;
   bf16 *q_s = sh, *k_s = q_s + kPfQ * QS, *v_s = k_s + 2 * kPfK * QS;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, g = h / (m.heads / m.kv_heads);
-  const int r0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * kPfQ;  // the longest rows first
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x, g = h / (m.heads / m.kv_heads);
+  const int r0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * kPfQ;  // the longest rows of all heads first
   pdl_wait();
   pdl_launch();
   const int start = a.positions[0] + r0, last = start + min(kPfQ, a.rows - r0) - 1;  // positions of this tile's queries
@@ -552,7 +552,7 @@ int32_t prefill(const WindowArgs &a, bool pdl, cudaStream_t s) {
     CMLD_TRY(allow_smem(window_prefill_kernel<DV>, kMaxSmem));
     ready = true;
   }
-  return launch_kernel(window_prefill_kernel<DV>, dim3((a.rows + kPfQ - 1) / kPfQ, a.m.heads), dim3(kPfThreads), pf_smem(window_pad(a.m.dim), DV), pdl, s, a);
+  return launch_kernel(window_prefill_kernel<DV>, dim3(a.m.heads, (a.rows + kPfQ - 1) / kPfQ), dim3(kPfThreads), pf_smem(window_pad(a.m.dim), DV), pdl, s, a);
 }
 
 size_t plain_smem(const WindowShape &m) { return (size_t)(m.dim + 8 * m.vdim) * 4; }
