@@ -386,11 +386,22 @@ __device__ __forceinline__ float2 cta_total2(float2 v, float *red) {
 }
 __device__ __forceinline__ float dot4(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
 
-// x + y' of a single stream (see StreamMix); put(i, v) takes values 4i .. 4i + 3 of the result.  The row stays in registers,
+// x + y' of a single stream, or its embedding row (see StreamMix); put(i, v) takes values 4i .. 4i + 3 of the result.  The row stays in registers,
 // V times four values per thread (width a multiple of four, at most 4 V blockDim.x).  `red` holds 2 * blockDim.x / 32 floats.
 template <int V, typename Put>
 __device__ __forceinline__ void post_norm_row(const StreamMix &m, int64_t row, float *red, Put put) {
   const int n4 = m.width / 4;
+  if (m.embed) {
+    const uint2 *e = reinterpret_cast<const uint2 *>(m.embed + (int64_t)m.tokens[row] * m.embed_ld);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const int i = threadIdx.x + j * blockDim.x;
+      if (i >= n4) break;
+      const uint2 v = e[i];
+      put(i, make_float4(m.embed_scale * bf16_lo(v.x), m.embed_scale * bf16_hi(v.x), m.embed_scale * bf16_lo(v.y), m.embed_scale * bf16_hi(v.y)));
+    }
+    return;
+  }
   const float4 *x = reinterpret_cast<const float4 *>(m.x_in + row * m.width), *y = reinterpret_cast<const float4 *>(m.y + row * m.width);
   float4 xv[V], yv[V];
 #pragma unroll

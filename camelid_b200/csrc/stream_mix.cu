@@ -20,7 +20,8 @@ __global__ void __launch_bounds__(kMixThreads) stream_mix_kernel(const StreamMix
   for (int i = threadIdx.x; i < m.width; i += blockDim.x) act_store(out.p, out.half, r * out.ld + i, u[i]);
 }
 
-// One stream with norms on the sublayers' outputs and no norm in front of the next: the row stays in registers.
+// One stream with norms on the sublayers' outputs (or the embedding) and no norm in front of the next: the row stays in
+// registers.
 template <int V>
 __global__ void __launch_bounds__(V == 4 ? 512 : kMixThreads) post_norm_kernel(const __grid_constant__ StreamMix m, ActBuf out) {
   __shared__ __align__(8) float red[2 * kMixThreads / 32];
@@ -86,7 +87,7 @@ __global__ void __launch_bounds__(256) rms_groups_kernel(const float *x, int64_t
 }  // namespace
 
 int32_t launch_stream_mix(const StreamMix &m, int32_t rows, ActBuf out, bool pdl, cudaStream_t s) {
-  if (!m.embed && !m.mix && !m.norm_w && !m.row_map && m.width % 4 == 0 && m.width <= 8192 && out.ld % 4 == 0) {
+  if (!m.mix && !m.enorm_w && m.streams == 1 && !m.in && !m.norm_w && !m.row_map && m.width % 4 == 0 && m.width <= 8192 && out.ld % 4 == 0) {
     // many rows: small CTAs, several values per thread
     const int n4 = m.width / 4, per = rows >= 256 ? 4 : 1, threads = std::min(per == 4 ? 512 : kMixThreads, ((n4 + per - 1) / per + 31) & ~31);
     const int v = (n4 + threads - 1) / threads;
