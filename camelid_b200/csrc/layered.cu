@@ -200,10 +200,11 @@ struct Rotation {
   }
 };
 
-// Angles position * frequency in 32-bit, their cosine and sine: [position][pair][2].
+// Cosine and sine of position * frequency, formed in 64-bit on the host: [position][pair][2] in 32-bit.
 int32_t rotation_table(cmld_engine *e, int64_t max_pos, const Rotation &r, float **out) {
   const int dims = r.dims, half = dims / 2;
-  std::vector<float> f(half), t((size_t)max_pos * dims);
+  std::vector<double> f(half);
+  std::vector<float> t((size_t)max_pos * dims);
   double lo = 0.0, hi = 0.0, gain = 1.0;
   if (r.factor > 0.0) {
     auto place = [&](double turns) { return dims * std::log(r.original / (2.0 * M_PI * turns)) / (2.0 * std::log(r.base)); };
@@ -217,13 +218,13 @@ int32_t rotation_table(cmld_engine *e, int64_t max_pos, const Rotation &r, float
       const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
       v = v / r.factor * ramp + v * (1.0 - ramp);
     }
-    f[i] = (float)v;
+    f[i] = v;
   }
   for (int64_t p = 0; p < max_pos; ++p)
     for (int i = 0; i < half; ++i) {
-      const float a = (float)p * f[i];
-      t[(size_t)p * dims + 2 * i] = (float)(gain * std::cos((double)a));
-      t[(size_t)p * dims + 2 * i + 1] = (float)(gain * std::sin((double)a));
+      const double a = (double)p * f[i];
+      t[(size_t)p * dims + 2 * i] = (float)(gain * std::cos(a));
+      t[(size_t)p * dims + 2 * i + 1] = (float)(gain * std::sin(a));
     }
   CMLD_TRY(dev_alloc(e, out, (int64_t)t.size(), false));
   CMLD_CUDA(cudaMemcpyAsync(*out, t.data(), t.size() * 4, cudaMemcpyHostToDevice, e->stream));

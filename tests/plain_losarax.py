@@ -1,6 +1,6 @@
 """A plain, slow evaluation of the Losarax design in numpy, one function per mechanism, for the tests to compare the
-engine with.  Everything runs over a whole sequence at once in float64 (rotation angles are formed in float32, as
-the engine forms them); there is no cache, no state carried between calls and no code shared with the package.
+engine with.  Everything runs over a whole sequence at once in float64; there is no cache, no state carried between calls
+and no code shared with the package.
 
 ``params`` maps tensor names to arrays, ``cfg`` is the parsed config.json.
 """
@@ -32,9 +32,9 @@ def linear(w, x):
 
 def rotate_interleaved(x, positions, dims, base):
     """x[tokens, ..., n]: pairs (2i, 2i+1) of the first `dims` values turn by position * base^(-2i/dims)."""
-    f = np.array([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)]).astype(np.float32)
-    a = np.asarray(positions, np.float32)[:, None] * f[None, :]
-    a = a.astype(np.float64).reshape((x.shape[0],) + (1,) * (x.ndim - 2) + (dims // 2,))
+    f = np.array([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)])
+    a = np.asarray(positions, np.float64)[:, None] * f[None, :]
+    a = a.reshape((x.shape[0],) + (1,) * (x.ndim - 2) + (dims // 2,))
     out = np.array(x, np.float64)
     u, v = x[..., 0:dims:2], x[..., 1:dims:2]
     out[..., 0:dims:2] = u * np.cos(a) - v * np.sin(a)

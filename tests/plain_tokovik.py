@@ -1,6 +1,6 @@
 """A plain, slow evaluation of the Tokovik design in numpy, one function per mechanism, for the tests to compare the
-engine with.  Everything runs over a whole sequence at once in float64 (rotation angles are formed in float32, as
-the engine forms them); there is no cache, no state carried between calls and no code shared with the package.
+engine with.  Everything runs over a whole sequence at once in float64; there is no cache, no state carried between calls
+and no code shared with the package.
 
 ``params`` maps tensor names to arrays, ``cfg`` is the parsed config.json.
 """
@@ -46,8 +46,8 @@ def rotated_halves(x, positions, rot):
     """x[tokens, ..., n]: dimension i turns together with dimension i + dims / 2, i < dims / 2; the rest passes."""
     half = rot["dims"] // 2
     f, m = yarn_frequencies(rot)
-    a = np.asarray(positions, np.float32)[:, None] * np.array(f).astype(np.float32)[None, :]
-    a = a.astype(np.float64).reshape((x.shape[0],) + (1,) * (x.ndim - 2) + (half,))
+    a = np.asarray(positions, np.float64)[:, None] * np.array(f)[None, :]
+    a = a.reshape((x.shape[0],) + (1,) * (x.ndim - 2) + (half,))
     c, s = m * np.cos(a), m * np.sin(a)
     out = np.array(x, np.float64)
     u, v = x[..., :half], x[..., half:2 * half]
